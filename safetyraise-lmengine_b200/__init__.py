@@ -7,6 +7,7 @@ the scheduler), ``SamplingParams``, and the command line
 ``python -m safetyraise_lmengine_b200 inspect|run|benchmark|replay``.
 """
 from .config import dovorax as _dovorax
+from .config import lokizen as _lokizen
 from .config import nekedra as _nekedra
 from .config import qwen3 as _qwen3
 from .config import pabalorn as _pabalorn
@@ -27,6 +28,7 @@ register_architecture(_tonanex.ARCHITECTURE, _tonanex.read_spec, _build_decoder)
 register_architecture(_pabalorn.ARCHITECTURE, _pabalorn.read_spec, _build_decoder)
 
 register_architecture(_dovorax.ARCHITECTURE, _dovorax.read_spec, _build_decoder)
+register_architecture(_lokizen.ARCHITECTURE, _lokizen.read_spec, _build_decoder)
 
 __version__ = "0.1.0"
 

@@ -35,6 +35,7 @@ class CacheGroupSpec:
     state_shape: Tuple[int, ...] = ()
     state_dtype: torch.dtype = torch.float32
     v_head_dim: Optional[int] = None         # None: values as wide as keys; 0: no value pool; else their own size
+    keep_first: int = 0                      # window groups: the first tokens of a sequence, whose pages stay
 
     @property
     def value_dim(self) -> int:
@@ -56,7 +57,7 @@ class CacheGroupSpec:
             return len(self.entries) * n * self.state_dtype.itemsize
         tokens = context
         if self.kind == PAGED_WINDOW and self.window:
-            tokens = min(context, self.window + page_size)
+            tokens = min(context, self.window + page_size + -(-self.keep_first // page_size) * page_size)
         return self.bytes_per_token(dtype) * -(-tokens // page_size) * page_size
 
 
@@ -69,7 +70,7 @@ def runtime():
         from ..csrc.build import build_runtime
         lib = C.CDLL(build_runtime())
         lib.srlm_cache_create.restype = C.c_void_p
-        lib.srlm_cache_create.argtypes = [C.c_int, C.c_int] + [C.POINTER(C.c_int)] * 4
+        lib.srlm_cache_create.argtypes = [C.c_int, C.c_int] + [C.POINTER(C.c_int)] * 5
         lib.srlm_sched_create.restype = C.c_void_p
         lib.srlm_sched_create.argtypes = [C.c_void_p] + [C.c_int] * 5
         for name in ("open", "close", "reserve", "fit_tokens", "commit", "truncate", "length", "reserved",
@@ -120,7 +121,7 @@ class CacheManager:
             max_requests, n,
             arr([1 if g.kind == PAGED_WINDOW else 0 for g in self._paged]),
             arr([page_size] * n), arr([num_pages] * n),
-            arr([g.window or 0 for g in self._paged]))
+            arr([g.window or 0 for g in self._paged]), arr([g.keep_first for g in self._paged]))
         if not self._h:
             raise ConfigError("the cache manager refused its configuration")
         # device memory: per paged group [entries, 2, num_pages, kv_heads, page_size, head_dim]:

@@ -211,6 +211,73 @@ class DistanceAttentionSpec(MixerSpec):
 
 
 @dataclass(frozen=True)
+class MixedHeadAttentionNames:
+    """Tensor names of an attention whose heads share their weights, each appended to its layer's ``weight_prefix``."""
+    q: str = "mix.q"
+    k: str = "mix.k"
+    v: str = "mix.v"
+    o: str = "mix.o"
+    q_norm: str = "mix.q.norm"              # [heads * head_dim]
+    k_norm: str = "mix.k.norm"              # [kv_heads * head_dim]
+    distance_bias: str = "mix.rel"          # [buckets, heads]; the number of buckets is the tensor's
+    head_mix: str = "mix.talk"              # [heads, heads]
+    gate: str = "mix.g"                     # [heads * v_head_dim, hidden]
+
+
+@dataclass(frozen=True)
+class MixedHeadAttentionSpec(MixerSpec):
+    """Grouped-query attention without a rotation, with a learned bias per bucket of distances, over a sliding window that
+    never lets go of a sequence's first tokens, whose heads exchange their weights behind the softmax:
+
+        score_h(i, j) = (q_i . k_j) * softmax_scale + bias[bucket(i - j), h],   0 <= i - j and (i - j < window or j < keep_first)
+        p_h = softmax_j(score_h);   w_h = sum_g head_mix[h, g] p_g;   out_h = sum_j w_h(i, j) v_j   (v of h's own KV head)
+
+    q and k are RMS-normed over all heads at once when ``qk_norm_eps`` is given; with B rows of bias, h = B / 2 and
+    D = bias_max, bucket(n) = n for n < h, else min(B - 1, h + floor(ln(n / h) / ln(D / h) (B - h))).  ``output_gate``:
+    every element of the heads' outputs is multiplied by the logistic of its own row of a projection of the input."""
+    hidden_size: int = 0
+    heads: int = 0
+    kv_heads: int = 0
+    head_dim: int = 0                       # query / key size
+    v_head_dim: int = 0                     # value size
+    softmax_scale: float = 0.0
+    qk_norm_eps: Optional[float] = None     # None: q and k as projected
+    bias_max: Optional[float] = None        # None: no bias by distance
+    window: Optional[int] = None            # None: every earlier key is visible
+    keep_first: int = 0                     # with a window: keys of the first tokens that stay visible behind it
+    head_mix: bool = True                   # False: every head applies its own weights
+    output_gate: bool = True
+    names: MixedHeadAttentionNames = MixedHeadAttentionNames()
+
+
+@dataclass(frozen=True)
+class RetentionNames:
+    q: str = "mix.q"
+    k: str = "mix.k"
+    v: str = "mix.v"
+    gate: str = "mix.g"                     # [heads * v_head_dim, hidden]
+    o: str = "mix.o"
+
+
+@dataclass(frozen=True)
+class RetentionSpec(MixerSpec):
+    """A linear attention whose matrix of state S [head_dim, v_head_dim] per head fades at a fixed rate:
+
+        S <- decay_h S + k v^T;   o = S^T q,   q = R(W_q h),  k = R(W_k h) / sqrt(head_dim),  v = W_v h
+        out = W_o (U(o) * silu(W_g h))          R: the rotary encoding; U: each head over its root mean square
+
+    S starts at zero and is float32."""
+    hidden_size: int = 0
+    heads: int = 0
+    head_dim: int = 0
+    v_head_dim: int = 0
+    decay: Tuple[float, ...] = ()           # one number per head
+    position: Optional[PositionSpec] = None
+    norm_eps: float = 1e-6
+    names: RetentionNames = RetentionNames()
+
+
+@dataclass(frozen=True)
 class RotatedAttentionNames:
     """Tensor names of a rotated attention mixer, each appended to its layer's ``weight_prefix``; a bias is its
     weight's name + ``bias_suffix``."""
@@ -403,6 +470,7 @@ class RoutedExpertsNames:
     """Tensor names of a routed feed-forward; expert e's tensors start with ``expert.format(e)``."""
     router: str = "mlp.router"
     router_bias: str = "mlp.router.b"
+    correction: str = "mlp.correction"      # [experts]
     expert: str = "mlp.e{}."
     shared: str = "mlp.shared."
     gate: str = "gate"
@@ -432,7 +500,11 @@ class RoutedExpertsSpec(FeedForwardSpec):
     weight_on_input: bool = False           # a weight multiplies its expert's input instead of its output
     groups: int = 1
     groups_kept: int = 1
-    gated: bool = True                      # False: an expert is W_down act(W_up h) (activation "gelu"), and so is the shared one
+    gated: bool = True                      # False: an expert is W_down act(W_up h) (activation "gelu", or "relu_squared":
+                                            # max(z, 0)^2), and so is the shared one
+    correction: bool = False                # scoring "logistic": the experts are chosen by their scores plus a learned number
+                                            # each; the weights are the scores without it
+    weight_scale: float = 1.0               # a factor on every weight
     expert_names: RoutedExpertsNames = RoutedExpertsNames()
 
 
@@ -463,6 +535,7 @@ class RunStep:
     cache: int                 # cache entry (per-step key/value or state storage) it uses
     writes_cache: bool = True  # False: reads what another step wrote under ``cache``
     more_caches: Tuple[int, ...] = ()   # a mixer made of several (side by side): the entries of the second, third, ...
+    add_embedding: bool = False         # what the embedding left (the stream ahead of the first run step) joins the stream first
 
 
 @dataclass(frozen=True)
@@ -483,6 +556,7 @@ class ModelSpec:
     embed_position_name: str = "model.embed_positions.weight"
     embed_norm: Optional[NormSpec] = None           # a norm of the embedded tokens before the first layer
     embed_norm_name: str = "embed.norm"
+    embed_scale: float = 1.0                        # a factor on the embedded tokens
     logit_softcap: Optional[float] = None           # logits <- cap * tanh(logits / cap)
     extra: dict = field(default_factory=dict, compare=False)
 

@@ -55,6 +55,10 @@ int CacheManager::first_needed_page(const Group& g, int length) const {
   return first_key / g.spec.page_size;
 }
 
+int CacheManager::kept_pages(const Group& g) const {
+  return g.spec.kind == GROUP_WINDOW ? ceil_div(g.spec.keep_first, g.spec.page_size) : 0;
+}
+
 int CacheManager::reserve(int slot, int new_len) {
   if (!valid(slot) || new_len < 0) return -1;
   Slot& s = slots_[slot];
@@ -101,7 +105,7 @@ int CacheManager::commit(int slot, int new_len) {
   for (size_t g = 0; g < groups_.size(); ++g) {
     Group& grp = groups_[g];
     int first = std::min(first_needed_page(grp, new_len), static_cast<int>(s.tables[g].size()));
-    for (int p = 0; p < first; ++p) {
+    for (int p = kept_pages(grp); p < first; ++p) {
       if (s.tables[g][p] >= 0) {
         grp.free_list.push_back(s.tables[g][p]);
         s.tables[g][p] = -1;
@@ -118,8 +122,10 @@ int CacheManager::truncate(int slot, int len) {
   if (len < s.length) {
     for (size_t g = 0; g < groups_.size(); ++g) {
       const Group& grp = groups_[g];
-      int first = first_needed_page(grp, len);
-      if (first < static_cast<int>(s.tables[g].size()) && s.tables[g][first] < 0) return -3;
+      // pages come back in order, the kept ones never: the first page that len's window needs behind the kept ones tells
+      int first = std::max(first_needed_page(grp, len), kept_pages(grp));
+      if (first < static_cast<int>(s.tables[g].size()) && s.tables[g][first] < 0 &&
+          first < ceil_div(len, grp.spec.page_size)) return -3;
     }
   }
   for (size_t g = 0; g < groups_.size(); ++g) {
@@ -161,7 +167,7 @@ int CacheManager::peak_pages(int group, int total_len, int max_step) const {
   if (s.kind != GROUP_WINDOW) return all;
   // a step of max_step tokens needs its own keys and the window before its first query,
   // which may straddle one more page at each end
-  return std::min(all, ceil_div(s.window + max_step, s.page_size) + 1);
+  return std::min(all, ceil_div(s.window + max_step, s.page_size) + 1 + kept_pages(groups_[group]));
 }
 
 int CacheManager::audit() const {

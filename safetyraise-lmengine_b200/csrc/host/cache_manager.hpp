@@ -26,6 +26,7 @@ struct GroupSpec {
   int page_size;
   int num_pages;
   int window;  // tokens a query sees, itself included; only for GROUP_WINDOW
+  int keep_first = 0;  // first tokens of a sequence that stay visible behind the window: their pages are never given back early
 };
 
 class CacheManager {
@@ -76,6 +77,7 @@ class CacheManager {
     std::vector<std::vector<int32_t>> tables;  // [group][page index] -> page id or -1
   };
   int first_needed_page(const Group& g, int length) const;
+  int kept_pages(const Group& g) const;     // leading pages that hold tokens every later query sees
   bool valid(int slot) const { return slot >= 0 && slot < max_requests() && slots_[slot].open; }
 
   std::vector<Group> groups_;

@@ -11,13 +11,13 @@ using srlm::Scheduler;
 extern "C" {
 
 void* srlm_cache_create(int max_requests, int n_groups, const int* kinds, const int* page_sizes,
-                        const int* num_pages, const int* windows) {
+                        const int* num_pages, const int* windows, const int* keep_first) {
   if (max_requests <= 0 || n_groups < 0) return nullptr;
   std::vector<srlm::GroupSpec> groups;
   for (int g = 0; g < n_groups; ++g) {
     if (page_sizes[g] <= 0 || num_pages[g] <= 0) return nullptr;
-    if (kinds[g] == srlm::GROUP_WINDOW && windows[g] <= 0) return nullptr;
-    groups.push_back(srlm::GroupSpec{kinds[g], page_sizes[g], num_pages[g], windows[g]});
+    if (kinds[g] == srlm::GROUP_WINDOW && (windows[g] <= 0 || keep_first[g] < 0)) return nullptr;
+    groups.push_back(srlm::GroupSpec{kinds[g], page_sizes[g], num_pages[g], windows[g], keep_first[g]});
   }
   return new CacheManager(max_requests, groups);
 }

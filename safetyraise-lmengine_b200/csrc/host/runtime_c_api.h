@@ -9,7 +9,7 @@ extern "C" {
 #endif
 
 void* srlm_cache_create(int max_requests, int n_groups, const int* kinds, const int* page_sizes,
-                        const int* num_pages, const int* windows);
+                        const int* num_pages, const int* windows, const int* keep_first);
 void srlm_cache_destroy(void* cache);
 int srlm_cache_open(void* cache);
 int srlm_cache_close(void* cache, int slot);

@@ -24,18 +24,21 @@ __global__ void patch_words_kernel(int* __restrict__ words, long long words_len,
 
 template <typename TW>
 __global__ void embed_gather_kernel(const int* __restrict__ ids, const TW* __restrict__ table,
-                                    float* __restrict__ out, int H, int vocab, int* __restrict__ bad) {
+                                    float* __restrict__ out, int H, int vocab, int* __restrict__ bad, float scale, int add) {
   pdl_wait();
   pdl_trigger();
   const int t = blockIdx.x;
   const int id = ids[t];
   if (id < 0 || id >= vocab) {          // the host checks too; never read outside the table
     if (threadIdx.x == 0) atomicExch(bad, 1);
-    for (int i = threadIdx.x; i < H; i += blockDim.x) out[(size_t)t * H + i] = 0.f;
+    for (int i = threadIdx.x; i < H && !add; i += blockDim.x) out[(size_t)t * H + i] = 0.f;
     return;
   }
   const TW* row = table + (size_t)id * H;
-  for (int i = threadIdx.x; i < H; i += blockDim.x) out[(size_t)t * H + i] = to_float(row[i]);
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    const float v = to_float(row[i]) * scale;
+    out[(size_t)t * H + i] = add ? out[(size_t)t * H + i] + v : v;
+  }
 }
 
 // x = residual[src] (+ delta[src]); residual[src] = x when rows == nullptr;
@@ -208,12 +211,12 @@ static inline int flat_grid(size_t n, int block) {
 using namespace srlm;
 
 extern "C" int srlm_embed_gather(const int* ids, const void* table, int table_dtype, float* out, int T,
-                                 int H, int vocab, int* bad_flag, cudaStream_t stream) {
+                                 int H, int vocab, int* bad_flag, float scale, int add, cudaStream_t stream) {
   if (T <= 0) return ST_OK;
   if (H <= 0 || vocab <= 0) return refuse(ST_BAD_SIZE, "embed_gather: H=%d vocab=%d", H, vocab);
   const int block = H >= 1024 ? 256 : 128;
   SRLM_DISPATCH_ACT(table_dtype, TW, launch_pdl(embed_gather_kernel<TW>, dim3(T), dim3(block), 0, stream,
-      ids, (const TW*)table, out, H, vocab, bad_flag));
+      ids, (const TW*)table, out, H, vocab, bad_flag, scale, add));
   return launched();
 }
 

@@ -36,19 +36,25 @@ __device__ __forceinline__ float clamped_glu(float gate, float up, float limit, 
   return g * (1.f / (1.f + expf(-alpha * g))) * (u + 1.f);
 }
 
-// The activation of an expert without a gate: 0 none, 1 the exact gelu.
+// The activation of an expert without a gate: 0 none, 1 the exact gelu, 2 the square of the positive part.
 __device__ __forceinline__ float plain_activation(float z, int act) {
+  if (act == 2) return z < 0.f ? 0.f : z * z;      // (a NaN stays one)
   return act == 1 ? 0.5f * z * (1.f + erff(z * 0.70710678118654752440f)) : z;
 }
 
 // One warp routes a token.  The row of logits sits in shared memory (z: E floats of the warp's own); `top` times
 // the warp takes the largest value left (ties: the lowest index) and strikes it out.  weights = softmax over the
-// chosen values; scoring 1: weight = logistic of the chosen value itself.
+// chosen values; scoring 1: weight = logistic of the chosen value itself, the choice by that logistic plus the
+// expert's `correction` when there is one (the weight does not see it).  Every weight is multiplied by wscale.
 __device__ __forceinline__ void route_token(const float* __restrict__ logits, long long ld, const float* __restrict__ bias,
                                             int t, int E, int top, float* z, int* __restrict__ choice,
-                                            float* __restrict__ weight, int scoring, int groups, int kept) {
+                                            float* __restrict__ weight, int scoring, int groups, int kept,
+                                            const float* __restrict__ correction, float wscale) {
   const int lane = threadIdx.x & 31;
-  for (int e = lane; e < E; e += 32) z[e] = logits[(size_t)t * ld + e] + (bias ? bias[e] : 0.f);
+  for (int e = lane; e < E; e += 32) {
+    const float v = logits[(size_t)t * ld + e] + (bias ? bias[e] : 0.f);
+    z[e] = correction ? 1.f / (1.f + expf(-v)) + correction[e] : v;
+  }
   __syncwarp();
   float first = 0.f, sum = 0.f;
   float z_max = 0.f, z_den = 1.f;          // scoring 2: score(e) = exp(z[e] - z_max) / z_den
@@ -102,7 +108,8 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, lo
     }
     if (at >= E) at = c < E ? c : 0;            // a row of NaN: any valid expert; the step's finite check reports it
     if (c == 0) first = best;
-    const float p = scoring == 1 ? 1.f / (1.f + expf(-best)) : scoring == 2 ? expf(best - z_max) / z_den : expf(best - first);
+    if (correction) best = logits[(size_t)t * ld + at] + (bias ? bias[at] : 0.f);      // the weight is the score without it
+    const float p = scoring == 1 ? wscale / (1.f + expf(-best)) : scoring == 2 ? expf(best - z_max) / z_den : expf(best - first);
     sum += p;
     if (lane == 0) {
       choice[(size_t)t * top + c] = at;
@@ -113,22 +120,23 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, lo
   }
   __syncwarp();
   if (scoring == 0)
-    for (int c = lane; c < top; c += 32) weight[(size_t)t * top + c] /= sum;
+    for (int c = lane; c < top; c += 32) weight[(size_t)t * top + c] = weight[(size_t)t * top + c] / sum * wscale;
   if (scoring == 2)
-    for (int c = lane; c < top; c += 32) weight[(size_t)t * top + c] /= sum + 1e-20f;
+    for (int c = lane; c < top; c += 32) weight[(size_t)t * top + c] = weight[(size_t)t * top + c] / (sum + 1e-20f) * wscale;
   __syncwarp();
 }
 
 __global__ void moe_route_kernel(const float* __restrict__ logits, long long ld, const float* __restrict__ bias,
                                  int T, int E, int top, int* __restrict__ choice, float* __restrict__ weight, int scoring,
-                                 int groups, int kept) {
+                                 int groups, int kept, const float* __restrict__ correction, float wscale) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ float route_smem[];
   const int warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
   const int t = blockIdx.x * warps + warp;
   if (t >= T) return;
-  route_token(logits, ld, bias, t, E, top, route_smem + (size_t)warp * E, choice, weight, scoring, groups, kept);
+  route_token(logits, ld, bias, t, E, top, route_smem + (size_t)warp * E, choice, weight, scoring, groups, kept, correction,
+              wscale);
 }
 
 // One block.  offsets[E + 1]: first row of each expert; tiles[E + 1]: first tile of each expert (tiles of
@@ -143,7 +151,8 @@ __global__ void moe_sort_kernel(int* __restrict__ choice, int n, int E, int tile
                                 int* __restrict__ offsets, int* __restrict__ tiles, int* __restrict__ pair_of_row,
                                 int* __restrict__ row_of_pair, int* __restrict__ group_of_tile, int max_tiles, int rows_cap,
                                 const float* __restrict__ logits, long long ld, const float* __restrict__ bias, int top,
-                                float* __restrict__ weight, int scoring, int groups, int kept) {
+                                float* __restrict__ weight, int scoring, int groups, int kept,
+                                const float* __restrict__ correction, float wscale) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ int sort_smem[];
@@ -151,7 +160,8 @@ __global__ void moe_sort_kernel(int* __restrict__ choice, int n, int E, int tile
   int* start = count + E;            // [E + 1]
   if (logits) {
     float* z = reinterpret_cast<float*>(start + E + 1) + (size_t)(threadIdx.x >> 5) * E;
-    for (int t = threadIdx.x >> 5; t < n / top; t += blockDim.x >> 5) route_token(logits, ld, bias, t, E, top, z, choice, weight, scoring, groups, kept);
+    for (int t = threadIdx.x >> 5; t < n / top; t += blockDim.x >> 5)
+      route_token(logits, ld, bias, t, E, top, z, choice, weight, scoring, groups, kept, correction, wscale);
     __syncthreads();                 // the choices of all tokens are written (and visible to the block)
   }
   for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = 0;
@@ -495,15 +505,17 @@ static int routing_ok(const char* what, int E, int top, int scoring, int groups,
 }
 
 extern "C" int srlm_moe_route(const float* logits, long long ld, const float* bias, int T, int E, int top, int* choice,
-                              float* weight, int scoring, int groups, int kept, cudaStream_t stream) {
+                              float* weight, int scoring, int groups, int kept, const float* correction, float weight_scale,
+                              cudaStream_t stream) {
   if (T <= 0) return ST_OK;
   if (E <= 0 || top <= 0 || top > E || ld < E || E > 8192)
     return refuse(ST_BAD_SIZE, "moe_route: experts=%d top=%d ld=%lld (at most 8192 experts)", E, top, ld);
   if (int r = routing_ok("moe_route", E, top, scoring, groups, kept)) return r;
+  if (correction && scoring != 1) return refuse(ST_BAD_SIZE, "moe_route: corrected choices come with scoring 1");
   int warps = 4;
   while (warps > 1 && (size_t)warps * E * sizeof(float) > 40 * 1024) warps >>= 1;
   launch_pdl(moe_route_kernel, dim3((T + warps - 1) / warps), dim3(warps * 32), (size_t)warps * E * sizeof(float), stream,
-             logits, ld, bias, T, E, top, choice, weight, scoring, groups, kept);
+             logits, ld, bias, T, E, top, choice, weight, scoring, groups, kept, correction, weight_scale);
   return launched();
 }
 
@@ -518,11 +530,12 @@ extern "C" int srlm_moe_sort_routes(int tokens, int E) { return tokens <= 512 &&
 extern "C" int srlm_moe_sort(int* choice, int n, int E, int* offsets, int* tiles, int* pair_of_row,
                              int* row_of_pair, int tile_rows, int* group_of_tile, int max_tiles, int rows_cap,
                              const float* logits, long long ld, const float* bias, int top, float* weight, int scoring,
-                             int groups, int kept, cudaStream_t stream) {
+                             int groups, int kept, const float* correction, float weight_scale, cudaStream_t stream) {
   if (n <= 0) return ST_OK;
   if (E <= 0 || E > 4096) return refuse(ST_BAD_SIZE, "moe_sort: experts=%d (at most 4096)", E);
   if (logits)
     if (int r = routing_ok("moe_sort", E, top, scoring, groups, kept)) return r;
+  if (correction && (!logits || scoring != 1)) return refuse(ST_BAD_SIZE, "moe_sort: corrected choices come with scoring 1");
   if (logits && (top <= 0 || top > E || n % top || ld < E || !weight || !srlm_moe_sort_routes(n / top, E)))
     return refuse(ST_BAD_SIZE, "moe_sort: routing %d pairs, top=%d of %d experts, ld=%lld", n, top, E, ld);
   const int align = tile_rows > 0;
@@ -533,7 +546,7 @@ extern "C" int srlm_moe_sort(int* choice, int n, int E, int* offsets, int* tiles
   const size_t smem = (size_t)(2 * E + 1) * sizeof(int) + (logits ? (size_t)32 * E * sizeof(float) : 0);
   launch_pdl(moe_sort_kernel, dim3(1), dim3(1024), smem, stream, choice, n, E,
              align ? tile_rows : kTile, align, offsets, tiles, pair_of_row, row_of_pair, group_of_tile, max_tiles, rows_cap,
-             logits, ld, bias, top, weight, scoring, groups, kept);
+             logits, ld, bias, top, weight, scoring, groups, kept, correction, weight_scale);
   return launched();
 }
 
@@ -557,7 +570,7 @@ static inline int tile_bound(int n, int E) {
 }
 
 // glu != 0: W [E, 2 N, K], C [n, N] = the experts' activation; else W [E, N, K], C [n, N] = the product, through the
-// exact gelu when act == 1.
+// exact gelu when act == 1, through the square of its positive part when act == 2.
 // pair_of_row null: row r of A is row r of C (the experts' second product); else A's row is the pair's token.
 extern "C" int srlm_moe_grouped_simt(const void* A, int a_dtype, long long lda, const int* pair_of_row, int pairs_per_token,
                                      const void* W, int w_dtype, void* C, int c_dtype, long long ldc, const int* offsets,

@@ -137,11 +137,12 @@ class KernelLibrary:
             raise RuntimeError(f"{what} failed with CUDA error {status}: {msg}")
 
     # ---- elementwise -----------------------------------------------------
-    def embed_gather(self, ids, table, out, bad_flag):
+    def embed_gather(self, ids, table, out, bad_flag, scale=1.0, add=False):
+        """out [T, H] float32 = the table's rows of the token ids, times scale; add: they are added to out."""
         T, H = out.shape
         self._check(self.lib.srlm_embed_gather(_ptr(ids), _ptr(table), dtype_code(table.dtype), _ptr(out),
                                                C.c_int(T), C.c_int(H), C.c_int(table.shape[0]),
-                                               _ptr(bad_flag), _stream()), "embed_gather")
+                                               _ptr(bad_flag), C.c_float(scale), C.c_int(int(add)), _stream()), "embed_gather")
 
     def add_rmsnorm(self, residual, delta, weight, eps, out, rows=None, unit_offset=False):
         R, H = out.shape
@@ -942,12 +943,14 @@ class KernelLibrary:
     ROUTER_SCORING = {"softmax_of_chosen": 0, "logistic": 1, "softmax_over_all": 2}
 
     def moe_route(self, logits, bias, top, choice, weight, column=0, experts=None, scoring="softmax_of_chosen",
-                  groups=(1, 1)):
+                  groups=(1, 1), correction=None, weight_scale=1.0):
         """logits float32 [T, E] (+ bias float32 [E]) -> choice int32 [T, top], the experts with the largest
         logits (ties: the lowest index), and weight float32 [T, top]: the softmax over the chosen logits, or
         (scoring "logistic") the logistic of each chosen logit, not renormalised, or (scoring "softmax_over_all") the
         softmax over all logits, renormalised over the chosen ones; then groups = (count, kept): the experts form
         ``count`` equal groups of neighbours and only experts of the ``kept`` groups with the largest scores are chosen.
+        correction (float32 [E], scoring "logistic"): the experts with the largest logistic plus correction are chosen, the
+        weights are the logistics without it.  weight_scale: a factor on every weight.
         column / experts: the logits are those columns of a wider tensor."""
         T = logits.shape[0]
         E = logits.shape[1] - column if experts is None else experts
@@ -957,14 +960,14 @@ class KernelLibrary:
         self._check(self.lib.srlm_moe_route(ptr, ld, _ptr(bias), C.c_int(T), C.c_int(E),
                                             C.c_int(top), _ptr(choice), _ptr(weight),
                                             C.c_int(self.ROUTER_SCORING[scoring]), C.c_int(groups[0]), C.c_int(groups[1]),
-                                            _stream()), "moe_route")
+                                            _ptr(correction), C.c_float(weight_scale), _stream()), "moe_route")
 
     def moe_sort_routes(self, tokens, experts) -> bool:
         """Whether moe_sort(..., route=...) routes a step of this many tokens itself."""
         return bool(self.lib.srlm_moe_sort_routes(C.c_int(tokens), C.c_int(experts)))
 
     def moe_sort(self, choice, experts, offsets, tiles, pair_of_row, row_of_pair, tile_rows=0, group_of_tile=None,
-                 route=None, scoring="softmax_of_chosen", groups=(1, 1)):
+                 route=None, scoring="softmax_of_chosen", groups=(1, 1), correction=None, weight_scale=1.0):
         """The (token, choice) pairs ordered by expert: offsets / tiles int32 [experts + 1] (first row and first
         tile of each expert), pair_of_row / row_of_pair int32 [pairs].  tile_rows > 0: every expert's rows start at
         a multiple of tile_rows; pair_of_row then covers all rows of group_of_tile's tiles (-1: a row without a
@@ -981,7 +984,7 @@ class KernelLibrary:
             _ptr(row_of_pair), C.c_int(tile_rows), _ptr(group_of_tile),
             C.c_int(group_of_tile.numel() if group_of_tile is not None else 0),
             C.c_int(pair_of_row.numel()), *routing, C.c_int(self.ROUTER_SCORING[scoring]), C.c_int(groups[0]),
-            C.c_int(groups[1]), _stream()), "moe_sort")
+            C.c_int(groups[1]), _ptr(correction), C.c_float(weight_scale), _stream()), "moe_sort")
 
     GROUPED_TILE = 128       # token rows of a tile of the grouped tensor-memory product (one SM a tile)
     GROUPED_PAIR_TILE = 256  # ... of its pair form (two SMs on 256 weight rows x 256 tokens)
@@ -1005,8 +1008,8 @@ class KernelLibrary:
     def gemm_tn_tcgen05_grouped(self, x, w, out, group_of_tile, glu=False, limit=0.0, alpha=0.0, tile_rows=128, act=None):
         """out[r] = x[r] . w[group of r's tile]^T on the persistent tensor-memory kernel: x [rows, K] bfloat16 in tiles
         of tile_rows rows (128, or 256: pairs of SMs), w [groups, N, K]; a tile whose group is negative is skipped.
-        glu: w's rows in blocks of 8 gate and 8 up rows, out [rows, N / 2] = the clamped GLU.  act "gelu" (without glu):
-        out = the exact gelu of the product."""
+        glu: w's rows in blocks of 8 gate and 8 up rows, out [rows, N / 2] = the clamped GLU.  act (without glu): out =
+        the exact gelu ("gelu") or the square of the positive part ("relu_squared") of the product."""
         rows, K = x.shape
         G, N, _ = w.shape
         if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or w.shape[2] != K or group_of_tile.numel() * tile_rows < rows:
@@ -1019,7 +1022,7 @@ class KernelLibrary:
             C.c_float(limit), C.c_float(alpha), C.c_int(self.PLAIN_ACTIVATIONS[act]), _ptr(err), _stream()),
             "gemm_tn_tcgen05_grouped")
 
-    PLAIN_ACTIVATIONS = {None: 0, "gelu": 1}
+    PLAIN_ACTIVATIONS = {None: 0, "gelu": 1, "relu_squared": 2}
 
     def moe_grouped(self, a, pair_of_row, pairs_per_token, w, out, offsets, tiles, glu=False, interleaved=False,
                     limit=0.0, alpha=0.0, pair_scale=None, act=None):
@@ -1028,8 +1031,8 @@ class KernelLibrary:
         the gate and up halves (interleaved: in blocks of 8 gate rows and 8 up rows, else all gate rows first);
         limit 0: the plain GLU, gate * logistic(gate) * up.  pair_scale (float32, one number a pair; with glu): the
         gate and up sums of a row are multiplied by its pair's number ahead of the activation, which for experts
-        without biases is the activation of the scaled input.  act "gelu" (without glu): out gets the exact gelu of
-        the product."""
+        without biases is the activation of the scaled input.  act "gelu" / "relu_squared" (without glu): out gets that
+        activation of the product."""
         E, rows, K = w.shape
         n, N = out.shape
         if a.shape[1] != K or rows != (2 * N if glu else N):
@@ -1220,6 +1223,63 @@ class KernelLibrary:
                                                     C.c_longlong(state.stride(0)), _ptr(ctx.cu_q), _ptr(ctx.slots),
                                                     _ptr(out), dtype_code(out.dtype), C.c_int(ctx.n_entries), C.c_int(Cn),
                                                     C.c_int(int(in_segments)), _stream()), "linear_recurrence")
+
+    # ---- attention whose heads mix their weights -----------------------------------------------------
+    def attention_wide_norm_append(self, proj, q_norm_w, k_norm_w, eps, q_out, k_cache, v_cache, kv_slot, nq, nkv, dk, dv,
+                                   write_kv=True):
+        """From a stacked q | k | v (| more) projection (float32 [T, >= nq dk + nkv (dk + dv)]): q and k RMS-normed over all
+        their heads at once with q_norm_w (float32 [nq dk]) and k_norm_w (eps None: as projected); q to q_out (float32 or
+        bfloat16), k and v to the pages."""
+        self._check(self.lib.srlm_attention_wide_norm_append(
+            _ptr(proj), dtype_code(proj.dtype), C.c_longlong(proj.stride(0)), C.c_float(eps or 0.0), _ptr(q_norm_w),
+            _ptr(k_norm_w), _ptr(q_out), dtype_code(q_out.dtype), _ptr(k_cache), _ptr(v_cache), dtype_code(k_cache.dtype),
+            _ptr(kv_slot), C.c_int(int(write_kv)), C.c_int(proj.shape[0]), C.c_int(nq), C.c_int(nkv), C.c_int(dk), C.c_int(dv),
+            C.c_int(k_cache.shape[2]), _stream()), "attention_wide_norm_append")
+
+    def mixed_head_attention(self, ctx, q, k_cache, v_cache, out, block_table, nq, nkv, dk, dv, scale, window=0, keep_first=0,
+                             bias=None, mix=None, gate=None):
+        """Causal attention of the batch of ``ctx`` whose heads exchange their weights behind the softmax: head h applies
+        sum_g mix[h, g] p_g to the values of its own KV head.  q [T, nq dk]; pages as paged_attention_general's; out
+        [T, nq dv] in the cache's dtype; bias float32 [nq, n] or None: added to the scaled score of a key at distance
+        n' = min(i - j, n - 1); window > 0: a query sees itself, the window - 1 keys before it and the first keep_first
+        keys; mix float32 [nq, nq] or None; gate (float32 tensor [T, >= column + nq dv], column) or None: every element is
+        multiplied by the logistic of its own column."""
+        T = q.shape[0]
+        gate_args = (C.c_void_p(0), C.c_longlong(0)) if gate is None else self._columns(gate[0], gate[1], nq * dv)
+        n_dist = bias.shape[1] if bias is not None else 0
+        if q.dtype != torch.float32:
+            raise ShapeError("mixed_head_attention: float32 queries")
+        self._check(self.lib.srlm_mixed_head_attention(
+            _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), dtype_code(k_cache.dtype), dtype_code(out.dtype),
+            _ptr(block_table), C.c_int(block_table.stride(0)), _ptr(ctx.entry_of_token), _ptr(ctx.positions), C.c_int(T),
+            C.c_int(nq), C.c_int(nkv), C.c_int(dk), C.c_int(dv), C.c_int(k_cache.shape[2]), C.c_float(scale),
+            C.c_int(window or 0), C.c_int(keep_first), _ptr(bias), C.c_int(n_dist), _ptr(mix), *gate_args, _stream()),
+            "mixed_head_attention")
+
+    # ---- retention --------------------------------------------------------------------------------------
+    def retention(self, ctx, proj, rotation, decay, eps, state, out, H, d, dv):
+        """out [T, H dv] = per head o / sqrt(mean(o^2) + eps) * silu(gate), o the read-out of a state that fades by decay[h]
+        a token, from the stacked projection q | k | v | gate (float32), whose leading 2 * pairs elements of every q and k
+        head are turned by ``rotation``; state float32 [slots, >= H d dv], renewed."""
+        pairs = rotation.pairs if rotation is not None else 0
+        if pairs and rotation.interleaved:
+            raise ShapeError("retention: half-split pairs only")
+        T = proj.shape[0]
+        o = None
+        if not self.lib.srlm_retention_walk_finishes(C.c_int(dv)):
+            o = ctx.workspace.get("retention.o", T, H * dv, torch.float32)
+        self._check(self.lib.srlm_retention_walk(
+            _ptr(proj), C.c_longlong(proj.stride(0)), _ptr(rotation.cos if pairs else None),
+            _ptr(rotation.sin if pairs else None), C.c_int(pairs), _ptr(decay), C.c_float(eps), _ptr(state),
+            C.c_longlong(state.stride(0)), _ptr(ctx.cu_q), _ptr(ctx.slots), _ptr(o), _ptr(out), dtype_code(out.dtype),
+            C.c_int(ctx.n_entries), C.c_int(H), C.c_int(d), C.c_int(dv), _stream()), "retention_walk")
+        if o is not None:
+            self._retention_output(o, eps, proj, 2 * H * d + H * dv, out, H, dv)
+
+    def _retention_output(self, o, eps, proj, gate_off, out, H, dv):
+        self._check(self.lib.srlm_retention_output(
+            _ptr(o), C.c_float(eps), _ptr(proj), C.c_longlong(proj.stride(0)), C.c_int(gate_off), _ptr(out),
+            dtype_code(out.dtype), C.c_int(o.shape[0]), C.c_int(H), C.c_int(dv), _stream()), "retention_output")
 
     # ---- attention over a cached latent ----------------------------------------------------
     def latent_append(self, proj, c_off, norm_w, eps, rotation, cache, kv_slot, rank, rot, q_norm=None):

@@ -65,6 +65,7 @@ class CacheNeed:
     state_dtype: torch.dtype = torch.float32
     v_head_dim: Optional[int] = None          # None: values as wide as keys; 0: no value pool (the values are
                                               # read from the keys); else the values' own size
+    keep_first: int = 0                       # with a window: the first tokens of a sequence, which stay visible behind it
 
 
 @dataclass

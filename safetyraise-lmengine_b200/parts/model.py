@@ -71,7 +71,7 @@ def cache_groups_of(spec: ModelSpec) -> List[CacheGroupSpec]:
         groups.append(CacheGroupSpec(name=f"g{i}:{need.kind}", kind=need.kind, entries=tuple(entries),
                                      kv_heads=need.kv_heads, head_dim=need.head_dim, window=need.window,
                                      state_shape=need.state_shape, state_dtype=need.state_dtype,
-                                     v_head_dim=need.v_head_dim))
+                                     v_head_dim=need.v_head_dim, keep_first=need.keep_first))
     return groups
 
 
@@ -95,6 +95,8 @@ class DecoderModel:
                                                                       tensors, mctx)
         # tied: the head IS the embedding table (same storage), src/model/native.rs:171-179
         self.head = Linear(self.embed if spec.tie_word_embeddings else tensors[spec.head_name], "lm_head")
+        self.keeps_embedding = any(s.add_embedding for s in spec.run_order) and \
+            (self.embed_norm is not None or self.embed_position is not None)
         for step in spec.run_order:
             if not 0 <= step.layer < len(self.blocks):
                 raise ConfigError(f"run order names layer {step.layer}, the model has {len(self.blocks)}")
@@ -114,16 +116,27 @@ class DecoderModel:
         if self.embed_norm is not None:
             # the stream starts from the normed rows of the table: gathered beside it, normed into it (float32)
             rows = ctx.workspace.get("embed.rows", ctx.T, H, torch.float32)
-            ops.embed_gather(ctx.token_ids, self.embed, rows, status[FAULT_TOKEN:FAULT_TOKEN + 1])
+            ops.embed_gather(ctx.token_ids, self.embed, rows, status[FAULT_TOKEN:FAULT_TOKEN + 1], scale=self.spec.embed_scale)
             self.embed_norm.apply(rows, None, residual)
         else:
-            ops.embed_gather(ctx.token_ids, self.embed, residual, status[FAULT_TOKEN:FAULT_TOKEN + 1])
+            ops.embed_gather(ctx.token_ids, self.embed, residual, status[FAULT_TOKEN:FAULT_TOKEN + 1], scale=self.spec.embed_scale)
         if self.embed_position is not None:
             self.embed_position.add_to_embedding(ctx, residual)
+        kept = None
+        if self.keeps_embedding:         # more than the table's rows: a later step needs a copy of what the embedding left
+            kept = ctx.workspace.get("embed.kept", ctx.T, H, torch.float32)
+            ops.cast(residual, kept)
         pending = None
         order = self.spec.run_order
         for i, step in enumerate(order):
-            nxt = self.blocks[order[i + 1].layer] if i + 1 < len(order) else None
+            if step.add_embedding:
+                if kept is not None:
+                    ops.residual_add(residual, kept)
+                else:                    # the rows themselves, read from the table again
+                    ops.embed_gather(ctx.token_ids, self.embed, residual, status[FAULT_TOKEN:FAULT_TOKEN + 1],
+                                     scale=self.spec.embed_scale, add=True)
+            # a block ahead of an addition to the stream prepares no input: what it leaves is pending or in the stream
+            nxt = self.blocks[order[i + 1].layer] if i + 1 < len(order) and not order[i + 1].add_embedding else None
             pending = self.blocks[step.layer].forward(ctx, residual, pending, step, nxt)
         # NaN and infinity stay in a residual stream that is only ever added to, and every key or value
         # a step writes is read by its own token: one look at the end covers every block

@@ -11,7 +11,9 @@ experts have no biases, so W (w h) = w (W h), and the first grouped product mult
 the pair's weight ahead of the activation (steps of many tokens, whose rows are gathered into tiles, scale the
 gathered rows).
 
-``gated`` False: an expert (and the shared one) is W_down act(W_up h) with ``activation`` "gelu" (the exact one).
+``gated`` False: an expert (and the shared one) is W_down act(W_up h) with ``activation`` "gelu" (the exact one), or
+(without a shared one) "relu_squared", max(z, 0)^2.  ``correction``: with logistic scores s, the experts with the largest
+s + correction are chosen and weighted by s; ``weight_scale`` is a factor on every weight.
 ``scoring`` "softmax_over_all": the scores are the softmax over all experts' logits, the choice may be limited to the
 best ``groups_kept`` of ``groups`` equal groups of neighbouring experts (a group counts as its largest score), and the
 weights are the chosen scores over their sum.
@@ -37,16 +39,21 @@ from .linear import Linear
 @register_feed_forward("routed_experts")
 class RoutedExperts(Part):
     def __init__(self, spec: RoutedExpertsSpec, prefix: str, tensors: dict, mctx):
-        if spec.activation not in (("clamped_glu", "silu") if spec.gated else ("gelu",)):
+        if spec.activation not in (("clamped_glu", "silu") if spec.gated else ("gelu", "relu_squared")):
             raise Unsupported(f"routed experts with activation {spec.activation!r} are not implemented")
         if not spec.gated and spec.weight_on_input:
             raise Unsupported("a weight on an expert's input comes with gated experts only")
         if spec.scoring not in ops.ROUTER_SCORING:
             raise Unsupported(f"routed experts with router scoring {spec.scoring!r} are not implemented")
+        if spec.correction and spec.scoring != "logistic":
+            raise Unsupported("a correction of the experts' choice comes with logistic scores only")
+        if spec.activation == "relu_squared" and spec.shared_size:
+            raise Unsupported("an expert that every token runs comes without the squared activation")
         if spec.activation == "silu" and spec.shared_size:
             raise Unsupported("an expert that every token runs comes with the clamped activation only")
         self.spec = spec
-        self.groups = (spec.groups, spec.groups_kept)
+        self.routing = dict(scoring=spec.scoring, groups=(spec.groups, spec.groups_kept), weight_scale=spec.weight_scale,
+                            correction=tensors[prefix + spec.expert_names.correction] if spec.correction else None)
         if not spec.gated:
             self._init_plain(spec, prefix, tensors, mctx)
             return
@@ -112,6 +119,8 @@ class RoutedExperts(Part):
         decls.append(TensorDecl(p + nm.router, (s.experts, H), MATRIX))
         if s.router_bias:
             decls.append(TensorDecl(p + nm.router_bias, (s.experts,), VECTOR))
+        if s.correction:
+            decls.append(TensorDecl(p + nm.correction, (s.experts,), VECTOR))
         if s.shared_size:
             sp = p + nm.shared
             if s.gated:
@@ -137,7 +146,7 @@ class RoutedExperts(Part):
         if (self.in_tiles and ops.grouped_products_in_tensor_memory and pairs >= 64 * s.experts
                 and s.intermediate_size % 8 == 0):
             ops.moe_route(first, self.router_bias, s.top, choice, weight, column=self.router_column, experts=s.experts,
-                          scoring=s.scoring, groups=self.groups)
+                          **self.routing)
             return self._forward_tiles(ctx, x, first, choice, weight, add)
         heads = ws.get("moe.heads", 2, s.experts + 1, torch.int32, reserve=2)
         order = ws.get("moe.order", 2 * T, s.top, torch.int32, reserve=2 * ws.max_tokens)
@@ -145,11 +154,10 @@ class RoutedExperts(Part):
         pair_of_row, row_of_pair = order[:T].view(-1), order[T:].view(-1)
         if ops.moe_sort_routes(T, s.experts):          # a small step: the block that orders the pairs routes them too
             ops.moe_sort(choice, s.experts, offsets, tiles, pair_of_row, row_of_pair,
-                         route=(first, self.router_column, self.router_bias, weight), scoring=s.scoring,
-                         groups=self.groups)
+                         route=(first, self.router_column, self.router_bias, weight), **self.routing)
         else:
             ops.moe_route(first, self.router_bias, s.top, choice, weight, column=self.router_column, experts=s.experts,
-                          scoring=s.scoring, groups=self.groups)
+                          **self.routing)
             ops.moe_sort(choice, s.experts, offsets, tiles, pair_of_row, row_of_pair)
         y = ws.get("moe.y", pairs, s.intermediate_size, ctx.dtype, reserve=ws.max_tokens * s.top)
         if s.gated:

@@ -13,7 +13,7 @@ widened to float32 when the engine runs its float32 path); a tensor stored in
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Dict, Iterable, Sequence, Tuple
+from typing import Dict, Iterable, Optional, Sequence, Tuple
 
 import torch
 
@@ -25,8 +25,17 @@ MATRIX, VECTOR, TABLE, INT_TABLE = "matrix", "vector", "table", "int_table"
 @dataclass(frozen=True)
 class TensorDecl:
     name: str
-    shape: Tuple[int, ...]
+    shape: Tuple[Optional[int], ...]      # None: a free dimension, whose size is the stored tensor's
     role: str = MATRIX        # MATRIX | VECTOR (norm scale) | TABLE (embedding rows) | INT_TABLE
+    free_size: int = 32       # what a free dimension is made as where weights are generated and not read
+
+    @property
+    def made_shape(self) -> Tuple[int, ...]:
+        return tuple(self.free_size if s is None else s for s in self.shape)
+
+
+def _fits(shape, declared) -> bool:
+    return len(shape) == len(declared) and all(d is None and n > 0 or n == d for n, d in zip(shape, declared))
 
 
 def check_against(decls: Sequence[TensorDecl], available: Dict[str, Tuple[int, ...]]) -> None:
@@ -35,7 +44,7 @@ def check_against(decls: Sequence[TensorDecl], available: Dict[str, Tuple[int, .
     missing = [n for n in wanted if n not in available]
     unexpected = [n for n in available if n not in wanted]
     misshaped = [(n, tuple(available[n]), wanted[n].shape) for n in wanted
-                 if n in available and tuple(available[n]) != tuple(wanted[n].shape)]
+                 if n in available and not _fits(tuple(available[n]), tuple(wanted[n].shape))]
     if not (missing or unexpected or misshaped):
         return
     lines = ["weights do not match the configuration:"]
@@ -45,7 +54,8 @@ def check_against(decls: Sequence[TensorDecl], available: Dict[str, Tuple[int, .
         lines.append(f"  unexpected tensors ({len(unexpected)}): " + ", ".join(sorted(unexpected)))
     if misshaped:
         lines.append(f"  wrong shapes ({len(misshaped)}): " + "; ".join(
-            f"{n} is {list(got)}, expected {list(exp)}" for n, got, exp in sorted(misshaped)))
+            f"{n} is {list(got)}, expected {['any' if d is None else d for d in exp]}"
+            for n, got, exp in sorted(misshaped, key=lambda m: m[0])))
     raise WeightError("\n".join(lines))
 
 

@@ -33,10 +33,10 @@ def random_tensor(decl: TensorDecl, seed: int, device="cpu", matrix_dtype=torch.
     gen = torch.Generator(device=device)
     gen.manual_seed(_seed_for(seed, decl.name))
     if decl.role == VECTOR:
-        return 1.0 + 0.1 * torch.randn(decl.shape, generator=gen, device=device, dtype=torch.float32)
+        return 1.0 + 0.1 * torch.randn(decl.made_shape, generator=gen, device=device, dtype=torch.float32)
     if decl.role == INT_TABLE:
-        return torch.randint(0, 2 ** 31 - 1, decl.shape, generator=gen, device=device, dtype=torch.int32)
-    t = torch.empty(decl.shape, device=device, dtype=matrix_dtype)
+        return torch.randint(0, 2 ** 31 - 1, decl.made_shape, generator=gen, device=device, dtype=torch.int32)
+    t = torch.empty(decl.made_shape, device=device, dtype=matrix_dtype)
     # generated in slabs so that a large table needs no float32 copy of itself
     flat = t.view(-1)
     step = 1 << 26
@@ -60,10 +60,10 @@ class RandomWeights:
     def meta(self, name):
         d = self._decls[name]
         n = 1
-        for s in d.shape:
+        for s in d.made_shape:
             n *= s
         dt = torch.float32 if d.role == VECTOR else torch.int32 if d.role == INT_TABLE else self.matrix_dtype
-        return dt, tuple(d.shape), n * dt.itemsize
+        return dt, d.made_shape, n * dt.itemsize
 
     def get(self, name):
         return random_tensor(self._decls[name], self.seed, self.device, self.matrix_dtype)
