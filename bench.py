@@ -636,6 +636,31 @@ def dovorax_config(size: dict, kinds) -> dict:
                        for i, k in enumerate(kinds)]}
 
 
+LOKIZEN_WINDOW, LOKIZEN_KEPT = 1024, 16
+
+
+def lokizen_config(size: dict, kinds) -> dict:
+    """A Lokizen configuration whose layers have the sizes of a Qwen3 layer of the same width: attention with heads of 128
+    for keys and values, a window of 1,024 tokens that keeps the first 16 and biases of distances up to 2,048; a
+    retention of as many heads of 128 x 128, all of each head rotated; 16 ungated experts of three quarters of a width
+    of which a token runs 4: three widths of feed-forward rows a token.  'loop' in the list: the layer behind it runs
+    twice."""
+    W, H, G = size["width"], size["heads"], size["kv_heads"]
+    mixers = {
+        "attention": {"heads": H, "kv_heads": G, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "bias_max": 2048,
+                      "mask": {"size": LOKIZEN_WINDOW, "keep_first": LOKIZEN_KEPT}},
+        "retention": {"heads": H, "dim": 128, "vdim": 128, "rot": {"base": 10000.0, "dims": 128},
+                      "decay": [1.0 - 2.0 ** (-5.0 - 7.0 * h / H) for h in range(H)]},
+    }
+    mlp = {"kind": "moe", "expert": {"ff": 3 * W // 4}, "router": {"experts": 16, "top": 4, "scale": 1.5}}
+    cfg = {"architecture": "Lokizen", "width": W, "vocab": DESIGN_VOCAB, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+           "layers": [{"type": k, "mixer": mixers[k], "mlp": mlp} for k in kinds if k != "loop"]}
+    if "loop" in kinds:
+        at = kinds.index("loop")
+        cfg["loop"] = {"start": at, "stop": at + 1, "times": 2}
+    return cfg
+
+
 def qwen3_config(size: dict) -> dict:
     return dict(BASE, num_hidden_layers=DESIGN_LAYERS, hidden_size=size["width"], num_attention_heads=size["heads"],
                 num_key_value_heads=size["kv_heads"], intermediate_size=3 * size["width"], vocab_size=DESIGN_VOCAB)
@@ -667,14 +692,23 @@ def run_design(args) -> dict:
                   "dovorax recurrence": ["rglru"] * DESIGN_LAYERS,
                   "dovorax mixed": ["latent_attention", "parallel", "rglru", "latent_attention"]}
         make = lambda size, kinds: (tonanex_config if kinds[0] == "moe" else nekedra_config if kinds[0] == "delta" else None)(size, kinds)
+    if args.design == "lokizen":
+        stacks = {"qwen3": None, "tonanex experts": ["moe"] * DESIGN_LAYERS, "nekedra delta": ["delta"] * DESIGN_LAYERS,
+                  "lokizen attention": ["attention"] * DESIGN_LAYERS, "lokizen retention": ["retention"] * DESIGN_LAYERS,
+                  "lokizen looped": ["retention", "loop", "attention", "retention"]}
+        make = tonanex_config
     out = {"metric": args.design + "_beside_qwen3", "layers": DESIGN_LAYERS, "prefill_tokens": PREFILL_TOKENS,
            "decode_batch": batch, "decode_context": context, "dtype": "bf16", "data": "synthetic", "sizes": {}}
     sizes = [args.design_size] if args.design_size else sorted(DESIGN_SIZES)
     for name in sizes:
         size, rows = DESIGN_SIZES[name], {}
         for label, kinds in stacks.items():
+            if args.design_stack and not label.startswith(args.design_stack):
+                continue
             if label.startswith("dovorax"):
                 cfg = dovorax_config(size, kinds)
+            elif label.startswith("lokizen"):
+                cfg = lokizen_config(size, kinds)
             elif label.startswith("nekedra"):
                 cfg = nekedra_config(size, kinds)
             else:
@@ -717,9 +751,10 @@ def main() -> int:
     ap.add_argument("--only-prefill", action="store_true", help="run just the 2,048-token prefill (for profilers)")
     ap.add_argument("--streaming-kernel", action="store_true",
                     help="steps of up to 8 tokens on the weight-streaming mma.sync kernel instead of the tensor-core one")
-    ap.add_argument("--design", default=None, choices=["nekedra", "tonanex", "pabalorn", "dovorax"],
-                    help="instead of the default workload: prefill and decode of Nekedra, Tonanex, Pabalorn or Dovorax stacks "
-                         "beside the Qwen3 decoder at equal layer sizes")
+    ap.add_argument("--design", default=None, choices=["nekedra", "tonanex", "pabalorn", "dovorax", "lokizen"],
+                    help="instead of the default workload: prefill and decode of that design's stacks beside the Qwen3 decoder "
+                         "at equal layer sizes")
+    ap.add_argument("--design-stack", default=None, help="only the stacks of --design whose name begins so")
     ap.add_argument("--design-size", default=None, choices=sorted(DESIGN_SIZES), help="one width of --design")
     ap.add_argument("--min-seconds", type=float, default=MIN_TIMED_SECONDS,
                     help="repeat the block of --steps steps until this much is timed (0: one block, for profilers)")

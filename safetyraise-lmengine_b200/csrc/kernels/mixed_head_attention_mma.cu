@@ -1,0 +1,779 @@
+// The mixed-head attention of mixed_head_attention.cu on bfloat16 tensor cores (mma.sync m16n8k16, float32 sums).
+//
+// Prompts, portions and mixed steps take two kernels.  Scores are kept in units of log2, so a softmax is one 2^x:
+//   mixed_head_lse      every row's logarithm of the softmax's sum, L = log2 sum_j 2^(s_j), a block for 64 rows (tokens x
+//                       query heads) of one KV head: the running maximum and sum of an ordinary attention, without values;
+//   mixed_head_attention_mma   a block for 16 / HT tokens and ALL heads.  Per tile of 32 keys: every warp forms the scores
+//                       of its 16 rows (HT heads x 16 / HT tokens) and p = 2^(s - L), finished weights; the block mixes
+//                       them; every warp multiplies its rows of the mixture with its KV head's values.
+// The mixture is a product of mix [H, H] with the weights of a tile [H, tokens x keys], on tensor cores with the weights as
+// pairs of bfloat16 (p = hi + lo, 16 significant bits each way of the exact sum), float32 sums; mix itself is rounded to such
+// a pair when its values are no bfloat16 numbers.  Keys and values have one buffer each: the next tile's keys are fetched
+// while the block mixes and multiplies values, this tile's values while it forms scores.
+//
+// Decode steps (one token an entry) take one kernel: a thread-block cluster for an entry, a slice of its visible keys for
+// each block.  A block forms the scores of all heads over its slice and keeps them in shared memory; the blocks exchange
+// maxima and sums through distributed shared memory; each turns its scores into finished weights, mixes them, multiplies
+// its slice's values; and the blocks add their sums, a share of the columns each, as they gate and write them.
+#include <math_constants.h>
+
+#include "common.cuh"
+#include "mixed_head_attention.cuh"
+#include "mma_sync.cuh"
+
+namespace srlm {
+
+constexpr float kLog2e = 1.4426950408889634f;
+constexpr int kMhKeys = 32;                   // keys of a tile
+constexpr int kMhPad = 8;
+constexpr int kMhRow = kMhKeys + kMhPad;      // a token's weights of a tile in shared memory
+
+// The tiles of `width` keys that some query at min_pos .. max_pos sees: those of the kept tokens, then those from the
+// window's first key on.
+struct MixTiles {
+  int kept, base, count;
+  __device__ __forceinline__ MixTiles(const MixMask& mask, int min_pos, int max_pos, int width) {
+    base = mask.first_key(min_pos) / width;
+    kept = mask.window > 0 ? min((mask.keep + width - 1) / width, base) : 0;
+    count = kept + max_pos / width - base + 1;
+  }
+  __device__ __forceinline__ int key(int n, int width) const { return (n < kept ? n : base + n - kept) * width; }
+};
+
+// ---- the softmax's sums -------------------------------------------------------------------------------------------
+constexpr int kLseRows = 64, kLseKeys = 64;
+
+__global__ void __launch_bounds__(128)
+mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache, float* __restrict__ lse,
+                      const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_q,
+                      const int* __restrict__ kv_lens, int nq, int nkv, int dk, int page_size, float scale2, MixMask mask,
+                      DistanceBias bias, int span) {
+  pdl_wait();
+  pdl_trigger();
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  const int e = blockIdx.z, kvh = blockIdx.y, G = nq / nkv;
+  const int t0 = cu_q[e], q_len = cu_q[e + 1] - t0, start = kv_lens[e] - q_len, rows = q_len * G;
+  const int r0 = (gridDim.x - 1 - blockIdx.x) * kLseRows;      // the last rows see the most keys: they start first
+  if (r0 >= rows) return;
+  const int ks = dk + kMhPad;
+  bf16* q_s = reinterpret_cast<bf16*>(smem_raw);               // [64][dk + 8]
+  bf16* k_s = q_s + kLseRows * ks;                             // [2][64][dk + 8]
+  float* bias_s = reinterpret_cast<float*>(k_s + 2 * kLseKeys * ks);    // [2][G][span]
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int* table = block_table + (size_t)e * table_stride;
+  const int kvec = dk / 8;
+  for (int idx = tid; idx < kLseRows * kvec; idx += blockDim.x) {
+    const int r = idx / kvec, c = idx - r * kvec, row = r0 + r;
+    const bool there = row < rows;
+    const bf16* src = there ? q + ((size_t)(t0 + row / G) * nq + kvh * G + row % G) * dk + c * 8 : q;
+    cp_async_16(q_s + r * ks + c * 8, src, there);
+  }
+  float m[2], l[2];
+  int pos[2], head[2];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int row = r0 + warp * 16 + (lane >> 2) + 8 * i;
+    pos[i] = row < rows ? start + row / G : -1;
+    head[i] = row < rows ? row % G : 0;
+    m[i] = -CUDART_INF_F;
+    l[i] = 0.f;
+  }
+  const int last_row = min(rows, r0 + kLseRows) - 1;
+  const int max_pos = start + last_row / G, min_pos = start + r0 / G;
+  const int first_seen = mask.first_key(min_pos);
+  const MixTiles tiles(mask, min_pos, max_pos, kLseKeys);
+  auto fetch = [&](int jb, int buf) {
+    for (int idx = tid; idx < kLseKeys * kvec; idx += blockDim.x) {
+      const int jj = idx / kvec, c = idx - jj * kvec, j = jb + jj;
+      const bool there = j <= max_pos && (j >= first_seen || j < mask.keep);
+      const size_t row = there ? ((size_t)table[j / page_size] * nkv + kvh) * page_size + (j % page_size) : 0;
+      cp_async_16(k_s + (buf * kLseKeys + jj) * ks + c * 8, k_cache + row * dk + c * 8, there);
+    }
+    cp_async_commit();
+    if (bias.table) {
+      // bias_s[h][x] belongs to distance min_pos - (jb + 63) + x
+      const int d0 = min_pos - jb - (kLseKeys - 1);
+      for (int idx = tid; idx < G * span; idx += blockDim.x) {
+        const int h = idx / span, d = d0 + idx - h * span;
+        bias_s[(size_t)buf * G * span + idx] = bias.at(kvh * G + h, max(d, 0)) * kLog2e;
+      }
+    }
+  };
+  fetch(tiles.key(0, kLseKeys), 0);
+  for (int n = 0, buf = 0; n < tiles.count; ++n, buf ^= 1) {
+    const int jb = tiles.key(n, kLseKeys);
+    if (n + 1 < tiles.count) {
+      fetch(tiles.key(n + 1, kLseKeys), buf ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    float s[8][4];
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) s[i][c] = 0.f;
+    const bf16* qa = q_s + (warp * 16 + (lane & 15)) * ks + (lane >> 4) * 8;
+    const bf16* kb = k_s + (buf * kLseKeys + (lane & 7) + (lane >> 4) * 8) * ks + ((lane >> 3) & 1) * 8;
+    for (int k0 = 0; k0 < dk; k0 += 16) {
+      uint32_t a[4];
+      ldmatrix_x4(a, qa + k0);
+#pragma unroll
+      for (int n2 = 0; n2 < 4; ++n2) {
+        uint32_t b[4];
+        ldmatrix_x4(b, kb + n2 * 16 * ks + k0);
+        mma_bf16(s[2 * n2], a, b[0], b[1]);
+        mma_bf16(s[2 * n2 + 1], a, b[2], b[3]);
+      }
+    }
+    // every key of the tile visible to every row of the block: no masking
+    const bool whole = jb + kLseKeys - 1 <= min_pos && (mask.window <= 0 || jb > max_pos - mask.window) && r0 + kLseRows <= rows;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const float* bs = bias_s + (size_t)buf * G * span + head[i] * span + (pos[i] - min_pos) + (kLseKeys - 1);
+      float mx = -CUDART_INF_F;
+#pragma unroll
+      for (int x = 0; x < 8; ++x)
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+          const int jj = x * 8 + (lane & 3) * 2 + c;
+          float v = -CUDART_INF_F;
+          if (whole || mask.visible(pos[i], jb + jj)) v = fmaf(s[x][2 * i + c], scale2, bias.table ? bs[-jj] : 0.f);
+          s[x][2 * i + c] = v;
+          mx = fmaxf(mx, v);
+        }
+      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+      const float m_new = fmaxf(m[i], mx);
+      if (m_new != -CUDART_INF_F) {
+        float sum = 0.f;
+#pragma unroll
+        for (int x = 0; x < 8; ++x) sum += exp2f(s[x][2 * i] - m_new) + exp2f(s[x][2 * i + 1] - m_new);
+        l[i] = l[i] * exp2f(m[i] - m_new) + sum;               // the lane's own share of the row's sum
+        m[i] = m_new;
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    float sum = l[i];
+    sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+    sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+    const int row = r0 + warp * 16 + (lane >> 2) + 8 * i;
+    if (row < rows && (lane & 3) == 0) lse[(size_t)(t0 + row / G) * nq + kvh * G + row % G] = m[i] + log2f(sum);
+  }
+}
+
+// ---- weights, mixture, values ----------------------------------------------------------------------------------------
+// KS: 16-element steps of a key (at most), NT: 8-column tiles of the block's slab of values (at most), HT: 16-head tiles of
+// the mixture and heads of a warp's 16 rows.
+template <int KS, int NT, int HT>
+__global__ void __launch_bounds__(512)
+mixed_head_attention_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache,
+                                const bf16* __restrict__ v_cache, const float* __restrict__ lse, bf16* __restrict__ out,
+                                const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_q,
+                                const int* __restrict__ kv_lens, int nq, int nkv, int dk, int dv, int slab, int page_size,
+                                float scale2, MixMask mask, DistanceBias bias, const float* __restrict__ mix, int mix_low,
+                                ElementGate gate, int nsplit, float* __restrict__ part) {
+  pdl_wait();
+  pdl_trigger();
+  constexpr int R = 16 / HT;                                   // tokens of the block
+  constexpr int HP = 16 * HT;                                  // heads, padded
+  constexpr int RS = R * kMhRow + kMhPad;                      // a head's weights of a tile
+  constexpr int BL = R + kMhKeys;                              // distances of a tile
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  const int e = blockIdx.z, slabs = (dv + slab - 1) / slab, G = nq / nkv;
+  const int c0 = (blockIdx.y % slabs) * slab, split = blockIdx.y / slabs;
+  const int t0 = cu_q[e], q_len = cu_q[e + 1] - t0, start = kv_lens[e] - q_len;
+  const int i0 = (gridDim.x - 1 - blockIdx.x) * R;
+  if (i0 >= q_len) return;
+  const int ks = dk + kMhPad, width = min(slab, dv - c0), vs = slab + kMhPad;
+  bf16* k_s = reinterpret_cast<bf16*>(smem_raw);               // [nkv][32][dk + 8]
+  bf16* v_s = k_s + nkv * kMhKeys * ks;                        // [nkv][32][slab + 8]
+  bf16* p_hi = v_s + nkv * kMhKeys * vs;                       // [HP][RS]: weights, then their mixture
+  bf16* p_lo = p_hi + HP * RS;
+  bf16* mix_s = p_lo + HP * RS;                                // [2][HP][HP + 8]
+  float* bias_s = reinterpret_cast<float*>(mix_s + 2 * HP * (HP + kMhPad));   // [nq][BL]
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, warps = blockDim.x >> 5;
+  const int* table = block_table + (size_t)e * table_stride;
+  const int min_pos = start + i0, max_pos = start + min(q_len, i0 + R) - 1;
+  const int first_seen = mask.first_key(min_pos);
+  const MixTiles tiles(mask, min_pos, max_pos, kMhKeys);
+  const int per = (tiles.count + nsplit - 1) / nsplit;
+  const int n_first = split * per, n_last = min(tiles.count, n_first + per);
+  const int kvec = dk / 8, vvec = width / 8;
+
+  auto fetch_k = [&](int jb) {
+    for (int idx = tid; idx < nkv * kMhKeys * kvec; idx += blockDim.x) {
+      const int row = idx / kvec, c = idx - row * kvec, h = row / kMhKeys, j = jb + row % kMhKeys;
+      const bool there = j <= max_pos && (j >= first_seen || j < mask.keep);
+      const size_t at = there ? ((size_t)table[j / page_size] * nkv + h) * page_size + (j % page_size) : 0;
+      cp_async_16(k_s + row * ks + c * 8, k_cache + at * dk + c * 8, there);
+    }
+    cp_async_commit();
+  };
+  auto fetch_v = [&](int jb) {
+    for (int idx = tid; idx < nkv * kMhKeys * vvec; idx += blockDim.x) {
+      const int row = idx / vvec, c = idx - row * vvec, h = row / kMhKeys, j = jb + row % kMhKeys;
+      const bool there = j <= max_pos && (j >= first_seen || j < mask.keep);
+      const size_t at = there ? ((size_t)table[j / page_size] * nkv + h) * page_size + (j % page_size) : 0;
+      cp_async_16(v_s + row * vs + c * 8, v_cache + at * dv + c0 + c * 8, there);
+    }
+    cp_async_commit();
+  };
+  if (n_first < n_last) fetch_k(tiles.key(n_first, kMhKeys));
+
+  // the mixture's matrix as a pair of bfloat16 (the rounding, and what it leaves), and zero rows for heads that do not exist
+  for (int idx = tid; idx < HP * (HP + kMhPad); idx += blockDim.x) {
+    const int h = idx / (HP + kMhPad), g = idx % (HP + kMhPad);
+    const float v = h < nq && g < nq ? (mix ? mix[h * nq + g] : h == g ? 1.f : 0.f) : 0.f;
+    const bf16 hi = __float2bfloat16_rn(v);
+    mix_s[idx] = hi;
+    mix_s[HP * (HP + kMhPad) + idx] = __float2bfloat16_rn(v - __bfloat162float(hi));
+  }
+  for (int idx = tid; idx < (HP - nq) * RS; idx += blockDim.x) {
+    p_hi[nq * RS + idx] = __float2bfloat16_rn(0.f);
+    p_lo[nq * RS + idx] = __float2bfloat16_rn(0.f);
+  }
+
+  // a warp's rows: HT heads of one KV head x R tokens; a thread's two rows are lane / 4 and lane / 4 + 8
+  const int head0 = warp * HT, kvh = head0 / G;
+  uint32_t qf[KS][4];
+  float L[2];
+  int pos[2], at[2], bias_at[2];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int r = (lane >> 2) + 8 * i, h = head0 + r / R, tok = r % R;
+    const bool live = i0 + tok < q_len;
+    pos[i] = live ? min_pos + tok : -1;
+    at[i] = h * RS + tok * kMhRow;
+    bias_at[i] = h * BL + tok + kMhKeys - 1;
+    L[i] = live ? lse[(size_t)(t0 + i0 + tok) * nq + h] : 0.f;
+    const bf16* src = q + ((size_t)(t0 + i0 + (live ? tok : 0)) * nq + h) * dk + (lane & 3) * 2;
+#pragma unroll
+    for (int k = 0; k < KS; ++k) {
+      const bool there = live && k * 16 < dk;
+      qf[k][i] = there ? *reinterpret_cast<const uint32_t*>(src + k * 16) : 0u;
+      qf[k][2 + i] = there ? *reinterpret_cast<const uint32_t*>(src + k * 16 + 8) : 0u;
+    }
+  }
+  float o[NT][4];
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) o[n][c] = 0.f;
+
+  for (int n = n_first; n < n_last; ++n) {
+    const int jb = tiles.key(n, kMhKeys);
+    if (bias.table) {                                          // bias_s[h][x]: distance min_pos - (jb + 31) + x
+      const int d0 = min_pos - jb - (kMhKeys - 1);
+      for (int idx = tid; idx < nq * BL; idx += blockDim.x) {
+        const int h = idx / BL, d = d0 + idx - h * BL;
+        bias_s[idx] = bias.at(h, max(d, 0)) * kLog2e;
+      }
+    }
+    cp_async_wait<0>();
+    __syncthreads();                                           // the keys are here; the values and weights before are read
+    fetch_v(jb);
+
+    float s[kMhKeys / 8][4];
+#pragma unroll
+    for (int x = 0; x < kMhKeys / 8; ++x)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) s[x][c] = 0.f;
+    const bf16* kb = k_s + (kvh * kMhKeys + (lane & 7) + (lane >> 4) * 8) * ks + ((lane >> 3) & 1) * 8;
+#pragma unroll
+    for (int k = 0; k < KS; ++k) {
+      if (k * 16 < dk) {
+#pragma unroll
+        for (int n2 = 0; n2 < kMhKeys / 16; ++n2) {
+          uint32_t b[4];
+          ldmatrix_x4(b, kb + n2 * 16 * ks + k * 16);
+          mma_bf16(s[2 * n2], qf[k], b[0], b[1]);
+          mma_bf16(s[2 * n2 + 1], qf[k], b[2], b[3]);
+        }
+      }
+    }
+    const bool whole = jb + kMhKeys - 1 <= min_pos && (mask.window <= 0 || jb > max_pos - mask.window) && i0 + R <= q_len;
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int x = 0; x < kMhKeys / 8; ++x) {
+        float p[2];
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+          const int jj = x * 8 + (lane & 3) * 2 + c;
+          p[c] = 0.f;
+          if (whole || mask.visible(pos[i], jb + jj))
+            p[c] = exp2f(fmaf(s[x][2 * i + c], scale2, (bias.table ? bias_s[bias_at[i] - jj] : 0.f) - L[i]));
+        }
+        const __nv_bfloat162 hi = __floats2bfloat162_rn(p[0], p[1]);
+        const float2 back = __bfloat1622float2(hi);
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(p[0] - back.x, p[1] - back.y);
+        const int to = at[i] + x * 8 + (lane & 3) * 2;
+        *reinterpret_cast<__nv_bfloat162*>(p_hi + to) = hi;
+        *reinterpret_cast<__nv_bfloat162*>(p_lo + to) = lo;
+      }
+    __syncthreads();                                           // all heads' weights are written; the keys are read
+    if (n + 1 < n_last) fetch_k(tiles.key(n + 1, kMhKeys));
+
+    // the mixture, in place: a warp takes 8 keys of a token at a time, all heads
+    for (int ct = warp; ct < R * (kMhKeys / 8); ct += warps) {
+      const int col = (ct / (kMhKeys / 8)) * kMhRow + (ct % (kMhKeys / 8)) * 8;
+      uint32_t b[HT][4];
+#pragma unroll
+      for (int k = 0; k < HT; ++k) ldmatrix_x4_trans(b[k], ((lane >> 4) ? p_lo : p_hi) + (k * 16 + (lane & 15)) * RS + col);
+      __syncwarp();
+#pragma unroll
+      for (int mt = 0; mt < HT; ++mt) {
+        float d[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int k = 0; k < HT; ++k) {
+          uint32_t a[4];
+          ldmatrix_x4(a, mix_s + (mt * 16 + (lane & 15)) * (HP + kMhPad) + k * 16 + (lane >> 4) * 8);
+          mma_bf16(d, a, b[k][2], b[k][3]);
+          mma_bf16(d, a, b[k][0], b[k][1]);
+          if (mix_low) {
+            ldmatrix_x4(a, mix_s + (HP + mt * 16 + (lane & 15)) * (HP + kMhPad) + k * 16 + (lane >> 4) * 8);
+            mma_bf16(d, a, b[k][0], b[k][1]);
+          }
+        }
+        bf16* w = p_hi + (mt * 16 + (lane >> 2)) * RS + col + (lane & 3) * 2;
+        *reinterpret_cast<__nv_bfloat162*>(w) = __floats2bfloat162_rn(d[0], d[1]);
+        *reinterpret_cast<__nv_bfloat162*>(w + 8 * RS) = __floats2bfloat162_rn(d[2], d[3]);
+      }
+    }
+    if (n + 1 < n_last) cp_async_wait<1>();
+    else cp_async_wait<0>();
+    __syncthreads();                                           // the mixture and the values are here
+
+    const bf16* wa = p_hi + (head0 + (lane & 15) / R) * RS + ((lane & 15) % R) * kMhRow + (lane >> 4) * 8;
+    const bf16* vb = v_s + (kvh * kMhKeys + (lane & 15)) * vs + (lane >> 4) * 8;
+#pragma unroll
+    for (int kk = 0; kk < kMhKeys / 16; ++kk) {
+      uint32_t a[4];
+      ldmatrix_x4(a, wa + kk * 16);
+#pragma unroll
+      for (int n2 = 0; n2 < NT / 2; ++n2) {
+        if (n2 * 16 < width) {
+          uint32_t b[4];
+          ldmatrix_x4_trans(b, vb + kk * 16 * vs + n2 * 16);
+          mma_bf16(o[2 * n2], a, b[0], b[1]);
+          mma_bf16(o[2 * n2 + 1], a, b[2], b[3]);
+        }
+      }
+    }
+  }
+
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int r = (lane >> 2) + 8 * i, h = head0 + r / R, tok = i0 + r % R;
+    if (tok >= q_len) continue;
+#pragma unroll
+    for (int n = 0; n < NT; ++n) {
+      if (n * 8 >= width) continue;
+      const int c = h * dv + c0 + n * 8 + (lane & 3) * 2;
+      if (nsplit > 1) {
+        *reinterpret_cast<float2*>(part + ((size_t)(t0 + tok) * nsplit + split) * nq * dv + c) = make_float2(o[n][2 * i], o[n][2 * i + 1]);
+      } else {
+        const float a = o[n][2 * i] * gate.at(t0 + tok, c), b = o[n][2 * i + 1] * gate.at(t0 + tok, c + 1);
+        *reinterpret_cast<__nv_bfloat162*>(out + (size_t)(t0 + tok) * nq * dv + c) = __floats2bfloat162_rn(a, b);
+      }
+    }
+  }
+}
+
+// out[t, c] = (sum over the key slices of part[t, slice, c]) * gate; the slices' weights are finished, so they just add.
+__global__ void mixed_head_add_kernel(const float* __restrict__ part, bf16* __restrict__ out, int nsplit, int columns,
+                                      ElementGate gate) {
+  pdl_wait();
+  pdl_trigger();
+  const size_t t = blockIdx.x;
+  for (int c = threadIdx.x; c < columns; c += blockDim.x) {
+    float a = 0.f;
+    for (int s = 0; s < nsplit; ++s) a += part[(t * nsplit + s) * columns + c];
+    out[t * columns + c] = __float2bfloat16_rn(a * gate.at(t, c));
+  }
+}
+
+// ---- decode steps ----------------------------------------------------------------------------------------------------
+__device__ __forceinline__ void mh_cluster_sync() {
+  asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+// The float at `p` of this block's shared memory, in block `rank` of the cluster.
+__device__ __forceinline__ float mh_remote(const float* p, int rank) {
+  const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
+  uint32_t r;
+  float v;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(a), "r"(rank));
+  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(r) : "memory");
+  return v;
+}
+
+constexpr int kMdThreads = 256, kMdWarps = kMdThreads / 32;
+
+struct MixDecodeLayout {             // offsets in bytes of a block's shared memory
+  int q, tile, tile_bytes, w, s, stats, lse, mix, total, keys;      // keys: a head's row of scores
+  __host__ __device__ MixDecodeLayout(int nq, int nkv, int row_tiles, int dk, int dv, int tiles_here, int nbuf) {
+    const int rows = nkv * row_tiles * 16, wide = (dk > dv ? dk : dv) + kMhPad;
+    keys = tiles_here * kMhKeys + 4;
+    q = 0;
+    tile = q + rows * (dk + kMhPad) * 2;
+    tile_bytes = nkv * kMhKeys * wide * 2;
+    int buffers = nbuf * tile_bytes;
+    if (buffers < nq * dv * 4) buffers = nq * dv * 4;                // the block's sums lie there at the end
+    w = tile + buffers;
+    s = w + rows * kMhRow * 2;
+    stats = s + nq * keys * 4;
+    lse = stats + nq * 8;
+    mix = (lse + nq * 4 + 15) / 16 * 16;
+    total = mix + nq * (nq + 1) * 4;
+  }
+};
+
+// UN: units of 32 value columns of 16 rows that a warp holds.  grid (cluster, entries).
+template <int UN>
+__global__ void __launch_bounds__(kMdThreads)
+mixed_head_attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache,
+                                   const bf16* __restrict__ v_cache, bf16* __restrict__ out,
+                                   const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_q,
+                                   const int* __restrict__ kv_lens, int nq, int nkv, int row_tiles, int dk, int dv,
+                                   int page_size, float scale2, MixMask mask, DistanceBias bias,
+                                   const float* __restrict__ mix, ElementGate gate, int tiles_cap, int nbuf) {
+  pdl_wait();
+  pdl_trigger();
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  const MixDecodeLayout at(nq, nkv, row_tiles, dk, dv, tiles_cap, nbuf);
+  bf16* q_s = reinterpret_cast<bf16*>(smem_raw + at.q);        // [nkv][row_tiles * 16][dk + 8]
+  bf16* w_s = reinterpret_cast<bf16*>(smem_raw + at.w);        // [nkv][row_tiles * 16][40]
+  float* s_s = reinterpret_cast<float*>(smem_raw + at.s);      // [nq][keys]
+  float* stats = reinterpret_cast<float*>(smem_raw + at.stats);     // [nq][2]: maximum and sum of the slice
+  float* lse = reinterpret_cast<float*>(smem_raw + at.lse);    // [nq]
+  float* mix_s = reinterpret_cast<float*>(smem_raw + at.mix);  // [nq][nq + 1]
+  float* o_s = reinterpret_cast<float*>(smem_raw + at.tile);   // [nq][dv], at the end
+  const int rank = blockIdx.x, cluster = gridDim.x, e = blockIdx.y;
+  const int G = nq / nkv, rows_c = row_tiles * 16, ks = dk + kMhPad, vs = dv + kMhPad;
+  const int t = cu_q[e], pos = kv_lens[e] - 1;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int* table = block_table + (size_t)e * table_stride;
+  const MixTiles tiles(mask, pos, pos, kMhKeys);
+  int per = (tiles.count + cluster - 1) / cluster;             // (never above tiles_cap: the host planned for the longest)
+  if (per > tiles_cap) per = tiles_cap;
+  const int n0 = min(tiles.count, rank * per), n_here = min(tiles.count - n0, per);
+  const int kvec = dk / 8, vvec = dv / 8;
+
+  // stage x: 0 .. n_here - 1 fetch keys, n_here .. 2 n_here - 1 values, buffer x % nbuf
+  auto fetch = [&](int x) {
+    const bool values = x >= n_here;
+    const int jb = tiles.key(n0 + (values ? x - n_here : x), kMhKeys);
+    bf16* dst = reinterpret_cast<bf16*>(smem_raw + at.tile + (x % nbuf) * at.tile_bytes);
+    const int vec = values ? vvec : kvec, stride = values ? vs : ks, dim = values ? dv : dk;
+    const bf16* pool = values ? v_cache : k_cache;
+    for (int idx = tid; idx < nkv * kMhKeys * vec; idx += blockDim.x) {
+      const int row = idx / vec, c = idx - row * vec, h = row / kMhKeys, j = jb + row % kMhKeys;
+      const bool there = mask.visible(pos, j);
+      const size_t src = there ? ((size_t)table[j / page_size] * nkv + h) * page_size + (j % page_size) : 0;
+      cp_async_16(dst + row * stride + c * 8, pool + src * dim + c * 8, there);
+    }
+    cp_async_commit();
+  };
+  const int stages = 2 * n_here;
+  if (stages) fetch(0);
+  for (int idx = tid; idx < nkv * rows_c * kvec; idx += blockDim.x) {
+    const int row = idx / kvec, c = idx - row * kvec, h = row / rows_c, r = row % rows_c;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (r < G) v = *reinterpret_cast<const uint4*>(q + ((size_t)t * nq + h * G + r) * dk + c * 8);
+    *reinterpret_cast<uint4*>(q_s + row * ks + c * 8) = v;
+  }
+  for (int idx = tid; idx < nkv * rows_c * kMhRow; idx += blockDim.x) w_s[idx] = __float2bfloat16_rn(0.f);
+  for (int idx = tid; idx < nq * nq; idx += blockDim.x)
+    mix_s[idx / nq * (nq + 1) + idx % nq] = mix ? mix[idx] : idx / nq == idx % nq ? 1.f : 0.f;
+
+  float o[UN][4][4];
+#pragma unroll
+  for (int u = 0; u < UN; ++u)
+#pragma unroll
+    for (int n = 0; n < 4; ++n)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) o[u][n][c] = 0.f;
+  const int col_units = (dv + 31) / 32, units = nkv * row_tiles * col_units;
+
+  for (int x = 0; x < stages; ++x) {
+    if (nbuf > 1 && x + 1 < stages) {
+      fetch(x + 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    const bf16* buf = reinterpret_cast<const bf16*>(smem_raw + at.tile + (x % nbuf) * at.tile_bytes);
+    if (x < n_here) {
+      // scores of 16 rows x 16 keys a job
+      const int jb = tiles.key(n0 + x, kMhKeys);
+      for (int job = warp; job < nkv * row_tiles * (kMhKeys / 16); job += kMdWarps) {
+        const int n2 = job % (kMhKeys / 16), rt = job / (kMhKeys / 16), h = rt / row_tiles, r0 = (rt % row_tiles) * 16;
+        float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+        const bf16* qa = q_s + (rt * 16 + (lane & 15)) * ks + (lane >> 4) * 8;
+        const bf16* kb = buf + (h * kMhKeys + n2 * 16 + (lane & 7) + (lane >> 4) * 8) * ks + ((lane >> 3) & 1) * 8;
+        for (int k0 = 0; k0 < dk; k0 += 16) {
+          uint32_t a[4], b[4];
+          ldmatrix_x4(a, qa + k0);
+          ldmatrix_x4(b, kb + k0);
+          mma_bf16(s[0], a, b[0], b[1]);
+          mma_bf16(s[1], a, b[2], b[3]);
+        }
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int r = r0 + (lane >> 2) + 8 * i;
+          if (r >= G) continue;
+#pragma unroll
+          for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int c = 0; c < 2; ++c) {
+              const int jj = n2 * 16 + n * 8 + (lane & 3) * 2 + c;
+              float v = -CUDART_INF_F;
+              if (mask.visible(pos, jb + jj)) v = fmaf(s[n][2 * i + c], scale2, bias.at(h * G + r, pos - jb - jj) * kLog2e);
+              s_s[(size_t)(h * G + r) * at.keys + x * kMhKeys + jj] = v;
+            }
+        }
+      }
+      if (x == n_here - 1) {
+        // the slice's maximum and sum of every head, exchanged; then the scores become finished weights
+        __syncthreads();
+        for (int h = warp; h < nq; h += kMdWarps) {
+          float m = -CUDART_INF_F, l = 0.f;
+          for (int j = lane; j < n_here * kMhKeys; j += 32) m = fmaxf(m, s_s[(size_t)h * at.keys + j]);
+          m = warp_max(m);
+          if (m != -CUDART_INF_F)
+            for (int j = lane; j < n_here * kMhKeys; j += 32) l += exp2f(s_s[(size_t)h * at.keys + j] - m);
+          l = warp_sum(l);
+          if (lane == 0) { stats[2 * h] = m; stats[2 * h + 1] = l; }
+        }
+      }
+    }
+    if (x == n_here - 1) {
+      mh_cluster_sync();
+      for (int h = tid; h < nq; h += blockDim.x) {
+        float m = -CUDART_INF_F, l = 0.f;
+        for (int r = 0; r < cluster; ++r) m = fmaxf(m, mh_remote(stats + 2 * h, r));
+        for (int r = 0; r < cluster; ++r) {
+          const float mr = mh_remote(stats + 2 * h, r);
+          if (mr != -CUDART_INF_F) l += mh_remote(stats + 2 * h + 1, r) * exp2f(mr - m);
+        }
+        lse[h] = m + log2f(l);
+      }
+      __syncthreads();
+      for (int h = warp; h < nq; h += kMdWarps)
+        for (int j = lane; j < n_here * kMhKeys; j += 32) s_s[(size_t)h * at.keys + j] = exp2f(s_s[(size_t)h * at.keys + j] - lse[h]);
+    }
+    if (x >= n_here) {
+      const int j0 = (x - n_here) * kMhKeys;
+      for (int h = warp; h < nq; h += kMdWarps) {
+        float a = 0.f;
+        for (int g = 0; g < nq; ++g) a += mix_s[h * (nq + 1) + g] * s_s[(size_t)g * at.keys + j0 + lane];
+        w_s[((h / G) * rows_c + h % G) * kMhRow + lane] = __float2bfloat16_rn(a);
+      }
+      __syncthreads();
+#pragma unroll
+      for (int u = 0; u < UN; ++u) {
+        const int unit = warp + u * kMdWarps;
+        if (unit < units) {
+          const int rt = unit / col_units, cu = (unit % col_units) * 32, h = rt / row_tiles;
+#pragma unroll
+          for (int kk = 0; kk < kMhKeys / 16; ++kk) {
+            uint32_t a[4];
+            ldmatrix_x4(a, w_s + (rt * 16 + (lane & 15)) * kMhRow + kk * 16 + (lane >> 4) * 8);
+#pragma unroll
+            for (int n2 = 0; n2 < 2; ++n2) {
+              if (cu + n2 * 16 < dv) {
+                uint32_t b[4];
+                ldmatrix_x4_trans(b, buf + (h * kMhKeys + kk * 16 + (lane & 15)) * vs + cu + n2 * 16 + (lane >> 4) * 8);
+                mma_bf16(o[u][2 * n2], a, b[0], b[1]);
+                mma_bf16(o[u][2 * n2 + 1], a, b[2], b[3]);
+              }
+            }
+          }
+        }
+      }
+    }
+    __syncthreads();                                           // the buffer and the weights are read
+    if (nbuf == 1 && x + 1 < stages) fetch(x + 1);
+  }
+  if (n_here == 0) {                                           // a block without keys still takes part in the exchange
+    for (int h = tid; h < nq; h += blockDim.x) { stats[2 * h] = -CUDART_INF_F; stats[2 * h + 1] = 0.f; }
+    mh_cluster_sync();
+  }
+
+  // the block's sums, then every block adds a share of the columns over the cluster
+#pragma unroll
+  for (int u = 0; u < UN; ++u) {
+    const int unit = warp + u * kMdWarps;
+    if (unit < units) {
+      const int rt = unit / col_units, cu = (unit % col_units) * 32, h = rt / row_tiles, r0 = (rt % row_tiles) * 16;
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int r = r0 + (lane >> 2) + 8 * i;
+        if (r >= G) continue;
+#pragma unroll
+        for (int n = 0; n < 4; ++n) {
+          const int c = cu + n * 8 + (lane & 3) * 2;
+          if (c < dv) {
+            o_s[(size_t)(h * G + r) * dv + c] = o[u][n][2 * i];
+            o_s[(size_t)(h * G + r) * dv + c + 1] = o[u][n][2 * i + 1];
+          }
+        }
+      }
+    }
+  }
+  mh_cluster_sync();
+  for (int c = rank * kMdThreads + tid; c < nq * dv; c += cluster * kMdThreads) {
+    float a = 0.f;
+    for (int r = 0; r < cluster; ++r) a += mh_remote(o_s + c, r);
+    out[(size_t)t * nq * dv + c] = __float2bfloat16_rn(a * gate.at(t, c));
+  }
+  mh_cluster_sync();                                           // nobody leaves while its sums are read
+}
+
+}  // namespace srlm
+
+using namespace srlm;
+
+static int mh_heads_tiles(int nq, int nkv) {      // 16-head tiles of the rows form, 0: not taken
+  if (nq <= 16) return 1;
+  if (nq <= 32 && nq % 2 == 0 && (nq / nkv) % 2 == 0) return 2;
+  return 0;
+}
+static int mh_slab(int dv) { return dv <= 128 ? dv : 128; }
+static size_t mh_rows_smem(int nq, int nkv, int dk, int dv) {
+  const int ht = mh_heads_tiles(nq, nkv), hp = 16 * ht, R = 16 / ht, rs = R * kMhRow + kMhPad, slab = mh_slab(dv);
+  return (size_t)nkv * kMhKeys * (dk + kMhPad) * 2 + (size_t)nkv * kMhKeys * (slab + kMhPad) * 2 + 2ull * hp * rs * 2 +
+         2ull * hp * (hp + kMhPad) * 2 + (size_t)nq * (R + kMhKeys) * 4;
+}
+static int mh_lse_span(int G) { return kLseKeys + kLseRows / G + 1; }
+static size_t mh_lse_smem(int G, int dk) {
+  return (size_t)(kLseRows + 2 * kLseKeys) * (dk + kMhPad) * 2 + 2ull * G * mh_lse_span(G) * 4;
+}
+
+// Whether the tensor-core forms take these sizes (bfloat16 cache): up to 16 heads, or an even number up to 32 with an even
+// number a KV head; key size a multiple of 16 up to 128, value size a multiple of 16.
+extern "C" int srlm_mixed_head_attention_mma_takes(int nq, int nkv, int dk, int dv) {
+  if (nq <= 0 || nkv <= 0 || nq % nkv || !mh_heads_tiles(nq, nkv) || dk <= 0 || dk % 16 || dk > 128 || dv <= 0 || dv % 16) return 0;
+  return mh_rows_smem(nq, nkv, dk, dv) <= 220 * 1024 && mh_lse_smem(nq / nkv, dk) <= 220 * 1024;
+}
+
+extern "C" int srlm_mixed_head_tokens(int nq, int nkv) { const int ht = mh_heads_tiles(nq, nkv); return ht ? 16 / ht : 0; }
+
+// q bfloat16 [T, nq, dk]; lse float32 [T, nq] (written by the first kernel, read by the second); part float32
+// [T, nsplit, nq dv] when nsplit > 1 (the visible keys in nsplit slices, added by a third kernel).
+extern "C" int srlm_mixed_head_attention_mma(const void* q, const void* k_cache, const void* v_cache, void* out, float* lse,
+                                             const int* block_table, int table_stride, const int* cu_q, const int* kv_lens,
+                                             int n_entries, int max_q_len, int T, int nq, int nkv, int dk, int dv,
+                                             int page_size, float scale, int window, int keep, const float* bias, int n_dist,
+                                             const float* mix, int mix_low, const float* gate_logits, long long ld_gate,
+                                             int nsplit, float* part, cudaStream_t stream) {
+  if (n_entries <= 0 || max_q_len <= 0 || T <= 0) return ST_OK;
+  if (!srlm_mixed_head_attention_mma_takes(nq, nkv, dk, dv) || page_size <= 0 || window < 0 || keep < 0 || (bias && n_dist <= 0) || !lse)
+    return refuse(ST_BAD_SIZE, "mixed_head_attention_mma: nq=%d nkv=%d dk=%d dv=%d", nq, nkv, dk, dv);
+  if ((((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15) != 0)
+    return refuse(ST_BAD_ALIGN, "mixed_head_attention_mma: queries and pools must be 16-byte aligned");
+  if (nsplit < 1) nsplit = 1;
+  if (nsplit > 1 && !part) return refuse(ST_BAD_SIZE, "mixed_head_attention_mma: %d key slices need a workspace", nsplit);
+  const int G = nq / nkv, ht = mh_heads_tiles(nq, nkv), R = 16 / ht, slab = mh_slab(dv), slabs = (dv + slab - 1) / slab;
+  if (n_entries > 65535 || nkv > 65535 || (long long)slabs * nsplit > 65535)
+    return refuse(ST_BAD_SIZE, "mixed_head_attention_mma: %d entries", n_entries);
+  const MixMask mask{window, window > 0 ? keep : 0};
+  const DistanceBias db{bias, n_dist};
+  const ElementGate gate{gate_logits, ld_gate};
+  const float scale2 = scale * kLog2e;
+  {
+    const size_t smem = mh_lse_smem(G, dk);
+    if (smem > 48 * 1024) cudaFuncSetAttribute(mixed_head_lse_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    launch_pdl(mixed_head_lse_kernel, dim3((unsigned)(((long long)max_q_len * G + kLseRows - 1) / kLseRows), nkv, n_entries), dim3(128),
+               smem, stream, (const bf16*)q, (const bf16*)k_cache, lse, block_table, table_stride, cu_q, kv_lens, nq, nkv, dk,
+               page_size, scale2, mask, db, mh_lse_span(G));
+  }
+  const size_t smem = mh_rows_smem(nq, nkv, dk, dv);
+  const dim3 grid((unsigned)((max_q_len + R - 1) / R), (unsigned)(slabs * nsplit), (unsigned)n_entries);
+  const int threads = nq / ht * 32;
+#define SRLM_MH(KS, NT, HT)                                                                                             \
+  do {                                                                                                                  \
+    auto kern = mixed_head_attention_mma_kernel<KS, NT, HT>;                                                            \
+    if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);           \
+    launch_pdl(kern, grid, dim3(threads), smem, stream, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, lse, \
+               (bf16*)out, block_table, table_stride, cu_q, kv_lens, nq, nkv, dk, dv, slab, page_size, scale2, mask, db, \
+               mix, mix_low, gate, nsplit, part);                                                                       \
+  } while (0)
+#define SRLM_MH_SIZES(HT)                               \
+  do {                                                  \
+    if (dk <= 64 && slab <= 64) SRLM_MH(4, 8, HT);      \
+    else SRLM_MH(8, 16, HT);                            \
+  } while (0)
+  if (ht == 1) SRLM_MH_SIZES(1);
+  else SRLM_MH_SIZES(2);
+#undef SRLM_MH_SIZES
+#undef SRLM_MH
+  if (nsplit > 1)
+    launch_pdl(mixed_head_add_kernel, dim3(T), dim3(256), 0, stream, part, (bf16*)out, nsplit, nq * dv, gate);
+  return launched();
+}
+
+// Bytes of shared memory of a block of the decode form whose slice has tiles_here tiles of 32 keys; 0: sizes not taken.
+extern "C" int srlm_mixed_head_decode_smem(int nq, int nkv, int dk, int dv, int tiles_here, int nbuf) {
+  if (nq <= 0 || nkv <= 0 || nq % nkv || nq > 128 || dk <= 0 || dk % 16 || dv <= 0 || dv % 16) return 0;
+  const int row_tiles = (nq / nkv + 15) / 16, units = nkv * row_tiles * ((dv + 31) / 32);
+  if (units > 8 * kMdWarps) return 0;
+  const MixDecodeLayout at(nq, nkv, row_tiles, dk, dv, tiles_here, nbuf);
+  return at.total <= 225 * 1024 ? at.total : 0;
+}
+
+// One token an entry; the visible keys of an entry, at most 32 * tiles_here * cluster of them, in `cluster` (1, 2, 4, 8 or 16)
+// slices of whole tiles.
+extern "C" int srlm_mixed_head_attention_decode(const void* q, const void* k_cache, const void* v_cache, void* out,
+                                                const int* block_table, int table_stride, const int* cu_q,
+                                                const int* kv_lens, int n_entries, int nq, int nkv, int dk, int dv,
+                                                int page_size, float scale, int window, int keep, const float* bias, int n_dist,
+                                                const float* mix, const float* gate_logits, long long ld_gate, int cluster,
+                                                int tiles_here, int nbuf, cudaStream_t stream) {
+  if (n_entries <= 0) return ST_OK;
+  const int smem = srlm_mixed_head_decode_smem(nq, nkv, dk, dv, tiles_here, nbuf);
+  if (!smem || page_size <= 0 || window < 0 || keep < 0 || (bias && n_dist <= 0) || tiles_here <= 0 || nbuf < 1 || nbuf > 2 ||
+      n_entries > 65535 || (cluster != 1 && cluster != 2 && cluster != 4 && cluster != 8 && cluster != 16))
+    return refuse(ST_BAD_SIZE, "mixed_head_attention_decode: nq=%d nkv=%d dk=%d dv=%d cluster=%d of %d tiles", nq, nkv, dk, dv,
+                  cluster, tiles_here);
+  if ((((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15) != 0)
+    return refuse(ST_BAD_ALIGN, "mixed_head_attention_decode: queries and pools must be 16-byte aligned");
+  const int row_tiles = (nq / nkv + 15) / 16, units = nkv * row_tiles * ((dv + 31) / 32);
+  const MixMask mask{window, window > 0 ? keep : 0};
+  const DistanceBias db{bias, n_dist};
+  const ElementGate gate{gate_logits, ld_gate};
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(cluster, n_entries, 1);
+  cfg.blockDim = dim3(kMdThreads, 1, 1);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = stream;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = cluster;
+  attr[0].val.clusterDim.y = 1;
+  attr[0].val.clusterDim.z = 1;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = pdl_enabled() ? 1 : 0;
+  cfg.attrs = attr;
+  cfg.numAttrs = 2;
+#define SRLM_MD(UN)                                                                                                   \
+  do {                                                                                                                \
+    auto kern = mixed_head_attention_decode_kernel<UN>;                                                               \
+    if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);              \
+    if (cluster > 8) cudaFuncSetAttribute(kern, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);                   \
+    cudaLaunchKernelEx(&cfg, kern, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, (bf16*)out, block_table, \
+                       table_stride, cu_q, kv_lens, nq, nkv, row_tiles, dk, dv, page_size, scale * kLog2e, mask, db, mix, \
+                       gate, tiles_here, nbuf);                                                                       \
+  } while (0)
+  if (units <= 2 * kMdWarps) SRLM_MD(2);
+  else if (units <= 4 * kMdWarps) SRLM_MD(4);
+  else SRLM_MD(8);
+#undef SRLM_MD
+  return launched();
+}

@@ -76,6 +76,9 @@ class KernelLibrary:
         self.sinks_in_tcgen05_prefill = True            # attention with sinks, heads of 128: prompts on the tcgen05 kernel
         self.grouped_products_on_tensor_cores = True    # routed experts in bfloat16: mma.sync, when the sizes fit
         self.grouped_products_in_tensor_memory = True   # ... and steps of many tokens: the persistent tcgen05 kernel
+        self.mixed_heads_on_tensor_cores = True         # attention that mixes its heads, bfloat16: mma.sync, when the sizes fit
+        self.mixed_heads_cluster = 16                   # ... most blocks of a decode step's cluster
+        self.split_mixed_heads = True                   # ... short prompts: the keys in slices
         self.grouped_pairs = True                       # ... whose largest steps run pairs of SMs on tiles of 256 tokens
 
     @property
@@ -1236,25 +1239,82 @@ class KernelLibrary:
             _ptr(kv_slot), C.c_int(int(write_kv)), C.c_int(proj.shape[0]), C.c_int(nq), C.c_int(nkv), C.c_int(dk), C.c_int(dv),
             C.c_int(k_cache.shape[2]), _stream()), "attention_wide_norm_append")
 
+    def mixed_head_query_dtype(self, dtype, nq, nkv, dk, dv):
+        """The dtype mixed_head_attention takes its queries in: bfloat16 where its tensor-core forms serve, else float32."""
+        on = (dtype == torch.bfloat16 and self.mixed_heads_on_tensor_cores
+              and self.lib.srlm_mixed_head_attention_mma_takes(C.c_int(nq), C.c_int(nkv), C.c_int(dk), C.c_int(dv)))
+        return torch.bfloat16 if on else torch.float32
+
+    @staticmethod
+    def mixed_head_tiles(kv_bound: int, window: int, keep_first: int) -> int:
+        """Most tiles of 32 keys that one query of a context of at most kv_bound keys sees."""
+        whole = (kv_bound + 31) // 32
+        return min(whole, (keep_first + 31) // 32 + (window + 30) // 32 + 1) if window else whole
+
+    def mixed_head_decode_plan(self, n_entries, tiles, smem_of):
+        """(cluster, tiles a block, buffers) of the decode form, or None: as many blocks an entry as keep the step within
+        one block an SM, more when a block's slice does not fit its shared memory (smem_of(tiles, buffers), 0: no)."""
+        sizes = [c for c in (1, 2, 4, 8, 16) if c <= self.mixed_heads_cluster]
+        fits = [c for c in sizes if c <= tiles and c * n_entries <= self.SMS] or [1]
+        for c in [fits[-1]] + [c for c in sizes if c > fits[-1]]:
+            here = -(-tiles // c)
+            for nbuf in (2, 1):
+                if smem_of(here, nbuf):
+                    return c, here, nbuf
+        return None
+
     def mixed_head_attention(self, ctx, q, k_cache, v_cache, out, block_table, nq, nkv, dk, dv, scale, window=0, keep_first=0,
-                             bias=None, mix=None, gate=None):
+                             bias=None, mix=None, gate=None, mix_low=True):
         """Causal attention of the batch of ``ctx`` whose heads exchange their weights behind the softmax: head h applies
-        sum_g mix[h, g] p_g to the values of its own KV head.  q [T, nq dk]; pages as paged_attention_general's; out
-        [T, nq dv] in the cache's dtype; bias float32 [nq, n] or None: added to the scaled score of a key at distance
-        n' = min(i - j, n - 1); window > 0: a query sees itself, the window - 1 keys before it and the first keep_first
-        keys; mix float32 [nq, nq] or None; gate (float32 tensor [T, >= column + nq dv], column) or None: every element is
-        multiplied by the logistic of its own column."""
+        sum_g mix[h, g] p_g to the values of its own KV head.  q [T, nq dk] in the dtype mixed_head_query_dtype names;
+        pages as paged_attention_general's; out [T, nq dv] in the cache's dtype; bias float32 [nq, n] or None: added to the
+        scaled score of a key at distance n' = min(i - j, n - 1); window > 0: a query sees itself, the window - 1 keys
+        before it and the first keep_first keys; mix float32 [nq, nq] or None; gate (float32 tensor [T, >= column + nq dv],
+        column) or None: every element is multiplied by the logistic of its own column.  mix_low False: mix holds bfloat16
+        numbers.
+
+        bfloat16 queries: the tensor-core forms of mixed_head_attention_mma.cu -- a cluster of blocks an entry for decode
+        steps, else the softmax's sums first and the mixture behind them.  float32 queries: float32 arithmetic, a block a
+        token."""
         T = q.shape[0]
         gate_args = (C.c_void_p(0), C.c_longlong(0)) if gate is None else self._columns(gate[0], gate[1], nq * dv)
-        n_dist = bias.shape[1] if bias is not None else 0
-        if q.dtype != torch.float32:
-            raise ShapeError("mixed_head_attention: float32 queries")
-        self._check(self.lib.srlm_mixed_head_attention(
-            _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), dtype_code(k_cache.dtype), dtype_code(out.dtype),
-            _ptr(block_table), C.c_int(block_table.stride(0)), _ptr(ctx.entry_of_token), _ptr(ctx.positions), C.c_int(T),
-            C.c_int(nq), C.c_int(nkv), C.c_int(dk), C.c_int(dv), C.c_int(k_cache.shape[2]), C.c_float(scale),
-            C.c_int(window or 0), C.c_int(keep_first), _ptr(bias), C.c_int(n_dist), _ptr(mix), *gate_args, _stream()),
-            "mixed_head_attention")
+        score_args = (C.c_float(scale), C.c_int(window or 0), C.c_int(keep_first), _ptr(bias),
+                      C.c_int(bias.shape[1] if bias is not None else 0), _ptr(mix))
+        if q.dtype == torch.float32:
+            self._check(self.lib.srlm_mixed_head_attention(
+                _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), dtype_code(k_cache.dtype), dtype_code(out.dtype),
+                _ptr(block_table), C.c_int(block_table.stride(0)), _ptr(ctx.entry_of_token), _ptr(ctx.positions), C.c_int(T),
+                C.c_int(nq), C.c_int(nkv), C.c_int(dk), C.c_int(dv), C.c_int(k_cache.shape[2]), *score_args, *gate_args,
+                _stream()), "mixed_head_attention")
+            return
+        if k_cache.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
+            raise ShapeError("mixed_head_attention: bfloat16 queries come with bfloat16 pages and output")
+        n = ctx.n_entries
+        batch_args = (_ptr(block_table), C.c_int(block_table.stride(0)), _ptr(ctx.cu_q), _ptr(ctx.kv_lens), C.c_int(n))
+        size_args = (C.c_int(nq), C.c_int(nkv), C.c_int(dk), C.c_int(dv), C.c_int(k_cache.shape[2]))
+        tiles = self.mixed_head_tiles(ctx.kv_bound, window or 0, keep_first)
+        if ctx.max_q_len == 1:
+            plan = self.mixed_head_decode_plan(n, tiles, lambda here, nbuf: self.lib.srlm_mixed_head_decode_smem(
+                *size_args[:4], C.c_int(here), C.c_int(nbuf)))
+            if plan is not None:
+                self._check(self.lib.srlm_mixed_head_attention_decode(
+                    _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), *batch_args, *size_args, *score_args, *gate_args,
+                    *(C.c_int(v) for v in plan), _stream()), "mixed_head_attention_decode")
+                return
+        lse = ctx.workspace.get("mixed_attn.lse", T, nq, torch.float32)
+        tokens = int(self.lib.srlm_mixed_head_tokens(C.c_int(nq), C.c_int(nkv)))
+        nsplit, part = 1, None
+        if self.split_mixed_heads and ctx.max_q_len > 1:
+            # blocks for tokens x entries x slabs of 128 value columns; few of them: the keys in slices of 4 tiles or more
+            blocks = sum(-(-ql // tokens) for ql in ctx.host["q_lens"]) * -(-dv // 128)
+            nsplit = max(1, min(self.SMS // max(1, blocks), tiles // 4, 8))
+            if nsplit > 1:
+                part = ctx.workspace.get("mixed_attn.part", T * nsplit, nq * dv, torch.float32, reserve=0)
+        self._check(self.lib.srlm_mixed_head_attention_mma(
+            _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(lse), *batch_args, C.c_int(ctx.max_q_len), C.c_int(T),
+            *size_args, *score_args, C.c_int(int(mix_low)), *gate_args, C.c_int(nsplit), _ptr(part), _stream()),
+            "mixed_head_attention_mma")
+        self.launches += 2 if nsplit > 1 else 1          # the softmax's sums ahead of it, the kernel that adds the slices
 
     # ---- retention --------------------------------------------------------------------------------------
     def retention(self, ctx, proj, rotation, decay, eps, state, out, H, d, dv):

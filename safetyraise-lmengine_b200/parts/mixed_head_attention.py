@@ -69,6 +69,7 @@ class MixedHeadAttention(Part):
             ids = torch.tensor(distance_buckets(table.shape[0], spec.bias_max), device=table.device)
             self.bias = table[ids].t().contiguous()
         self.mix = tensors[p + nm.head_mix].float().contiguous() if spec.head_mix else None
+        self.mix_low = self.mix is not None and not bool((self.mix.bfloat16().float() == self.mix).all())
         self.out = Linear(tensors[p + nm.o], p + nm.o)
 
     @classmethod
@@ -99,11 +100,12 @@ class MixedHeadAttention(Part):
         T = x.shape[0]
         proj = self.proj(ctx, x, "mixed_attn.proj", out_dtype=torch.float32)
         k_pool, v_pool, group = ctx.cache.kv_of_entry(run_step.cache)
-        q = ctx.workspace.get("mixed_attn.q", T, s.heads * s.head_dim, torch.float32)
+        q = ctx.workspace.get("mixed_attn.q", T, s.heads * s.head_dim,
+                              ops.mixed_head_query_dtype(ctx.dtype, s.heads, s.kv_heads, s.head_dim, s.v_head_dim))
         ops.attention_wide_norm_append(proj, self.q_norm, self.k_norm, s.qk_norm_eps, q, k_pool, v_pool, ctx.kv_slot[group],
                                        s.heads, s.kv_heads, s.head_dim, s.v_head_dim, run_step.writes_cache)
         attended = ctx.workspace.get("mixed_attn.out", T, s.heads * s.v_head_dim, ctx.dtype)
         ops.mixed_head_attention(ctx, q, k_pool, v_pool, attended, ctx.block_tables[group], s.heads, s.kv_heads, s.head_dim,
                                  s.v_head_dim, s.softmax_scale, s.window or 0, s.keep_first, bias=self.bias, mix=self.mix,
-                                 gate=(proj, self.gate_offset) if s.output_gate else None)
+                                 gate=(proj, self.gate_offset) if s.output_gate else None, mix_low=self.mix_low)
         return self.out(ctx, attended, "mixed_attn.o")
