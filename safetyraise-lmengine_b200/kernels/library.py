@@ -79,6 +79,7 @@ class KernelLibrary:
         self.mixed_heads_on_tensor_cores = True         # attention that mixes its heads, bfloat16: mma.sync, when the sizes fit
         self.mixed_heads_cluster = 16                   # ... most blocks of a decode step's cluster
         self.split_mixed_heads = True                   # ... short prompts: the keys in slices
+        self.retention_in_chunks = True                 # retention: portions in chunks of 64 tokens
         self.grouped_pairs = True                       # ... whose largest steps run pairs of SMs on tiles of 256 tokens
 
     @property
@@ -1317,10 +1318,13 @@ class KernelLibrary:
         self.launches += 2 if nsplit > 1 else 1          # the softmax's sums ahead of it, the kernel that adds the slices
 
     # ---- retention --------------------------------------------------------------------------------------
+    RETENTION_WALK = 8       # most tokens of an entry that walks its state token by token
+
     def retention(self, ctx, proj, rotation, decay, eps, state, out, H, d, dv):
         """out [T, H dv] = per head o / sqrt(mean(o^2) + eps) * silu(gate), o the read-out of a state that fades by decay[h]
         a token, from the stacked projection q | k | v | gate (float32), whose leading 2 * pairs elements of every q and k
-        head are turned by ``rotation``; state float32 [slots, >= H d dv], renewed."""
+        head are turned by ``rotation``; state float32 [slots, >= H d dv], renewed.  Entries of up to RETENTION_WALK tokens are
+        walked token by token, longer ones taken in chunks of 64."""
         pairs = rotation.pairs if rotation is not None else 0
         if pairs and rotation.interleaved:
             raise ShapeError("retention: half-split pairs only")
@@ -1328,11 +1332,22 @@ class KernelLibrary:
         o = None
         if not self.lib.srlm_retention_walk_finishes(C.c_int(dv)):
             o = ctx.workspace.get("retention.o", T, H * dv, torch.float32)
-        self._check(self.lib.srlm_retention_walk(
-            _ptr(proj), C.c_longlong(proj.stride(0)), _ptr(rotation.cos if pairs else None),
-            _ptr(rotation.sin if pairs else None), C.c_int(pairs), _ptr(decay), C.c_float(eps), _ptr(state),
-            C.c_longlong(state.stride(0)), _ptr(ctx.cu_q), _ptr(ctx.slots), _ptr(o), _ptr(out), dtype_code(out.dtype),
-            C.c_int(ctx.n_entries), C.c_int(H), C.c_int(d), C.c_int(dv), _stream()), "retention_walk")
+        head = (_ptr(proj), C.c_longlong(proj.stride(0)), _ptr(rotation.cos if pairs else None),
+                _ptr(rotation.sin if pairs else None), C.c_int(pairs), _ptr(decay), C.c_float(eps), _ptr(state),
+                C.c_longlong(state.stride(0)), _ptr(ctx.cu_q), _ptr(ctx.slots))
+        tail = (_ptr(o), _ptr(out), dtype_code(out.dtype), C.c_int(ctx.n_entries), C.c_int(H), C.c_int(d), C.c_int(dv))
+        walk_max = 1 << 30
+        if (self.retention_in_chunks and ctx.max_q_len > self.RETENTION_WALK
+                and self.lib.srlm_retention_chunks_take(C.c_int(d), C.c_int(dv))):
+            walk_max = self.RETENTION_WALK
+            per = int(self.lib.srlm_retention_chunk_tokens())
+            chunks = sum(-(-n // per) for n in ctx.host["q_lens"] if n > walk_max)
+            U = ctx.workspace.get("retention.chunks", chunks * H, d * dv, torch.float32, reserve=0)
+            self._check(self.lib.srlm_retention_in_chunks(*head, _ptr(U), *tail, C.c_int(walk_max), C.c_int(chunks), _stream()),
+                        "retention_in_chunks")
+            self.launches += 2           # the fold along the chunks, the read-outs
+        if walk_max > ctx.max_q_len or min(ctx.host["q_lens"]) <= walk_max:
+            self._check(self.lib.srlm_retention_walk(*head, *tail, C.c_int(walk_max), _stream()), "retention_walk")
         if o is not None:
             self._retention_output(o, eps, proj, 2 * H * d + H * dv, out, H, dv)
 
