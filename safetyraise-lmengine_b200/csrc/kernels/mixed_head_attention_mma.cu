@@ -40,14 +40,42 @@ struct MixTiles {
   __device__ __forceinline__ int key(int n, int width) const { return (n < kept ? n : base + n - kept) * width; }
 };
 
+// 2^x by the hardware's approximation (two units in the last place; results below 2^-126 become 0).
+__device__ __forceinline__ float pow2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// Pages of keys or values: the row of key j for KV head h is row(j) + h * size.  shift: log2 of the page size, or -1.
+struct MixPages {
+  const int* table;
+  int nkv, size, shift;
+  __device__ __forceinline__ int row(int j) const {
+    const int page = shift >= 0 ? j >> shift : j / size;
+    return __ldg(table + page) * nkv * size + (j - page * size);
+  }
+};
+
+// A thread's share of a copy of rows of `vec` 16-byte pieces: piece c of rows r, r + step, ...
+struct MixCopy {
+  int r, c, step;
+  __device__ __forceinline__ MixCopy(int vec, int threads) {
+    step = threads / vec;
+    r = (int)threadIdx.x / vec;
+    c = (int)threadIdx.x - r * vec;
+    if (r >= step) r = 1 << 30;               // threads left over copy nothing
+  }
+};
+
 // ---- the softmax's sums -------------------------------------------------------------------------------------------
 constexpr int kLseRows = 64, kLseKeys = 64;
 
 __global__ void __launch_bounds__(128)
 mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache, float* __restrict__ lse,
                       const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_q,
-                      const int* __restrict__ kv_lens, int nq, int nkv, int dk, int page_size, float scale2, MixMask mask,
-                      DistanceBias bias, int span) {
+                      const int* __restrict__ kv_lens, int nq, int nkv, int dk, int page_size, int page_shift, float scale2,
+                      MixMask mask, DistanceBias bias, int span) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -60,13 +88,13 @@ mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
   bf16* k_s = q_s + kLseRows * ks;                             // [2][64][dk + 8]
   float* bias_s = reinterpret_cast<float*>(k_s + 2 * kLseKeys * ks);    // [2][G][span]
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int* table = block_table + (size_t)e * table_stride;
-  const int kvec = dk / 8;
-  for (int idx = tid; idx < kLseRows * kvec; idx += blockDim.x) {
-    const int r = idx / kvec, c = idx - r * kvec, row = r0 + r;
+  const MixPages pages{block_table + (size_t)e * table_stride, nkv, page_size, page_shift};
+  const MixCopy copy(dk / 8, 128);
+  for (int x = copy.r; x < kLseRows; x += copy.step) {
+    const int row = r0 + x;
     const bool there = row < rows;
-    const bf16* src = there ? q + ((size_t)(t0 + row / G) * nq + kvh * G + row % G) * dk + c * 8 : q;
-    cp_async_16(q_s + r * ks + c * 8, src, there);
+    const bf16* src = there ? q + ((size_t)(t0 + row / G) * nq + kvh * G + row % G) * dk + copy.c * 8 : q;
+    cp_async_16(q_s + x * ks + copy.c * 8, src, there);
   }
   float m[2], l[2];
   int pos[2], head[2];
@@ -83,20 +111,20 @@ mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
   const int first_seen = mask.first_key(min_pos);
   const MixTiles tiles(mask, min_pos, max_pos, kLseKeys);
   auto fetch = [&](int jb, int buf) {
-    for (int idx = tid; idx < kLseKeys * kvec; idx += blockDim.x) {
-      const int jj = idx / kvec, c = idx - jj * kvec, j = jb + jj;
+#pragma unroll 4
+    for (int jj = copy.r; jj < kLseKeys; jj += copy.step) {
+      const int j = jb + jj;
       const bool there = j <= max_pos && (j >= first_seen || j < mask.keep);
-      const size_t row = there ? ((size_t)table[j / page_size] * nkv + kvh) * page_size + (j % page_size) : 0;
-      cp_async_16(k_s + (buf * kLseKeys + jj) * ks + c * 8, k_cache + row * dk + c * 8, there);
+      const size_t row = there ? pages.row(j) + kvh * page_size : 0;
+      cp_async_16(k_s + (buf * kLseKeys + jj) * ks + copy.c * 8, k_cache + row * dk + copy.c * 8, there);
     }
     cp_async_commit();
     if (bias.table) {
       // bias_s[h][x] belongs to distance min_pos - (jb + 63) + x
       const int d0 = min_pos - jb - (kLseKeys - 1);
-      for (int idx = tid; idx < G * span; idx += blockDim.x) {
-        const int h = idx / span, d = d0 + idx - h * span;
-        bias_s[(size_t)buf * G * span + idx] = bias.at(kvh * G + h, max(d, 0)) * kLog2e;
-      }
+      for (int h = warp; h < G; h += 4)
+        for (int x = lane; x < span; x += 32)
+          bias_s[(size_t)(buf * G + h) * span + x] = bias.at(kvh * G + h, max(d0 + x, 0)) * kLog2e;
     }
   };
   fetch(tiles.key(0, kLseKeys), 0);
@@ -131,26 +159,41 @@ mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
     const bool whole = jb + kLseKeys - 1 <= min_pos && (mask.window <= 0 || jb > max_pos - mask.window) && r0 + kLseRows <= rows;
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
-      const float* bs = bias_s + (size_t)buf * G * span + head[i] * span + (pos[i] - min_pos) + (kLseKeys - 1);
+      if (bias.table) {
+        const float* bs = bias_s + (size_t)(buf * G + head[i]) * span + max(pos[i] - min_pos, 0) + (kLseKeys - 1) - (lane & 3) * 2;
+#pragma unroll
+        for (int x = 0; x < 8; ++x) {
+          s[x][2 * i] = fmaf(s[x][2 * i], scale2, bs[-x * 8]);
+          s[x][2 * i + 1] = fmaf(s[x][2 * i + 1], scale2, bs[-x * 8 - 1]);
+        }
+      } else {
+#pragma unroll
+        for (int x = 0; x < 8; ++x) {
+          s[x][2 * i] *= scale2;
+          s[x][2 * i + 1] *= scale2;
+        }
+      }
+      if (!whole) {
+#pragma unroll
+        for (int x = 0; x < 8; ++x)
+#pragma unroll
+          for (int c = 0; c < 2; ++c)
+            if (!mask.visible(pos[i], jb + x * 8 + (lane & 3) * 2 + c)) s[x][2 * i + c] = -CUDART_INF_F;
+      }
       float mx = -CUDART_INF_F;
 #pragma unroll
-      for (int x = 0; x < 8; ++x)
-#pragma unroll
-        for (int c = 0; c < 2; ++c) {
-          const int jj = x * 8 + (lane & 3) * 2 + c;
-          float v = -CUDART_INF_F;
-          if (whole || mask.visible(pos[i], jb + jj)) v = fmaf(s[x][2 * i + c], scale2, bias.table ? bs[-jj] : 0.f);
-          s[x][2 * i + c] = v;
-          mx = fmaxf(mx, v);
-        }
+      for (int x = 0; x < 8; ++x) mx = fmaxf(mx, fmaxf(s[x][2 * i], s[x][2 * i + 1]));
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
       const float m_new = fmaxf(m[i], mx);
       if (m_new != -CUDART_INF_F) {
-        float sum = 0.f;
+        float sum[2] = {0.f, 0.f};
 #pragma unroll
-        for (int x = 0; x < 8; ++x) sum += exp2f(s[x][2 * i] - m_new) + exp2f(s[x][2 * i + 1] - m_new);
-        l[i] = l[i] * exp2f(m[i] - m_new) + sum;               // the lane's own share of the row's sum
+        for (int x = 0; x < 8; ++x) {
+          sum[0] += pow2(s[x][2 * i] - m_new);
+          sum[1] += pow2(s[x][2 * i + 1] - m_new);
+        }
+        l[i] = l[i] * pow2(m[i] - m_new) + sum[0] + sum[1];    // the lane's own share of the row's sum
         m[i] = m_new;
       }
     }
@@ -175,7 +218,7 @@ mixed_head_attention_mma_kernel(const bf16* __restrict__ q, const bf16* __restri
                                 const bf16* __restrict__ v_cache, const float* __restrict__ lse, bf16* __restrict__ out,
                                 const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_q,
                                 const int* __restrict__ kv_lens, int nq, int nkv, int dk, int dv, int slab, int page_size,
-                                float scale2, MixMask mask, DistanceBias bias, const float* __restrict__ mix, int mix_low,
+                                int page_shift, float scale2, MixMask mask, DistanceBias bias, const float* __restrict__ mix, int mix_low,
                                 ElementGate gate, int nsplit, float* __restrict__ part) {
   pdl_wait();
   pdl_trigger();
@@ -197,32 +240,26 @@ mixed_head_attention_mma_kernel(const bf16* __restrict__ q, const bf16* __restri
   bf16* mix_s = p_lo + HP * RS;                                // [2][HP][HP + 8]
   float* bias_s = reinterpret_cast<float*>(mix_s + 2 * HP * (HP + kMhPad));   // [nq][BL]
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, warps = blockDim.x >> 5;
-  const int* table = block_table + (size_t)e * table_stride;
+  const MixPages pages{block_table + (size_t)e * table_stride, nkv, page_size, page_shift};
   const int min_pos = start + i0, max_pos = start + min(q_len, i0 + R) - 1;
   const int first_seen = mask.first_key(min_pos);
   const MixTiles tiles(mask, min_pos, max_pos, kMhKeys);
   const int per = (tiles.count + nsplit - 1) / nsplit;
   const int n_first = split * per, n_last = min(tiles.count, n_first + per);
-  const int kvec = dk / 8, vvec = width / 8;
+  const MixCopy k_copy(dk / 8, blockDim.x), v_copy(width / 8, blockDim.x);
 
-  auto fetch_k = [&](int jb) {
-    for (int idx = tid; idx < nkv * kMhKeys * kvec; idx += blockDim.x) {
-      const int row = idx / kvec, c = idx - row * kvec, h = row / kMhKeys, j = jb + row % kMhKeys;
+  auto fetch = [&](int jb, const MixCopy& copy, bf16* dst, int stride, const bf16* pool, int dim) {
+#pragma unroll 4
+    for (int row = copy.r; row < nkv * kMhKeys; row += copy.step) {
+      const int h = row / kMhKeys, j = jb + row % kMhKeys;
       const bool there = j <= max_pos && (j >= first_seen || j < mask.keep);
-      const size_t at = there ? ((size_t)table[j / page_size] * nkv + h) * page_size + (j % page_size) : 0;
-      cp_async_16(k_s + row * ks + c * 8, k_cache + at * dk + c * 8, there);
+      const size_t at = there ? pages.row(j) + h * page_size : 0;
+      cp_async_16(dst + row * stride + copy.c * 8, pool + at * dim + copy.c * 8, there);
     }
     cp_async_commit();
   };
-  auto fetch_v = [&](int jb) {
-    for (int idx = tid; idx < nkv * kMhKeys * vvec; idx += blockDim.x) {
-      const int row = idx / vvec, c = idx - row * vvec, h = row / kMhKeys, j = jb + row % kMhKeys;
-      const bool there = j <= max_pos && (j >= first_seen || j < mask.keep);
-      const size_t at = there ? ((size_t)table[j / page_size] * nkv + h) * page_size + (j % page_size) : 0;
-      cp_async_16(v_s + row * vs + c * 8, v_cache + at * dv + c0 + c * 8, there);
-    }
-    cp_async_commit();
-  };
+  auto fetch_k = [&](int jb) { fetch(jb, k_copy, k_s, ks, k_cache, dk); };
+  auto fetch_v = [&](int jb) { fetch(jb, v_copy, v_s, vs, v_cache + c0, dv); };
   if (n_first < n_last) fetch_k(tiles.key(n_first, kMhKeys));
 
   // the mixture's matrix as a pair of bfloat16 (the rounding, and what it leaves), and zero rows for heads that do not exist
@@ -249,7 +286,7 @@ mixed_head_attention_mma_kernel(const bf16* __restrict__ q, const bf16* __restri
     const bool live = i0 + tok < q_len;
     pos[i] = live ? min_pos + tok : -1;
     at[i] = h * RS + tok * kMhRow;
-    bias_at[i] = h * BL + tok + kMhKeys - 1;
+    bias_at[i] = h * BL + tok + kMhKeys - 1 - (lane & 3) * 2;
     L[i] = live ? lse[(size_t)(t0 + i0 + tok) * nq + h] : 0.f;
     const bf16* src = q + ((size_t)(t0 + i0 + (live ? tok : 0)) * nq + h) * dk + (lane & 3) * 2;
 #pragma unroll
@@ -269,10 +306,12 @@ mixed_head_attention_mma_kernel(const bf16* __restrict__ q, const bf16* __restri
     const int jb = tiles.key(n, kMhKeys);
     if (bias.table) {                                          // bias_s[h][x]: distance min_pos - (jb + 31) + x
       const int d0 = min_pos - jb - (kMhKeys - 1);
-      for (int idx = tid; idx < nq * BL; idx += blockDim.x) {
-        const int h = idx / BL, d = d0 + idx - h * BL;
-        bias_s[idx] = bias.at(h, max(d, 0)) * kLog2e;
-      }
+#pragma unroll
+      for (int i = 0; i < HT; ++i)
+#pragma unroll
+        for (int x = 0; x < (BL + 31) / 32; ++x)
+          if (x * 32 + lane < BL)
+            bias_s[(head0 + i) * BL + x * 32 + lane] = bias.at(head0 + i, max(d0 + x * 32 + lane, 0)) * kLog2e;
     }
     cp_async_wait<0>();
     __syncthreads();                                           // the keys are here; the values and weights before are read
@@ -298,28 +337,44 @@ mixed_head_attention_mma_kernel(const bf16* __restrict__ q, const bf16* __restri
     }
     const bool whole = jb + kMhKeys - 1 <= min_pos && (mask.window <= 0 || jb > max_pos - mask.window) && i0 + R <= q_len;
 #pragma unroll
-    for (int i = 0; i < 2; ++i)
+    for (int i = 0; i < 2; ++i) {
+      if (bias.table) {
+        const float* bs = bias_s + bias_at[i];
+#pragma unroll
+        for (int x = 0; x < kMhKeys / 8; ++x) {
+          s[x][2 * i] = pow2(fmaf(s[x][2 * i], scale2, bs[-x * 8] - L[i]));
+          s[x][2 * i + 1] = pow2(fmaf(s[x][2 * i + 1], scale2, bs[-x * 8 - 1] - L[i]));
+        }
+      } else {
+#pragma unroll
+        for (int x = 0; x < kMhKeys / 8; ++x) {
+          s[x][2 * i] = pow2(fmaf(s[x][2 * i], scale2, -L[i]));
+          s[x][2 * i + 1] = pow2(fmaf(s[x][2 * i + 1], scale2, -L[i]));
+        }
+      }
+      if (!whole) {
+#pragma unroll
+        for (int x = 0; x < kMhKeys / 8; ++x)
+#pragma unroll
+          for (int c = 0; c < 2; ++c)
+            if (!mask.visible(pos[i], jb + x * 8 + (lane & 3) * 2 + c)) s[x][2 * i + c] = 0.f;
+      }
 #pragma unroll
       for (int x = 0; x < kMhKeys / 8; ++x) {
-        float p[2];
-#pragma unroll
-        for (int c = 0; c < 2; ++c) {
-          const int jj = x * 8 + (lane & 3) * 2 + c;
-          p[c] = 0.f;
-          if (whole || mask.visible(pos[i], jb + jj))
-            p[c] = exp2f(fmaf(s[x][2 * i + c], scale2, (bias.table ? bias_s[bias_at[i] - jj] : 0.f) - L[i]));
-        }
-        const __nv_bfloat162 hi = __floats2bfloat162_rn(p[0], p[1]);
+        const __nv_bfloat162 hi = __floats2bfloat162_rn(s[x][2 * i], s[x][2 * i + 1]);
         const float2 back = __bfloat1622float2(hi);
-        const __nv_bfloat162 lo = __floats2bfloat162_rn(p[0] - back.x, p[1] - back.y);
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(s[x][2 * i] - back.x, s[x][2 * i + 1] - back.y);
         const int to = at[i] + x * 8 + (lane & 3) * 2;
         *reinterpret_cast<__nv_bfloat162*>(p_hi + to) = hi;
         *reinterpret_cast<__nv_bfloat162*>(p_lo + to) = lo;
       }
+    }
     __syncthreads();                                           // all heads' weights are written; the keys are read
     if (n + 1 < n_last) fetch_k(tiles.key(n + 1, kMhKeys));
 
     // the mixture, in place: a warp takes 8 keys of a token at a time, all heads
+    uint32_t mix_f[4];                                         // one tile of heads: its matrix is loaded once
+    if (HT == 1) ldmatrix_x4(mix_f, mix_s + (lane & 15) * (HP + kMhPad) + (lane >> 4) * 8);
     for (int ct = warp; ct < R * (kMhKeys / 8); ct += warps) {
       const int col = (ct / (kMhKeys / 8)) * kMhRow + (ct % (kMhKeys / 8)) * 8;
       uint32_t b[HT][4];
@@ -332,7 +387,8 @@ mixed_head_attention_mma_kernel(const bf16* __restrict__ q, const bf16* __restri
 #pragma unroll
         for (int k = 0; k < HT; ++k) {
           uint32_t a[4];
-          ldmatrix_x4(a, mix_s + (mt * 16 + (lane & 15)) * (HP + kMhPad) + k * 16 + (lane >> 4) * 8);
+          if (HT == 1) { a[0] = mix_f[0]; a[1] = mix_f[1]; a[2] = mix_f[2]; a[3] = mix_f[3]; }
+          else ldmatrix_x4(a, mix_s + (mt * 16 + (lane & 15)) * (HP + kMhPad) + k * 16 + (lane >> 4) * 8);
           mma_bf16(d, a, b[k][2], b[k][3]);
           mma_bf16(d, a, b[k][0], b[k][1]);
           if (mix_low) {
@@ -440,7 +496,7 @@ mixed_head_attention_decode_kernel(const bf16* __restrict__ q, const bf16* __res
                                    const bf16* __restrict__ v_cache, bf16* __restrict__ out,
                                    const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_q,
                                    const int* __restrict__ kv_lens, int nq, int nkv, int row_tiles, int dk, int dv,
-                                   int page_size, float scale2, MixMask mask, DistanceBias bias,
+                                   int page_size, int page_shift, float scale2, MixMask mask, DistanceBias bias,
                                    const float* __restrict__ mix, ElementGate gate, int tiles_cap, int nbuf) {
   pdl_wait();
   pdl_trigger();
@@ -457,25 +513,28 @@ mixed_head_attention_decode_kernel(const bf16* __restrict__ q, const bf16* __res
   const int G = nq / nkv, rows_c = row_tiles * 16, ks = dk + kMhPad, vs = dv + kMhPad;
   const int t = cu_q[e], pos = kv_lens[e] - 1;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int* table = block_table + (size_t)e * table_stride;
+  const MixPages pages{block_table + (size_t)e * table_stride, nkv, page_size, page_shift};
   const MixTiles tiles(mask, pos, pos, kMhKeys);
   int per = (tiles.count + cluster - 1) / cluster;             // (never above tiles_cap: the host planned for the longest)
   if (per > tiles_cap) per = tiles_cap;
   const int n0 = min(tiles.count, rank * per), n_here = min(tiles.count - n0, per);
-  const int kvec = dk / 8, vvec = dv / 8;
+  const int kvec = dk / 8;
+  const MixCopy k_copy(dk / 8, kMdThreads), v_copy(dv / 8, kMdThreads);
 
   // stage x: 0 .. n_here - 1 fetch keys, n_here .. 2 n_here - 1 values, buffer x % nbuf
   auto fetch = [&](int x) {
     const bool values = x >= n_here;
     const int jb = tiles.key(n0 + (values ? x - n_here : x), kMhKeys);
     bf16* dst = reinterpret_cast<bf16*>(smem_raw + at.tile + (x % nbuf) * at.tile_bytes);
-    const int vec = values ? vvec : kvec, stride = values ? vs : ks, dim = values ? dv : dk;
+    const MixCopy& copy = values ? v_copy : k_copy;
+    const int stride = values ? vs : ks, dim = values ? dv : dk;
     const bf16* pool = values ? v_cache : k_cache;
-    for (int idx = tid; idx < nkv * kMhKeys * vec; idx += blockDim.x) {
-      const int row = idx / vec, c = idx - row * vec, h = row / kMhKeys, j = jb + row % kMhKeys;
+#pragma unroll 4
+    for (int row = copy.r; row < nkv * kMhKeys; row += copy.step) {
+      const int h = row / kMhKeys, j = jb + row % kMhKeys;
       const bool there = mask.visible(pos, j);
-      const size_t src = there ? ((size_t)table[j / page_size] * nkv + h) * page_size + (j % page_size) : 0;
-      cp_async_16(dst + row * stride + c * 8, pool + src * dim + c * 8, there);
+      const size_t src = there ? pages.row(j) + h * page_size : 0;
+      cp_async_16(dst + row * stride + copy.c * 8, pool + src * dim + copy.c * 8, there);
     }
     cp_async_commit();
   };
@@ -547,7 +606,7 @@ mixed_head_attention_decode_kernel(const bf16* __restrict__ q, const bf16* __res
           for (int j = lane; j < n_here * kMhKeys; j += 32) m = fmaxf(m, s_s[(size_t)h * at.keys + j]);
           m = warp_max(m);
           if (m != -CUDART_INF_F)
-            for (int j = lane; j < n_here * kMhKeys; j += 32) l += exp2f(s_s[(size_t)h * at.keys + j] - m);
+            for (int j = lane; j < n_here * kMhKeys; j += 32) l += pow2(s_s[(size_t)h * at.keys + j] - m);
           l = warp_sum(l);
           if (lane == 0) { stats[2 * h] = m; stats[2 * h + 1] = l; }
         }
@@ -560,13 +619,13 @@ mixed_head_attention_decode_kernel(const bf16* __restrict__ q, const bf16* __res
         for (int r = 0; r < cluster; ++r) m = fmaxf(m, mh_remote(stats + 2 * h, r));
         for (int r = 0; r < cluster; ++r) {
           const float mr = mh_remote(stats + 2 * h, r);
-          if (mr != -CUDART_INF_F) l += mh_remote(stats + 2 * h + 1, r) * exp2f(mr - m);
+          if (mr != -CUDART_INF_F) l += mh_remote(stats + 2 * h + 1, r) * pow2(mr - m);
         }
         lse[h] = m + log2f(l);
       }
       __syncthreads();
       for (int h = warp; h < nq; h += kMdWarps)
-        for (int j = lane; j < n_here * kMhKeys; j += 32) s_s[(size_t)h * at.keys + j] = exp2f(s_s[(size_t)h * at.keys + j] - lse[h]);
+        for (int j = lane; j < n_here * kMhKeys; j += 32) s_s[(size_t)h * at.keys + j] = pow2(s_s[(size_t)h * at.keys + j] - lse[h]);
     }
     if (x >= n_here) {
       const int j0 = (x - n_here) * kMhKeys;
@@ -645,6 +704,11 @@ static int mh_heads_tiles(int nq, int nkv) {      // 16-head tiles of the rows f
   if (nq <= 32 && nq % 2 == 0 && (nq / nkv) % 2 == 0) return 2;
   return 0;
 }
+static int mh_page_shift(int page_size) {
+  int s = 0;
+  while ((1 << s) < page_size) ++s;
+  return (1 << s) == page_size ? s : -1;
+}
 static int mh_slab(int dv) { return dv <= 128 ? dv : 128; }
 static size_t mh_rows_smem(int nq, int nkv, int dk, int dv) {
   const int ht = mh_heads_tiles(nq, nkv), hp = 16 * ht, R = 16 / ht, rs = R * kMhRow + kMhPad, slab = mh_slab(dv);
@@ -692,7 +756,7 @@ extern "C" int srlm_mixed_head_attention_mma(const void* q, const void* k_cache,
     if (smem > 48 * 1024) cudaFuncSetAttribute(mixed_head_lse_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     launch_pdl(mixed_head_lse_kernel, dim3((unsigned)(((long long)max_q_len * G + kLseRows - 1) / kLseRows), nkv, n_entries), dim3(128),
                smem, stream, (const bf16*)q, (const bf16*)k_cache, lse, block_table, table_stride, cu_q, kv_lens, nq, nkv, dk,
-               page_size, scale2, mask, db, mh_lse_span(G));
+               page_size, mh_page_shift(page_size), scale2, mask, db, mh_lse_span(G));
   }
   const size_t smem = mh_rows_smem(nq, nkv, dk, dv);
   const dim3 grid((unsigned)((max_q_len + R - 1) / R), (unsigned)(slabs * nsplit), (unsigned)n_entries);
@@ -702,7 +766,7 @@ extern "C" int srlm_mixed_head_attention_mma(const void* q, const void* k_cache,
     auto kern = mixed_head_attention_mma_kernel<KS, NT, HT>;                                                            \
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);           \
     launch_pdl(kern, grid, dim3(threads), smem, stream, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, lse, \
-               (bf16*)out, block_table, table_stride, cu_q, kv_lens, nq, nkv, dk, dv, slab, page_size, scale2, mask, db, \
+               (bf16*)out, block_table, table_stride, cu_q, kv_lens, nq, nkv, dk, dv, slab, page_size, mh_page_shift(page_size), scale2, mask, db, \
                mix, mix_low, gate, nsplit, part);                                                                       \
   } while (0)
 #define SRLM_MH_SIZES(HT)                               \
@@ -768,7 +832,7 @@ extern "C" int srlm_mixed_head_attention_decode(const void* q, const void* k_cac
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);              \
     if (cluster > 8) cudaFuncSetAttribute(kern, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);                   \
     cudaLaunchKernelEx(&cfg, kern, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, (bf16*)out, block_table, \
-                       table_stride, cu_q, kv_lens, nq, nkv, row_tiles, dk, dv, page_size, scale * kLog2e, mask, db, mix, \
+                       table_stride, cu_q, kv_lens, nq, nkv, row_tiles, dk, dv, page_size, mh_page_shift(page_size), scale * kLog2e, mask, db, mix, \
                        gate, tiles_here, nbuf);                                                                       \
   } while (0)
   if (units <= 2 * kMdWarps) SRLM_MD(2);

@@ -170,12 +170,65 @@ __device__ __forceinline__ ChunkHome chunk_home(const int* __restrict__ cu_q, in
   return ChunkHome{-1, 0, 0, 0};
 }
 
-// An element of a rotated head: x its projected elements, cs and sn the token's angles.
-__device__ __forceinline__ float rotated(const float* __restrict__ x, int i, const float* __restrict__ cs,
-                                         const float* __restrict__ sn, int pairs) {
-  const float own = x[i];
-  if (i >= 2 * pairs) return own;
-  return i < pairs ? own * cs[i] - x[i + pairs] * sn[i] : own * cs[i - pairs] + x[i - pairs] * sn[i - pairs];
+__device__ __forceinline__ void ret_copy_16(float* dst, const float* src) {
+  const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src));
+}
+__device__ __forceinline__ void ret_copy_4(float* dst, const float* src) {
+  const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(d), "l"(src));
+}
+__device__ __forceinline__ void ret_commit() { asm volatile("cp.async.commit_group;" ::); }
+template <int N> __device__ __forceinline__ void ret_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N)); }
+
+// dst[x][c] (row stride `stride`, a multiple of 4) = src[x * ld + c] for x < n and c < width, zeros up to `rows` rows and
+// `padded` columns; asynchronous, in 16-byte pieces when `vec` says that every row of src starts on 16 bytes and width and
+// padded are multiples of 4.
+__device__ __forceinline__ void ret_copy_rows(float* dst, int stride, const float* src, long long ld, int n, int rows, int width,
+                                              int padded, bool vec) {
+  if (vec) {
+    const int pieces = padded / 4, step = (int)blockDim.x / pieces, c = ((int)threadIdx.x % pieces) * 4;
+    if (step == 0) {                                   // rows of more pieces than the block has threads
+      for (int idx = threadIdx.x; idx < rows * pieces; idx += blockDim.x) {
+        const int x = idx / pieces, cc = (idx - x * pieces) * 4;
+        if (x < n && cc < width) ret_copy_16(dst + x * stride + cc, src + (size_t)x * ld + cc);
+        else *reinterpret_cast<float4*>(dst + x * stride + cc) = make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+      return;
+    }
+    if ((int)threadIdx.x >= step * pieces) return;
+#pragma unroll 4
+    for (int x = (int)threadIdx.x / pieces; x < rows; x += step) {
+      if (x < n && c < width) ret_copy_16(dst + x * stride + c, src + (size_t)x * ld + c);
+      else *reinterpret_cast<float4*>(dst + x * stride + c) = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  } else {
+    for (int idx = threadIdx.x; idx < rows * padded; idx += blockDim.x) {
+      const int x = idx / padded, c = idx - x * padded;
+      if (x < n && c < width) ret_copy_4(dst + x * stride + c, src + (size_t)x * ld + c);
+      else dst[x * stride + c] = 0.f;
+    }
+  }
+}
+
+// Turns the leading 2 pairs elements of rows of shared memory: row x by the angles of token t0 + x; then multiplies the
+// whole row by scale[x] (null: leaves it).
+__device__ __forceinline__ void ret_rotate_rows(float* rows_s, int stride, int n, int d, const float* __restrict__ cos_t,
+                                                const float* __restrict__ sin_t, int t0, int pairs, const float* scale) {
+  if (pairs) {
+#pragma unroll 4
+    for (int idx = threadIdx.x; idx < n * pairs; idx += blockDim.x) {
+      const int x = idx / pairs, i = idx - x * pairs;
+      const float c = __ldg(cos_t + (size_t)t0 * pairs + idx), sn = __ldg(sin_t + (size_t)t0 * pairs + idx);
+      float* row = rows_s + x * stride;
+      const float u = row[i], v = row[i + pairs], f = scale ? scale[x] : 1.f;
+      row[i] = (u * c - v * sn) * f;
+      row[i + pairs] = (v * c + u * sn) * f;
+    }
+  }
+  const int rest = d - 2 * pairs;
+  if (scale && rest > 0)
+    for (int idx = threadIdx.x; idx < n * rest; idx += blockDim.x) rows_s[(idx / rest) * stride + 2 * pairs + idx % rest] *= scale[idx / rest];
 }
 
 // U of a chunk and head: a tile of 16 TM rows (of d) x 16 TN columns (of dv) a block, TM x TN of it a thread.
@@ -183,67 +236,72 @@ template <int TM, int TN>
 __global__ void __launch_bounds__(256)
 retention_chunks_kernel(const float* __restrict__ proj, long long ldp, const float* __restrict__ cos_t,
                         const float* __restrict__ sin_t, int pairs, const float* __restrict__ decay,
-                        const int* __restrict__ cu_q, int n_entries, int walk_max, float* __restrict__ U, int H, int d, int dv) {
+                        const int* __restrict__ cu_q, int n_entries, int walk_max, float* __restrict__ U, int H, int d, int dv,
+                        int dp, int vec) {
   pdl_wait();
   pdl_trigger();
   constexpr int BM = 16 * TM, BN = 16 * TN;
   extern __shared__ __align__(16) float ret_chunk_smem[];
-  float* k_s = ret_chunk_smem;                       // [64][BM + 4]
-  float* v_s = k_s + kRetChunk * (BM + 4);           // [64][BN + 4]
+  const int ks = dp + 4;                             // dp: d rounded up to whole row tiles
+  float* k_s = ret_chunk_smem;                       // [64][dp + 4]
+  float* v_s = k_s + kRetChunk * ks;                 // [64][BN + 4]
   __shared__ float fade[kRetChunk];
-  const int h = blockIdx.y, col_tiles = (dv + BN - 1) / BN;
-  const int m0 = (blockIdx.z / col_tiles) * BM, c0 = (blockIdx.z % col_tiles) * BN;
+  const int h = blockIdx.y, c0 = blockIdx.z * BN;
   const ChunkHome home = chunk_home(cu_q, n_entries, walk_max, blockIdx.x);
   if (home.entry < 0) return;
   const int tid = threadIdx.x;
+  const float* first = proj + (size_t)home.t0 * ldp;
+  ret_copy_rows(k_s, ks, first + (size_t)(H + h) * d, ldp, home.n, kRetChunk, d, dp, vec);
+  ret_copy_rows(v_s, BN + 4, first + 2 * (size_t)H * d + (size_t)h * dv + c0, ldp, home.n, kRetChunk, min(BN, dv - c0), BN, vec);
+  ret_commit();
   if (tid < home.n) fade[tid] = decay_power(decay[h], home.n - 1 - tid) / sqrtf((float)d);
+  ret_wait<0>();
   __syncthreads();
-  for (int idx = tid; idx < kRetChunk * BM; idx += blockDim.x) {
-    const int s = idx / BM, i = idx - s * BM, t = home.t0 + s;
-    float v = 0.f;
-    if (s < home.n && m0 + i < d)
-      v = rotated(proj + (size_t)t * ldp + (size_t)(H + h) * d, m0 + i, cos_t + (size_t)t * pairs, sin_t + (size_t)t * pairs, pairs) * fade[s];
-    k_s[s * (BM + 4) + i] = v;
-  }
-  for (int idx = tid; idx < kRetChunk * BN; idx += blockDim.x) {
-    const int s = idx / BN, i = idx - s * BN;
-    v_s[s * (BN + 4) + i] = s < home.n && c0 + i < dv ? proj[(size_t)(home.t0 + s) * ldp + 2 * (size_t)H * d + (size_t)h * dv + c0 + i] : 0.f;
-  }
+  ret_rotate_rows(k_s, ks, home.n, d, cos_t, sin_t, home.t0, pairs, fade);
   __syncthreads();
-  const int tm = (tid / 16) * TM, tn = (tid % 16) * 2;        // a thread's columns: tn, tn + 1 of every 32
-  float2 acc[TM][TN / 2];
-#pragma unroll
-  for (int i = 0; i < TM; ++i)
-#pragma unroll
-    for (int j = 0; j < TN / 2; ++j) acc[i][j] = make_float2(0.f, 0.f);
-#pragma unroll 4
-  for (int s = 0; s < kRetChunk; ++s) {
-    float a[TM];
-    float2 b[TN / 2];
-#pragma unroll
-    for (int i = 0; i < TM; ++i) a[i] = k_s[s * (BM + 4) + tm + i];
-#pragma unroll
-    for (int j = 0; j < TN / 2; ++j) b[j] = *reinterpret_cast<const float2*>(v_s + s * (BN + 4) + tn + 32 * j);
+  const int tn = (tid % 16) * 2;                     // a thread's columns: tn, tn + 1 of every 32
+  float* dst = U + ((size_t)blockIdx.x * H + h) * d * dv;
+  for (int m0 = 0; m0 < d; m0 += BM) {
+    const int tm = m0 + (tid / 16) * TM;
+    float2 acc[TM][TN / 2];
 #pragma unroll
     for (int i = 0; i < TM; ++i)
 #pragma unroll
-      for (int j = 0; j < TN / 2; ++j) acc[i][j] = fma2(make_float2(a[i], a[i]), b[j], acc[i][j]);
-  }
-  float* dst = U + ((size_t)blockIdx.x * H + h) * d * dv;
+      for (int j = 0; j < TN / 2; ++j) acc[i][j] = make_float2(0.f, 0.f);
+#pragma unroll 4
+    for (int s = 0; s < kRetChunk; ++s) {
+      float a[TM];
+      float2 b[TN / 2];
 #pragma unroll
-  for (int i = 0; i < TM; ++i) {
-    const int r = m0 + tm + i;
-    if (r >= d) continue;
+      for (int i = 0; i < TM; ++i) a[i] = k_s[s * ks + tm + i];
 #pragma unroll
-    for (int j = 0; j < TN / 2; ++j) {
-      const int c = c0 + tn + 32 * j;
-      if (c < dv) dst[(size_t)r * dv + c] = acc[i][j].x;
-      if (c + 1 < dv) dst[(size_t)r * dv + c + 1] = acc[i][j].y;
+      for (int j = 0; j < TN / 2; ++j) b[j] = *reinterpret_cast<const float2*>(v_s + s * (BN + 4) + tn + 32 * j);
+#pragma unroll
+      for (int i = 0; i < TM; ++i)
+#pragma unroll
+        for (int j = 0; j < TN / 2; ++j) acc[i][j] = fma2(make_float2(a[i], a[i]), b[j], acc[i][j]);
+    }
+#pragma unroll
+    for (int i = 0; i < TM; ++i) {
+      const int r = tm + i;
+      if (r >= d) continue;
+#pragma unroll
+      for (int j = 0; j < TN / 2; ++j) {
+        const int c = c0 + tn + 32 * j;
+        if (vec) {
+          if (c < dv) *reinterpret_cast<float2*>(dst + (size_t)r * dv + c) = acc[i][j];
+        } else {
+          if (c < dv) dst[(size_t)r * dv + c] = acc[i][j].x;
+          if (c + 1 < dv) dst[(size_t)r * dv + c + 1] = acc[i][j].y;
+        }
+      }
     }
   }
 }
 
-// grid (elements of a state / 256, entries): S of the slot through the entry's chunks; U_c <- the state ahead of chunk c.
+// grid (elements of a state / (256 V), entries): S of the slot through the entry's chunks; U_c <- the state ahead of chunk
+// c.  V neighbouring elements a thread (4 when the rows of U and of the state allow 16-byte accesses).
+template <int V>
 __global__ void __launch_bounds__(256)
 retention_fold_kernel(float* __restrict__ U, const float* __restrict__ decay, float* __restrict__ state, long long state_stride,
                       const int* __restrict__ cu_q, const int* __restrict__ slots, int walk_max, int H, int d, int dv) {
@@ -257,134 +315,158 @@ retention_fold_kernel(float* __restrict__ U, const float* __restrict__ decay, fl
     const int l = cu_q[x + 1] - cu_q[x];
     if (l > walk_max) base += (l + kRetChunk - 1) / kRetChunk;
   }
-  const size_t per = (size_t)H * d * dv, i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  const size_t per = (size_t)H * d * dv, i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * V;
   if (i >= per) return;
   const int h = (int)(i / ((size_t)d * dv)), chunks = (len + kRetChunk - 1) / kRetChunk;
   const float whole = decay_power(decay[h], kRetChunk), rest = decay_power(decay[h], len - (chunks - 1) * kRetChunk);
   float* u = U + (size_t)base * per + i;
   float* slot = state + (size_t)slots[e] * state_stride + i;
-  float S = *slot;
+  auto get = [](const float* p, float (&v)[V]) {
+    if (V == 4) *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(p);
+    else v[0] = p[0];
+  };
+  auto put = [](float* p, const float (&v)[V]) {
+    if (V == 4) *reinterpret_cast<float4*>(p) = *reinterpret_cast<const float4*>(v);
+    else p[0] = v[0];
+  };
+  alignas(16) float S[V];
+  get(slot, S);
   constexpr int kAhead = 8;
   for (int c = 0; c < chunks; c += kAhead) {
-    float next[kAhead];
+    alignas(16) float next[kAhead][V];
 #pragma unroll
-    for (int x = 0; x < kAhead; ++x) next[x] = c + x < chunks ? u[(size_t)(c + x) * per] : 0.f;
+    for (int x = 0; x < kAhead; ++x)
+      if (c + x < chunks) get(u + (size_t)(c + x) * per, next[x]);
 #pragma unroll
     for (int x = 0; x < kAhead; ++x) {
       if (c + x < chunks) {
-        u[(size_t)(c + x) * per] = S;
-        S = fmaf(c + x + 1 < chunks ? whole : rest, S, next[x]);
+        put(u + (size_t)(c + x) * per, S);
+        const float f = c + x + 1 < chunks ? whole : rest;
+#pragma unroll
+        for (int y = 0; y < V; ++y) S[y] = fmaf(f, S[y], next[x][y]);
       }
     }
   }
-  *slot = S;
+  put(slot, S);
 }
 
 // A chunk of 64 tokens, one head, a tile of 16 TN value columns a block: thread (ty, tx) holds rows 4 ty .. 4 ty + 3 and
 // the column pairs 2 tx + 32 j.  Where one tile holds the head it norms and gates; else o_out.
+constexpr int kRetSlab = 16;                          // rows of the state that are multiplied at a time
+
 template <int TN, typename TO>
 __global__ void __launch_bounds__(256)
 retention_read_kernel(const float* __restrict__ proj, long long ldp, const float* __restrict__ cos_t,
                       const float* __restrict__ sin_t, int pairs, const float* __restrict__ decay, float eps,
                       const int* __restrict__ cu_q, int n_entries, int walk_max, const float* __restrict__ U,
-                      float* __restrict__ o_out, TO* __restrict__ out, int H, int d, int dv) {
+                      float* __restrict__ o_out, TO* __restrict__ out, int H, int d, int dv, int dp, int vec) {
   pdl_wait();
   pdl_trigger();
-  constexpr int BN = 16 * TN, TR = kRetChunk + 4;
+  constexpr int BN = 16 * TN, BS = BN + 4;
   extern __shared__ __align__(16) float ret_chunk_smem[];
-  float* q_t = ret_chunk_smem;                        // [d][68]: element, token
-  float* k_t = q_t + (size_t)d * TR;                  // [d][68], then slabs of S: [slab rows][BN + 4]
-  float* a_t = k_t + (size_t)d * TR;                  // [64][68]: (s, t): what token t takes of v_s
-  float* v_s = a_t + (size_t)kRetChunk * TR;          // [64][BN + 4]
+  const int qs = dp + 4;                              // dp: d rounded up to a multiple of 4 (zeros behind it)
+  float* q_s = ret_chunk_smem;                        // [64][dp + 4]
+  float* v_s = q_s + kRetChunk * qs;                  // [64][BN + 4]
+  float* k_s = v_s + kRetChunk * BS;                  // [64][dp + 4]; then a_t and two slabs of the state
+  float* a_t = k_s;                                   // [64][64]: (s, t): what token t takes of v_s
+  float* s_s = a_t + kRetChunk * kRetChunk;           // [2][16][BN + 4]
   __shared__ float pw[kRetChunk + 1];
-  const int h = blockIdx.y, c0 = blockIdx.z * BN;
+  const int h = blockIdx.y, c0 = blockIdx.z * BN, width = min(BN, dv - c0);
   const ChunkHome home = chunk_home(cu_q, n_entries, walk_max, blockIdx.x);
   if (home.entry < 0) return;
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int tid = threadIdx.x, warp = tid >> 5;
+  const float* first = proj + (size_t)home.t0 * ldp + (size_t)h * d;
+  ret_copy_rows(q_s, qs, first, ldp, home.n, kRetChunk, d, dp, vec);
+  ret_copy_rows(k_s, qs, first + (size_t)H * d, ldp, home.n, kRetChunk, d, dp, vec);
+  ret_commit();
+  ret_copy_rows(v_s, BS, proj + (size_t)home.t0 * ldp + 2 * (size_t)H * d + (size_t)h * dv + c0, ldp, home.n, kRetChunk, width, BN, vec);
+  ret_commit();
   if (tid <= kRetChunk) pw[tid] = decay_power(decay[h], tid);
-  const float k_scale = 1.f / sqrtf((float)d);
-  // q and k turned and transposed: a warp stores 8 elements x 4 tokens at a time, one bank each
-  const int dim_groups = (d + 7) / 8;
-  for (int job = warp; job < dim_groups * (kRetChunk / 4); job += 8) {
-    const int i = (job % dim_groups) * 8 + (lane & 7), s = (job / dim_groups) * 4 + (lane >> 3), t = home.t0 + s;
-    if (i < d) {
-      float q = 0.f, k = 0.f;
-      if (s < home.n) {
-        const float* x = proj + (size_t)t * ldp + (size_t)h * d;
-        q = rotated(x, i, cos_t + (size_t)t * pairs, sin_t + (size_t)t * pairs, pairs);
-        k = rotated(x + (size_t)H * d, i, cos_t + (size_t)t * pairs, sin_t + (size_t)t * pairs, pairs) * k_scale;
-      }
-      q_t[i * TR + s] = q;
-      k_t[i * TR + s] = k;
-    }
-  }
-  for (int idx = tid; idx < kRetChunk * BN; idx += blockDim.x) {
-    const int s = idx / BN, i = idx - s * BN;
-    v_s[s * (BN + 4) + i] = s < home.n && c0 + i < dv ? proj[(size_t)(home.t0 + s) * ldp + 2 * (size_t)H * d + (size_t)h * dv + c0 + i] : 0.f;
-  }
+  ret_wait<1>();
+  __syncthreads();
+  ret_rotate_rows(q_s, qs, home.n, d, cos_t, sin_t, home.t0, pairs, nullptr);
+  ret_rotate_rows(k_s, qs, home.n, d, cos_t, sin_t, home.t0, pairs, nullptr);
   __syncthreads();
 
   const int ty = tid / 16, tx = tid % 16, tm = ty * 4, tn = tx * 2;
+  const float k_scale = 1.f / sqrtf((float)d);
+  float dot[4][4];                                    // [t][s]: 4 tokens t = tm + i, 4 tokens s = tx + 16 j
   {
-    // a_t[s][t] = decay^(t - s) q_t . k_s: 4 tokens t x 4 tokens s a thread (s = tx + 16 j), nothing above the diagonal
-    float2 dot[4][2];                                 // [s][t pair]
+    float2 sum[4][4];                                 // even and odd elements apart
 #pragma unroll
-    for (int j = 0; j < 4; ++j) dot[j][0] = dot[j][1] = make_float2(0.f, 0.f);
-    for (int i = 0; i < d; ++i) {
-      const float4 a = *reinterpret_cast<const float4*>(q_t + i * TR + tm);
+    for (int i = 0; i < 4; ++i)
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const float b = k_t[i * TR + tx + 16 * j];
-        dot[j][0] = fma2(make_float2(b, b), make_float2(a.x, a.y), dot[j][0]);
-        dot[j][1] = fma2(make_float2(b, b), make_float2(a.z, a.w), dot[j][1]);
-      }
+      for (int j = 0; j < 4; ++j) sum[i][j] = make_float2(0.f, 0.f);
+#pragma unroll 2
+    for (int x = 0; x < dp; x += 4) {
+      float4 a[4], b[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) a[i] = *reinterpret_cast<const float4*>(q_s + (tm + i) * qs + x);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) b[j] = *reinterpret_cast<const float4*>(k_s + (tx + 16 * j) * qs + x);
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          sum[i][j] = fma2(make_float2(a[i].x, a[i].y), make_float2(b[j].x, b[j].y), sum[i][j]);
+          sum[i][j] = fma2(make_float2(a[i].z, a[i].w), make_float2(b[j].z, b[j].w), sum[i][j]);
+        }
     }
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int s = tx + 16 * j;
-      float4 v;
-      v.x = s <= tm ? dot[j][0].x * pw[tm - s] : 0.f;
-      v.y = s <= tm + 1 ? dot[j][0].y * pw[tm + 1 - s] : 0.f;
-      v.z = s <= tm + 2 ? dot[j][1].x * pw[tm + 2 - s] : 0.f;
-      v.w = s <= tm + 3 ? dot[j][1].y * pw[tm + 3 - s] : 0.f;
-      *reinterpret_cast<float4*>(a_t + s * TR + tm) = v;
-    }
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) dot[i][j] = (sum[i][j].x + sum[i][j].y) * k_scale;
   }
-  __syncthreads();                                    // a_t is written; k_t and the unscaled q_t are read
+  __syncthreads();                                    // k_s is read: a_t and the slabs take its place
+  const float* S = U + ((size_t)blockIdx.x * H + h) * d * dv + c0;
+  auto fetch = [&](int slab) {
+    const int r0 = slab * kRetSlab;
+    ret_copy_rows(s_s + (slab & 1) * kRetSlab * BS, BS, S + (size_t)r0 * dv, dv, min(kRetSlab, d - r0), kRetSlab, width, BN, vec);
+    ret_commit();
+  };
+  fetch(0);
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const int s = tx + 16 * j;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) dot[i][j] = s <= tm + i ? dot[i][j] * pw[max(tm + i - s, 0)] : 0.f;
+    *reinterpret_cast<float4*>(a_t + s * kRetChunk + tm) = make_float4(dot[0][j], dot[1][j], dot[2][j], dot[3][j]);
+  }
 
   float2 acc[4][TN / 2];
 #pragma unroll
   for (int i = 0; i < 4; ++i)
 #pragma unroll
     for (int j = 0; j < TN / 2; ++j) acc[i][j] = make_float2(0.f, 0.f);
-  // rows s of `left` (4 tokens of it a thread) times rows s of `right`
-  auto product = [&](const float* left, const float* right, int rows) {
-#pragma unroll 4
-    for (int s = 0; s < rows; ++s) {
-      const float4 a = *reinterpret_cast<const float4*>(left + s * TR + tm);
-      float2 b[TN / 2];
+  auto row_times = [&](float a0, float a1, float a2, float a3, const float* right) {
+    float2 b[TN / 2];
 #pragma unroll
-      for (int j = 0; j < TN / 2; ++j) b[j] = *reinterpret_cast<const float2*>(right + s * (BN + 4) + tn + 32 * j);
+    for (int j = 0; j < TN / 2; ++j) b[j] = *reinterpret_cast<const float2*>(right + tn + 32 * j);
 #pragma unroll
-      for (int j = 0; j < TN / 2; ++j) {
-        acc[0][j] = fma2(make_float2(a.x, a.x), b[j], acc[0][j]);
-        acc[1][j] = fma2(make_float2(a.y, a.y), b[j], acc[1][j]);
-        acc[2][j] = fma2(make_float2(a.z, a.z), b[j], acc[2][j]);
-        acc[3][j] = fma2(make_float2(a.w, a.w), b[j], acc[3][j]);
-      }
+    for (int j = 0; j < TN / 2; ++j) {
+      acc[0][j] = fma2(make_float2(a0, a0), b[j], acc[0][j]);
+      acc[1][j] = fma2(make_float2(a1, a1), b[j], acc[1][j]);
+      acc[2][j] = fma2(make_float2(a2, a2), b[j], acc[2][j]);
+      acc[3][j] = fma2(make_float2(a3, a3), b[j], acc[3][j]);
     }
   };
-  const float* S = U + ((size_t)blockIdx.x * H + h) * d * dv;
-  const int slab_rows = d * TR / (BN + 4) < d ? d * TR / (BN + 4) : d;
-  for (int r0 = 0; r0 < d; r0 += slab_rows) {
-    const int rows = min(slab_rows, d - r0);
-    if (r0) __syncthreads();
-    for (int idx = tid; idx < rows * BN; idx += blockDim.x) {
-      const int r = idx / BN, i = idx - r * BN;
-      k_t[r * (BN + 4) + i] = c0 + i < dv ? S[(size_t)(r0 + r) * dv + c0 + i] : 0.f;
+  const int slabs = (d + kRetSlab - 1) / kRetSlab;
+  for (int slab = 0; slab < slabs; ++slab) {
+    ret_wait<0>();
+    __syncthreads();                                  // the slab is here; the other one is read
+    if (slab + 1 < slabs) fetch(slab + 1);
+    const float* right = s_s + (slab & 1) * kRetSlab * BS;
+    const int r0 = slab * kRetSlab, rows = min(kRetSlab, dp - r0);
+#pragma unroll 2
+    for (int r = 0; r < rows; r += 4) {               // rows of the slab behind d are zeros, and so are q's elements there
+      float4 a[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) a[i] = *reinterpret_cast<const float4*>(q_s + (tm + i) * qs + r0 + r);
+      row_times(a[0].x, a[1].x, a[2].x, a[3].x, right + r * BS);
+      row_times(a[0].y, a[1].y, a[2].y, a[3].y, right + (r + 1) * BS);
+      row_times(a[0].z, a[1].z, a[2].z, a[3].z, right + (r + 2) * BS);
+      row_times(a[0].w, a[1].w, a[2].w, a[3].w, right + (r + 3) * BS);
     }
-    __syncthreads();
-    product(q_t + (size_t)r0 * TR, k_t, rows);
   }
 #pragma unroll
   for (int i = 0; i < 4; ++i)
@@ -393,7 +475,12 @@ retention_read_kernel(const float* __restrict__ proj, long long ldp, const float
       acc[i][j].x *= pw[tm + i + 1];
       acc[i][j].y *= pw[tm + i + 1];
     }
-  product(a_t, v_s, min(kRetChunk, (warp + 1) * 8));  // a warp's rows end at 8 warp + 7: no later s counts
+  const int s_end = (warp + 1) * 8;                   // a warp's rows end at 8 warp + 7: no later s counts
+#pragma unroll 4
+  for (int s = 0; s < s_end; ++s) {
+    const float4 a = *reinterpret_cast<const float4*>(a_t + s * kRetChunk + tm);
+    row_times(a.x, a.y, a.z, a.w, v_s + s * BS);
+  }
 
   // a row's columns lie with the 16 threads of its ty
 #pragma unroll
@@ -509,14 +596,18 @@ extern "C" int srlm_retention_output(const float* o, float eps, const float* pro
 }
 
 static size_t ret_read_smem(int d, int tn) {
-  const int tr = kRetChunk + 4;
-  return (2 * (size_t)d * tr + (size_t)kRetChunk * tr + (size_t)kRetChunk * (16 * tn + 4)) * sizeof(float);
+  const size_t qs = (d + 3) / 4 * 4 + 4, bs = 16 * tn + 4;
+  const size_t third = kRetChunk * kRetChunk + 2 * kRetSlab * bs;
+  return (kRetChunk * qs + kRetChunk * bs + (kRetChunk * qs > third ? kRetChunk * qs : third)) * sizeof(float);
 }
+static int ret_rows_padded(int d, int t) { return (d + 16 * t - 1) / (16 * t) * (16 * t); }
+static size_t ret_chunks_smem(int d, int t) { return (size_t)kRetChunk * (ret_rows_padded(d, t) + 4 + 16 * t + 4) * sizeof(float); }
 static int ret_tile(int n) { return n <= 32 ? 2 : n <= 64 ? 4 : 8; }
 
 // Whether entries may be taken in chunks: heads of up to 256 elements.
 extern "C" int srlm_retention_chunks_take(int d, int dv) {
-  return d > 0 && dv > 0 && d * (kRetChunk + 4) >= 16 * ret_tile(dv) + 4 && ret_read_smem(d, ret_tile(dv)) <= 220 * 1024;
+  const int tm = ret_tile(d), tn = ret_tile(dv);
+  return d > 0 && dv > 0 && d <= 256 && ret_read_smem(d, tn) <= 220 * 1024 && ret_chunks_smem(d, tm > tn ? tm : tn) <= 220 * 1024;
 }
 extern "C" int srlm_retention_chunk_tokens() { return kRetChunk; }
 
@@ -533,22 +624,29 @@ extern "C" int srlm_retention_in_chunks(const float* proj, long long ldp, const 
   const int tm = ret_tile(d), tn = ret_tile(dv), t = tm > tn ? tm : tn;
   const bool finishes = dv <= 128;
   if (finishes ? !out : !o_out) return refuse(ST_BAD_SIZE, "retention_in_chunks: no buffer for the result");
+  // 16-byte accesses: every row of the projection, of U and of the state starts on 16 bytes
+  const int vec = d % 4 == 0 && dv % 4 == 0 && ldp % 4 == 0 && state_stride % 4 == 0 &&
+                  (((uintptr_t)proj | (uintptr_t)U | (uintptr_t)state) & 15) == 0;
   {
-    const size_t smem = (size_t)kRetChunk * (2 * (16 * t + 4)) * sizeof(float);
-    const dim3 grid(chunks, H, ((d + 16 * t - 1) / (16 * t)) * ((dv + 16 * t - 1) / (16 * t)));
+    const size_t smem = ret_chunks_smem(d, t);
+    const dim3 grid(chunks, H, (dv + 16 * t - 1) / (16 * t));
 #define SRLM_CHUNKS(X)                                                                                                      \
   do {                                                                                                                      \
     auto kern = retention_chunks_kernel<X, X>;                                                                              \
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);               \
-    launch_pdl(kern, grid, dim3(256), smem, stream, proj, ldp, cos_t, sin_t, pairs, decay, cu_q, n_entries, walk_max, U, H, d, dv); \
+    launch_pdl(kern, grid, dim3(256), smem, stream, proj, ldp, cos_t, sin_t, pairs, decay, cu_q, n_entries, walk_max, U, H, d, dv, \
+               ret_rows_padded(d, t), vec);                                                                                 \
   } while (0)
     if (t == 2) SRLM_CHUNKS(2);
     else if (t == 4) SRLM_CHUNKS(4);
     else SRLM_CHUNKS(8);
 #undef SRLM_CHUNKS
   }
-  launch_pdl(retention_fold_kernel, dim3((unsigned)(((size_t)H * d * dv + 255) / 256), n_entries), dim3(256), 0, stream, U, decay,
-             state, state_stride, cu_q, slots, walk_max, H, d, dv);
+  const size_t elements = (size_t)H * d * dv;
+  if (vec) launch_pdl(retention_fold_kernel<4>, dim3((unsigned)((elements / 4 + 255) / 256), n_entries), dim3(256), 0, stream, U,
+                      decay, state, state_stride, cu_q, slots, walk_max, H, d, dv);
+  else launch_pdl(retention_fold_kernel<1>, dim3((unsigned)((elements + 255) / 256), n_entries), dim3(256), 0, stream, U, decay,
+                  state, state_stride, cu_q, slots, walk_max, H, d, dv);
   const size_t smem = ret_read_smem(d, tn);
   const dim3 grid(chunks, H, (dv + 16 * tn - 1) / (16 * tn));
 #define SRLM_READ(X)                                                                                                       \
@@ -556,7 +654,7 @@ extern "C" int srlm_retention_in_chunks(const float* proj, long long ldp, const 
     auto kern = retention_read_kernel<X, TO>;                                                                              \
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);              \
     launch_pdl(kern, grid, dim3(256), smem, stream, proj, ldp, cos_t, sin_t, pairs, decay, eps, cu_q, n_entries, walk_max, U, \
-               finishes ? (float*)nullptr : o_out, (TO*)out, H, d, dv);                                                    \
+               finishes ? (float*)nullptr : o_out, (TO*)out, H, d, dv, (d + 3) / 4 * 4, vec);                                                    \
   })
   if (tn == 2) SRLM_READ(2);
   else if (tn == 4) SRLM_READ(4);
