@@ -71,13 +71,16 @@ struct MixCopy {
 // ---- the softmax's sums -------------------------------------------------------------------------------------------
 constexpr int kLseRows = 64, kLseKeys = 64;
 
+// KS > 0: keys of exactly KS * 16 elements; 0: of dk_ elements.
+template <int KS>
 __global__ void __launch_bounds__(128)
 mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache, float* __restrict__ lse,
                       const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_q,
-                      const int* __restrict__ kv_lens, int nq, int nkv, int dk, int page_size, int page_shift, float scale2,
+                      const int* __restrict__ kv_lens, int nq, int nkv, int dk_, int page_size, int page_shift, float scale2,
                       MixMask mask, DistanceBias bias, int span) {
   pdl_wait();
   pdl_trigger();
+  const int dk = KS > 0 ? KS * 16 : dk_;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const int e = blockIdx.z, kvh = blockIdx.y, G = nq / nkv;
   const int t0 = cu_q[e], q_len = cu_q[e + 1] - t0, start = kv_lens[e] - q_len, rows = q_len * G;
@@ -111,12 +114,20 @@ mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
   const int first_seen = mask.first_key(min_pos);
   const MixTiles tiles(mask, min_pos, max_pos, kLseKeys);
   auto fetch = [&](int jb, int buf) {
-#pragma unroll 4
-    for (int jj = copy.r; jj < kLseKeys; jj += copy.step) {
-      const int j = jb + jj;
-      const bool there = j <= max_pos && (j >= first_seen || j < mask.keep);
-      const size_t row = there ? pages.row(j) + kvh * page_size : 0;
-      cp_async_16(k_s + (buf * kLseKeys + jj) * ks + copy.c * 8, k_cache + row * dk + copy.c * 8, there);
+    const bf16* pool = k_cache + (size_t)kvh * page_size * dk + copy.c * 8;
+    bf16* to = k_s + buf * kLseKeys * ks + copy.c * 8;
+    if (jb >= first_seen && jb + kLseKeys - 1 <= max_pos) {
+#pragma unroll
+      for (int x = 0; x < 8; ++x) {              // (a step of 8 rows or more: keys of up to 128 elements)
+        const int jj = copy.r + x * copy.step;
+        if (jj < kLseKeys) cp_async_16(to + jj * ks, pool + (size_t)pages.row(jb + jj) * dk, true);
+      }
+    } else {
+      for (int jj = copy.r; jj < kLseKeys; jj += copy.step) {
+        const int j = jb + jj;
+        const bool there = j <= max_pos && (j >= first_seen || j < mask.keep);
+        cp_async_16(to + jj * ks, there ? pool + (size_t)pages.row(j) * dk : k_cache, there);
+      }
     }
     cp_async_commit();
     if (bias.table) {
@@ -144,6 +155,7 @@ mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
       for (int c = 0; c < 4; ++c) s[i][c] = 0.f;
     const bf16* qa = q_s + (warp * 16 + (lane & 15)) * ks + (lane >> 4) * 8;
     const bf16* kb = k_s + (buf * kLseKeys + (lane & 7) + (lane >> 4) * 8) * ks + ((lane >> 3) & 1) * 8;
+#pragma unroll(KS > 0 ? KS : 1)
     for (int k0 = 0; k0 < dk; k0 += 16) {
       uint32_t a[4];
       ldmatrix_x4(a, qa + k0);
@@ -210,56 +222,60 @@ mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
 }
 
 // ---- weights, mixture, values ----------------------------------------------------------------------------------------
-// KS: 16-element steps of a key (at most), NT: 8-column tiles of the block's slab of values (at most), HT: 16-head tiles of
-// the mixture and heads of a warp's 16 rows.
-template <int KS, int NT, int HT>
+// KS: 16-element steps of a key, NT: 8-column tiles of the block's slab of values, HT: 16-head tiles of the mixture and heads
+// of a warp's 16 rows.  EXACT: exactly so many, 16 HT heads and one slab; else at most.
+template <int KS, int NT, int HT, bool EXACT>
 __global__ void __launch_bounds__(512)
 mixed_head_attention_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache,
                                 const bf16* __restrict__ v_cache, const float* __restrict__ lse, bf16* __restrict__ out,
                                 const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_q,
-                                const int* __restrict__ kv_lens, int nq, int nkv, int dk, int dv, int slab, int page_size,
+                                const int* __restrict__ kv_lens, int nq_, int nkv, int dk_, int dv_, int slab_, int page_size,
                                 int page_shift, float scale2, MixMask mask, DistanceBias bias, const float* __restrict__ mix, int mix_low,
                                 ElementGate gate, int nsplit, float* __restrict__ part) {
   pdl_wait();
   pdl_trigger();
+  const int dk = EXACT ? KS * 16 : dk_, dv = EXACT ? NT * 8 : dv_, slab = EXACT ? NT * 8 : slab_, nq = EXACT ? 16 * HT : nq_;
   constexpr int R = 16 / HT;                                   // tokens of the block
   constexpr int HP = 16 * HT;                                  // heads, padded
   constexpr int RS = R * kMhRow + kMhPad;                      // a head's weights of a tile
   constexpr int BL = R + kMhKeys;                              // distances of a tile
   extern __shared__ __align__(16) unsigned char smem_raw[];
-  const int e = blockIdx.z, slabs = (dv + slab - 1) / slab, G = nq / nkv;
-  const int c0 = (blockIdx.y % slabs) * slab, split = blockIdx.y / slabs;
+  const int e = blockIdx.z, slabs = EXACT ? 1 : (dv + slab - 1) / slab, G = nq / nkv;
+  const int c0 = EXACT ? 0 : (blockIdx.y % slabs) * slab, split = blockIdx.y / slabs;
   const int t0 = cu_q[e], q_len = cu_q[e + 1] - t0, start = kv_lens[e] - q_len;
   const int i0 = (gridDim.x - 1 - blockIdx.x) * R;
   if (i0 >= q_len) return;
-  const int ks = dk + kMhPad, width = min(slab, dv - c0), vs = slab + kMhPad;
+  const int ks = dk + kMhPad, width = EXACT ? slab : min(slab, dv - c0), vs = slab + kMhPad;
   bf16* k_s = reinterpret_cast<bf16*>(smem_raw);               // [nkv][32][dk + 8]
   bf16* v_s = k_s + nkv * kMhKeys * ks;                        // [nkv][32][slab + 8]
   bf16* p_hi = v_s + nkv * kMhKeys * vs;                       // [HP][RS]: weights, then their mixture
   bf16* p_lo = p_hi + HP * RS;
   bf16* mix_s = p_lo + HP * RS;                                // [2][HP][HP + 8]
   float* bias_s = reinterpret_cast<float*>(mix_s + 2 * HP * (HP + kMhPad));   // [nq][BL]
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, warps = blockDim.x >> 5;
+  const int threads = EXACT ? 512 : blockDim.x;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, warps = threads >> 5;
   const MixPages pages{block_table + (size_t)e * table_stride, nkv, page_size, page_shift};
   const int min_pos = start + i0, max_pos = start + min(q_len, i0 + R) - 1;
   const int first_seen = mask.first_key(min_pos);
   const MixTiles tiles(mask, min_pos, max_pos, kMhKeys);
   const int per = (tiles.count + nsplit - 1) / nsplit;
   const int n_first = split * per, n_last = min(tiles.count, n_first + per);
-  const MixCopy k_copy(dk / 8, blockDim.x), v_copy(width / 8, blockDim.x);
 
-  auto fetch = [&](int jb, const MixCopy& copy, bf16* dst, int stride, const bf16* pool, int dim) {
-#pragma unroll 4
-    for (int row = copy.r; row < nkv * kMhKeys; row += copy.step) {
-      const int h = row / kMhKeys, j = jb + row % kMhKeys;
+  // a thread looks a key up once and copies its piece of the key's row for every KV head
+  auto fetch = [&](int jb, int vec, bf16* dst, int stride, const bf16* pool, int dim) {
+    for (int slot = tid; slot < kMhKeys * vec; slot += threads) {
+      const int jj = slot / vec, c = (slot - jj * vec) * 8, j = jb + jj;
       const bool there = j <= max_pos && (j >= first_seen || j < mask.keep);
-      const size_t at = there ? pages.row(j) + h * page_size : 0;
-      cp_async_16(dst + row * stride + copy.c * 8, pool + at * dim + copy.c * 8, there);
+      const bf16* src = pool + (there ? (size_t)pages.row(j) * dim + c : 0);
+      bf16* to = dst + jj * stride + c;
+      const int src_step = there ? page_size * dim : 0, to_step = kMhKeys * stride;
+#pragma unroll 4
+      for (int h = 0; h < nkv; ++h, src += src_step, to += to_step) cp_async_16(to, src, there);
     }
     cp_async_commit();
   };
-  auto fetch_k = [&](int jb) { fetch(jb, k_copy, k_s, ks, k_cache, dk); };
-  auto fetch_v = [&](int jb) { fetch(jb, v_copy, v_s, vs, v_cache + c0, dv); };
+  auto fetch_k = [&](int jb) { fetch(jb, dk / 8, k_s, ks, k_cache, dk); };
+  auto fetch_v = [&](int jb) { fetch(jb, width / 8, v_s, vs, v_cache + c0, dv); };
   if (n_first < n_last) fetch_k(tiles.key(n_first, kMhKeys));
 
   // the mixture's matrix as a pair of bfloat16 (the rounding, and what it leaves), and zero rows for heads that do not exist
@@ -291,7 +307,7 @@ mixed_head_attention_mma_kernel(const bf16* __restrict__ q, const bf16* __restri
     const bf16* src = q + ((size_t)(t0 + i0 + (live ? tok : 0)) * nq + h) * dk + (lane & 3) * 2;
 #pragma unroll
     for (int k = 0; k < KS; ++k) {
-      const bool there = live && k * 16 < dk;
+      const bool there = live && (EXACT || k * 16 < dk);
       qf[k][i] = there ? *reinterpret_cast<const uint32_t*>(src + k * 16) : 0u;
       qf[k][2 + i] = there ? *reinterpret_cast<const uint32_t*>(src + k * 16 + 8) : 0u;
     }
@@ -325,7 +341,7 @@ mixed_head_attention_mma_kernel(const bf16* __restrict__ q, const bf16* __restri
     const bf16* kb = k_s + (kvh * kMhKeys + (lane & 7) + (lane >> 4) * 8) * ks + ((lane >> 3) & 1) * 8;
 #pragma unroll
     for (int k = 0; k < KS; ++k) {
-      if (k * 16 < dk) {
+      if (EXACT || k * 16 < dk) {
 #pragma unroll
         for (int n2 = 0; n2 < kMhKeys / 16; ++n2) {
           uint32_t b[4];
@@ -375,6 +391,7 @@ mixed_head_attention_mma_kernel(const bf16* __restrict__ q, const bf16* __restri
     // the mixture, in place: a warp takes 8 keys of a token at a time, all heads
     uint32_t mix_f[4];                                         // one tile of heads: its matrix is loaded once
     if (HT == 1) ldmatrix_x4(mix_f, mix_s + (lane & 15) * (HP + kMhPad) + (lane >> 4) * 8);
+#pragma unroll(EXACT ? R * (kMhKeys / 8) / 16 : 1)
     for (int ct = warp; ct < R * (kMhKeys / 8); ct += warps) {
       const int col = (ct / (kMhKeys / 8)) * kMhRow + (ct % (kMhKeys / 8)) * 8;
       uint32_t b[HT][4];
@@ -413,7 +430,7 @@ mixed_head_attention_mma_kernel(const bf16* __restrict__ q, const bf16* __restri
       ldmatrix_x4(a, wa + kk * 16);
 #pragma unroll
       for (int n2 = 0; n2 < NT / 2; ++n2) {
-        if (n2 * 16 < width) {
+        if (EXACT || n2 * 16 < width) {
           uint32_t b[4];
           ldmatrix_x4_trans(b, vb + kk * 16 * vs + n2 * 16);
           mma_bf16(o[2 * n2], a, b[0], b[1]);
@@ -429,7 +446,7 @@ mixed_head_attention_mma_kernel(const bf16* __restrict__ q, const bf16* __restri
     if (tok >= q_len) continue;
 #pragma unroll
     for (int n = 0; n < NT; ++n) {
-      if (n * 8 >= width) continue;
+      if (!EXACT && n * 8 >= width) continue;
       const int c = h * dv + c0 + n * 8 + (lane & 3) * 2;
       if (nsplit > 1) {
         *reinterpret_cast<float2*>(part + ((size_t)(t0 + tok) * nsplit + split) * nq * dv + c) = make_float2(o[n][2 * i], o[n][2 * i + 1]);
@@ -489,18 +506,20 @@ struct MixDecodeLayout {             // offsets in bytes of a block's shared mem
   }
 };
 
-// UN: units of 32 value columns of 16 rows that a warp holds.  grid (cluster, entries).
-template <int UN>
+// UN: units of 32 value columns of 16 rows that a warp holds; D > 0: keys and values of exactly D elements (0: of dk_ and
+// dv_).  grid (cluster, entries).
+template <int UN, int D>
 __global__ void __launch_bounds__(kMdThreads)
 mixed_head_attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache,
                                    const bf16* __restrict__ v_cache, bf16* __restrict__ out,
                                    const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_q,
-                                   const int* __restrict__ kv_lens, int nq, int nkv, int row_tiles, int dk, int dv,
+                                   const int* __restrict__ kv_lens, int nq, int nkv, int row_tiles, int dk_, int dv_,
                                    int page_size, int page_shift, float scale2, MixMask mask, DistanceBias bias,
                                    const float* __restrict__ mix, ElementGate gate, int tiles_cap, int nbuf) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ __align__(16) unsigned char smem_raw[];
+  const int dk = D > 0 ? D : dk_, dv = D > 0 ? D : dv_;
   const MixDecodeLayout at(nq, nkv, row_tiles, dk, dv, tiles_cap, nbuf);
   bf16* q_s = reinterpret_cast<bf16*>(smem_raw + at.q);        // [nkv][row_tiles * 16][dk + 8]
   bf16* w_s = reinterpret_cast<bf16*>(smem_raw + at.w);        // [nkv][row_tiles * 16][40]
@@ -519,22 +538,22 @@ mixed_head_attention_decode_kernel(const bf16* __restrict__ q, const bf16* __res
   if (per > tiles_cap) per = tiles_cap;
   const int n0 = min(tiles.count, rank * per), n_here = min(tiles.count - n0, per);
   const int kvec = dk / 8;
-  const MixCopy k_copy(dk / 8, kMdThreads), v_copy(dv / 8, kMdThreads);
 
   // stage x: 0 .. n_here - 1 fetch keys, n_here .. 2 n_here - 1 values, buffer x % nbuf
   auto fetch = [&](int x) {
     const bool values = x >= n_here;
     const int jb = tiles.key(n0 + (values ? x - n_here : x), kMhKeys);
     bf16* dst = reinterpret_cast<bf16*>(smem_raw + at.tile + (x % nbuf) * at.tile_bytes);
-    const MixCopy& copy = values ? v_copy : k_copy;
-    const int stride = values ? vs : ks, dim = values ? dv : dk;
+    const int vec = (values ? dv : dk) / 8, stride = values ? vs : ks, dim = values ? dv : dk;
     const bf16* pool = values ? v_cache : k_cache;
-#pragma unroll 4
-    for (int row = copy.r; row < nkv * kMhKeys; row += copy.step) {
-      const int h = row / kMhKeys, j = jb + row % kMhKeys;
+    for (int slot = tid; slot < kMhKeys * vec; slot += kMdThreads) {
+      const int jj = slot / vec, c = (slot - jj * vec) * 8, j = jb + jj;
       const bool there = mask.visible(pos, j);
-      const size_t src = there ? pages.row(j) + h * page_size : 0;
-      cp_async_16(dst + row * stride + copy.c * 8, pool + src * dim + copy.c * 8, there);
+      const bf16* src = pool + (there ? (size_t)pages.row(j) * dim + c : 0);
+      bf16* to = dst + jj * stride + c;
+      const int src_step = there ? page_size * dim : 0, to_step = kMhKeys * stride;
+#pragma unroll 4
+      for (int h = 0; h < nkv; ++h, src += src_step, to += to_step) cp_async_16(to, src, there);
     }
     cp_async_commit();
   };
@@ -576,6 +595,7 @@ mixed_head_attention_decode_kernel(const bf16* __restrict__ q, const bf16* __res
         float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
         const bf16* qa = q_s + (rt * 16 + (lane & 15)) * ks + (lane >> 4) * 8;
         const bf16* kb = buf + (h * kMhKeys + n2 * 16 + (lane & 7) + (lane >> 4) * 8) * ks + ((lane >> 3) & 1) * 8;
+#pragma unroll(D > 0 ? D / 16 : 1)
         for (int k0 = 0; k0 < dk; k0 += 16) {
           uint32_t a[4], b[4];
           ldmatrix_x4(a, qa + k0);
@@ -753,17 +773,18 @@ extern "C" int srlm_mixed_head_attention_mma(const void* q, const void* k_cache,
   const float scale2 = scale * kLog2e;
   {
     const size_t smem = mh_lse_smem(G, dk);
-    if (smem > 48 * 1024) cudaFuncSetAttribute(mixed_head_lse_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    launch_pdl(mixed_head_lse_kernel, dim3((unsigned)(((long long)max_q_len * G + kLseRows - 1) / kLseRows), nkv, n_entries), dim3(128),
+    auto kern = dk == 64 ? mixed_head_lse_kernel<4> : dk == 128 ? mixed_head_lse_kernel<8> : mixed_head_lse_kernel<0>;
+    if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    launch_pdl(kern, dim3((unsigned)(((long long)max_q_len * G + kLseRows - 1) / kLseRows), nkv, n_entries), dim3(128),
                smem, stream, (const bf16*)q, (const bf16*)k_cache, lse, block_table, table_stride, cu_q, kv_lens, nq, nkv, dk,
                page_size, mh_page_shift(page_size), scale2, mask, db, mh_lse_span(G));
   }
   const size_t smem = mh_rows_smem(nq, nkv, dk, dv);
   const dim3 grid((unsigned)((max_q_len + R - 1) / R), (unsigned)(slabs * nsplit), (unsigned)n_entries);
   const int threads = nq / ht * 32;
-#define SRLM_MH(KS, NT, HT)                                                                                             \
+#define SRLM_MH(KS, NT, HT, EX)                                                                                           \
   do {                                                                                                                  \
-    auto kern = mixed_head_attention_mma_kernel<KS, NT, HT>;                                                            \
+    auto kern = mixed_head_attention_mma_kernel<KS, NT, HT, EX>;                                                            \
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);           \
     launch_pdl(kern, grid, dim3(threads), smem, stream, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, lse, \
                (bf16*)out, block_table, table_stride, cu_q, kv_lens, nq, nkv, dk, dv, slab, page_size, mh_page_shift(page_size), scale2, mask, db, \
@@ -771,8 +792,10 @@ extern "C" int srlm_mixed_head_attention_mma(const void* q, const void* k_cache,
   } while (0)
 #define SRLM_MH_SIZES(HT)                               \
   do {                                                  \
-    if (dk <= 64 && slab <= 64) SRLM_MH(4, 8, HT);      \
-    else SRLM_MH(8, 16, HT);                            \
+    if (dk == 64 && dv == 64 && nq == 16 * HT) SRLM_MH(4, 8, HT, true);          \
+    else if (dk == 128 && dv == 128 && nq == 16 * HT) SRLM_MH(8, 16, HT, true);  \
+    else if (dk <= 64 && slab <= 64) SRLM_MH(4, 8, HT, false); \
+    else SRLM_MH(8, 16, HT, false);                     \
   } while (0)
   if (ht == 1) SRLM_MH_SIZES(1);
   else SRLM_MH_SIZES(2);
@@ -826,18 +849,24 @@ extern "C" int srlm_mixed_head_attention_decode(const void* q, const void* k_cac
   attr[1].val.programmaticStreamSerializationAllowed = pdl_enabled() ? 1 : 0;
   cfg.attrs = attr;
   cfg.numAttrs = 2;
-#define SRLM_MD(UN)                                                                                                   \
+#define SRLM_MD(UN, D)                                                                                                 \
   do {                                                                                                                \
-    auto kern = mixed_head_attention_decode_kernel<UN>;                                                               \
+    auto kern = mixed_head_attention_decode_kernel<UN, D>;                                                              \
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);              \
     if (cluster > 8) cudaFuncSetAttribute(kern, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);                   \
     cudaLaunchKernelEx(&cfg, kern, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, (bf16*)out, block_table, \
                        table_stride, cu_q, kv_lens, nq, nkv, row_tiles, dk, dv, page_size, mh_page_shift(page_size), scale * kLog2e, mask, db, mix, \
                        gate, tiles_here, nbuf);                                                                       \
   } while (0)
-  if (units <= 2 * kMdWarps) SRLM_MD(2);
-  else if (units <= 4 * kMdWarps) SRLM_MD(4);
-  else SRLM_MD(8);
+#define SRLM_MD_UNITS(D)                             \
+  do {                                              \
+    if (units <= 2 * kMdWarps) SRLM_MD(2, D);       \
+    else if (units <= 4 * kMdWarps) SRLM_MD(4, D);  \
+    else SRLM_MD(8, D);                             \
+  } while (0)
+  if (dk == 128 && dv == 128) SRLM_MD_UNITS(128);
+  else SRLM_MD_UNITS(0);
+#undef SRLM_MD_UNITS
 #undef SRLM_MD
   return launched();
 }
