@@ -18,9 +18,10 @@ struct MixMask {
 struct DistanceBias {
   const float* table;
   int n;
-  __device__ __forceinline__ float at(int head, int distance) const {
-    return table ? table[(size_t)head * n + (distance < n ? distance : n - 1)] : 0.f;
+  __device__ __forceinline__ const float* of(int head, int distance) const {
+    return table + (size_t)head * n + (distance < n ? distance : n - 1);
   }
+  __device__ __forceinline__ float at(int head, int distance) const { return table ? *of(head, distance) : 0.f; }
 };
 
 // Element c (head * dv + d) of token t is multiplied by logistic(logits[t * ld + c]); logits null: no gate.

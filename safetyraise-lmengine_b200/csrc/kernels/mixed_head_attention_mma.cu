@@ -1,6 +1,6 @@
 // The mixed-head attention of mixed_head_attention.cu on bfloat16 tensor cores (mma.sync m16n8k16, float32 sums).
 //
-// Prompts, portions and mixed steps take two kernels.  Scores are kept in units of log2, so a softmax is one 2^x:
+// Prompts, portions and mixed steps take two kernels:
 //   mixed_head_lse      every row's logarithm of the softmax's sum, L = log2 sum_j 2^(s_j), a block for 64 rows (tokens x
 //                       query heads) of one KV head: the running maximum and sum of an ordinary attention, without values;
 //   mixed_head_attention_mma   a block for 16 / HT tokens and ALL heads.  Per tile of 32 keys: every warp forms the scores
@@ -76,7 +76,7 @@ template <int KS>
 __global__ void __launch_bounds__(128)
 mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache, float* __restrict__ lse,
                       const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_q,
-                      const int* __restrict__ kv_lens, int nq, int nkv, int dk_, int page_size, int page_shift, float scale2,
+                      const int* __restrict__ kv_lens, int nq, int nkv, int dk_, int page_size, int page_shift, float scale,
                       MixMask mask, DistanceBias bias, int span) {
   pdl_wait();
   pdl_trigger();
@@ -129,14 +129,14 @@ mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
         cp_async_16(to + jj * ks, there ? pool + (size_t)pages.row(j) * dk : k_cache, there);
       }
     }
-    cp_async_commit();
     if (bias.table) {
       // bias_s[h][x] belongs to distance min_pos - (jb + 63) + x
       const int d0 = min_pos - jb - (kLseKeys - 1);
       for (int h = warp; h < G; h += 4)
         for (int x = lane; x < span; x += 32)
-          bias_s[(size_t)(buf * G + h) * span + x] = bias.at(kvh * G + h, max(d0 + x, 0)) * kLog2e;
+          cp_async_4(bias_s + (size_t)(buf * G + h) * span + x, bias.of(kvh * G + h, max(d0 + x, 0)));
     }
+    cp_async_commit();
   };
   fetch(tiles.key(0, kLseKeys), 0);
   for (int n = 0, buf = 0; n < tiles.count; ++n, buf ^= 1) {
@@ -175,14 +175,14 @@ mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
         const float* bs = bias_s + (size_t)(buf * G + head[i]) * span + max(pos[i] - min_pos, 0) + (kLseKeys - 1) - (lane & 3) * 2;
 #pragma unroll
         for (int x = 0; x < 8; ++x) {
-          s[x][2 * i] = fmaf(s[x][2 * i], scale2, bs[-x * 8]);
-          s[x][2 * i + 1] = fmaf(s[x][2 * i + 1], scale2, bs[-x * 8 - 1]);
+          s[x][2 * i] = fmaf(s[x][2 * i], scale, bs[-x * 8]);
+          s[x][2 * i + 1] = fmaf(s[x][2 * i + 1], scale, bs[-x * 8 - 1]);
         }
       } else {
 #pragma unroll
         for (int x = 0; x < 8; ++x) {
-          s[x][2 * i] *= scale2;
-          s[x][2 * i + 1] *= scale2;
+          s[x][2 * i] *= scale;
+          s[x][2 * i + 1] *= scale;
         }
       }
       if (!whole) {
@@ -199,13 +199,14 @@ mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
       const float m_new = fmaxf(m[i], mx);
       if (m_new != -CUDART_INF_F) {
+        const float m2 = m_new * kLog2e;
         float sum[2] = {0.f, 0.f};
 #pragma unroll
         for (int x = 0; x < 8; ++x) {
-          sum[0] += pow2(s[x][2 * i] - m_new);
-          sum[1] += pow2(s[x][2 * i + 1] - m_new);
+          sum[0] += pow2(fmaf(s[x][2 * i], kLog2e, -m2));
+          sum[1] += pow2(fmaf(s[x][2 * i + 1], kLog2e, -m2));
         }
-        l[i] = l[i] * pow2(m[i] - m_new) + sum[0] + sum[1];    // the lane's own share of the row's sum
+        l[i] = l[i] * pow2(fmaf(m[i], kLog2e, -m2)) + sum[0] + sum[1];    // the lane's own share of the row's sum
         m[i] = m_new;
       }
     }
@@ -217,7 +218,7 @@ mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
     sum += __shfl_xor_sync(0xffffffffu, sum, 1);
     sum += __shfl_xor_sync(0xffffffffu, sum, 2);
     const int row = r0 + warp * 16 + (lane >> 2) + 8 * i;
-    if (row < rows && (lane & 3) == 0) lse[(size_t)(t0 + row / G) * nq + kvh * G + row % G] = m[i] + log2f(sum);
+    if (row < rows && (lane & 3) == 0) lse[(size_t)(t0 + row / G) * nq + kvh * G + row % G] = m[i] * kLog2e + log2f(sum);
   }
 }
 
@@ -230,7 +231,7 @@ mixed_head_attention_mma_kernel(const bf16* __restrict__ q, const bf16* __restri
                                 const bf16* __restrict__ v_cache, const float* __restrict__ lse, bf16* __restrict__ out,
                                 const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_q,
                                 const int* __restrict__ kv_lens, int nq_, int nkv, int dk_, int dv_, int slab_, int page_size,
-                                int page_shift, float scale2, MixMask mask, DistanceBias bias, const float* __restrict__ mix, int mix_low,
+                                int page_shift, float scale, MixMask mask, DistanceBias bias, const float* __restrict__ mix, int mix_low,
                                 ElementGate gate, int nsplit, float* __restrict__ part) {
   pdl_wait();
   pdl_trigger();
@@ -261,22 +262,60 @@ mixed_head_attention_mma_kernel(const bf16* __restrict__ q, const bf16* __restri
   const int per = (tiles.count + nsplit - 1) / nsplit;
   const int n_first = split * per, n_last = min(tiles.count, n_first + per);
 
-  // a thread looks a key up once and copies its piece of the key's row for every KV head
-  auto fetch = [&](int jb, int vec, bf16* dst, int stride, const bf16* pool, int dim) {
-    for (int slot = tid; slot < kMhKeys * vec; slot += threads) {
-      const int jj = slot / vec, c = (slot - jj * vec) * 8, j = jb + jj;
-      const bool there = j <= max_pos && (j >= first_seen || j < mask.keep);
-      const bf16* src = pool + (there ? (size_t)pages.row(j) * dim + c : 0);
-      bf16* to = dst + jj * stride + c;
-      const int src_step = there ? page_size * dim : 0, to_step = kMhKeys * stride;
+  // A thread looks a key up once and copies its piece of the key's row for every KV head.  EXACT: one key a thread, whose
+  // row is looked up a tile ahead of its copies, so that no copy waits for the block table.
+  auto there = [&](int j) { return j <= max_pos && (j >= first_seen || j < mask.keep); };
+  auto copy = [&](const bf16* pool, int dim, int row, int c, bf16* to, int stride) {
+    const bf16* src = pool + (row >= 0 ? (size_t)row * dim + c : 0);
+    const int src_step = row >= 0 ? page_size * dim : 0, to_step = kMhKeys * stride;
 #pragma unroll 4
-      for (int h = 0; h < nkv; ++h, src += src_step, to += to_step) cp_async_16(to, src, there);
+    for (int h = 0; h < nkv; ++h, src += src_step, to += to_step) cp_async_16(to, src, row >= 0);
+  };
+  constexpr int EV = EXACT ? KS * 2 : 1;                       // EXACT: pieces of a row (keys and values alike)
+  static_assert(!EXACT || (kMhKeys * EV <= 512 && KS * 16 == NT * 8), "a thread copies one piece of one key");
+  const int my_key = tid / EV, my_c = (tid % EV) * 8;
+  auto look_up = [&](int n) {
+    const int j = my_key < kMhKeys && n < n_last ? tiles.key(n, kMhKeys) + my_key : 1 << 30;
+    return there(j) ? pages.row(j) : -1;
+  };
+  auto fetch_rows = [&](int jb, int vec, bf16* dst, int stride, const bf16* pool, int dim) {
+    for (int slot = tid; slot < kMhKeys * vec; slot += threads) {
+      const int jj = slot / vec, c = (slot - jj * vec) * 8;
+      copy(pool, dim, there(jb + jj) ? pages.row(jb + jj) : -1, c, dst + jj * stride + c, stride);
+    }
+  };
+  auto fetch_k = [&](int n, int row) {                         // and the biases of its distances
+    const int jb = tiles.key(n, kMhKeys);
+    if (EXACT) {
+      if (my_key < kMhKeys) copy(k_cache, dk, row, my_c, k_s + my_key * ks + my_c, ks);
+    } else {
+      fetch_rows(jb, dk / 8, k_s, ks, k_cache, dk);
+    }
+    if (bias.table) {                                          // bias_s[h][x]: distance min_pos - (jb + 31) + x
+      const int d0 = min_pos - jb - (kMhKeys - 1);
+#pragma unroll
+      for (int i = 0; i < HT; ++i)
+#pragma unroll
+        for (int x = 0; x < (BL + 31) / 32; ++x)
+          if (x * 32 + lane < BL)
+            cp_async_4(bias_s + (warp * HT + i) * BL + x * 32 + lane, bias.of(warp * HT + i, max(d0 + x * 32 + lane, 0)));
     }
     cp_async_commit();
   };
-  auto fetch_k = [&](int jb) { fetch(jb, dk / 8, k_s, ks, k_cache, dk); };
-  auto fetch_v = [&](int jb) { fetch(jb, width / 8, v_s, vs, v_cache + c0, dv); };
-  if (n_first < n_last) fetch_k(tiles.key(n_first, kMhKeys));
+  auto fetch_v = [&](int n, int row) {
+    if (EXACT) {
+      if (my_key < kMhKeys) copy(v_cache, dv, row, my_c, v_s + my_key * vs + my_c, vs);
+    } else {
+      fetch_rows(tiles.key(n, kMhKeys), width / 8, v_s, vs, v_cache + c0, dv);
+    }
+    cp_async_commit();
+  };
+  int row_now = -1, row_next = -1;                             // EXACT: of this tile's key, of the next tile's
+  if (EXACT) {
+    row_now = look_up(n_first);
+    row_next = look_up(n_first + 1);
+  }
+  if (n_first < n_last) fetch_k(n_first, row_now);
 
   // the mixture's matrix as a pair of bfloat16 (the rounding, and what it leaves), and zero rows for heads that do not exist
   for (int idx = tid; idx < HP * (HP + kMhPad); idx += blockDim.x) {
@@ -320,18 +359,9 @@ mixed_head_attention_mma_kernel(const bf16* __restrict__ q, const bf16* __restri
 
   for (int n = n_first; n < n_last; ++n) {
     const int jb = tiles.key(n, kMhKeys);
-    if (bias.table) {                                          // bias_s[h][x]: distance min_pos - (jb + 31) + x
-      const int d0 = min_pos - jb - (kMhKeys - 1);
-#pragma unroll
-      for (int i = 0; i < HT; ++i)
-#pragma unroll
-        for (int x = 0; x < (BL + 31) / 32; ++x)
-          if (x * 32 + lane < BL)
-            bias_s[(head0 + i) * BL + x * 32 + lane] = bias.at(head0 + i, max(d0 + x * 32 + lane, 0)) * kLog2e;
-    }
     cp_async_wait<0>();
     __syncthreads();                                           // the keys are here; the values and weights before are read
-    fetch_v(jb);
+    fetch_v(n, row_now);
 
     float s[kMhKeys / 8][4];
 #pragma unroll
@@ -358,14 +388,14 @@ mixed_head_attention_mma_kernel(const bf16* __restrict__ q, const bf16* __restri
         const float* bs = bias_s + bias_at[i];
 #pragma unroll
         for (int x = 0; x < kMhKeys / 8; ++x) {
-          s[x][2 * i] = pow2(fmaf(s[x][2 * i], scale2, bs[-x * 8] - L[i]));
-          s[x][2 * i + 1] = pow2(fmaf(s[x][2 * i + 1], scale2, bs[-x * 8 - 1] - L[i]));
+          s[x][2 * i] = pow2(fmaf(fmaf(s[x][2 * i], scale, bs[-x * 8]), kLog2e, -L[i]));
+          s[x][2 * i + 1] = pow2(fmaf(fmaf(s[x][2 * i + 1], scale, bs[-x * 8 - 1]), kLog2e, -L[i]));
         }
       } else {
 #pragma unroll
         for (int x = 0; x < kMhKeys / 8; ++x) {
-          s[x][2 * i] = pow2(fmaf(s[x][2 * i], scale2, -L[i]));
-          s[x][2 * i + 1] = pow2(fmaf(s[x][2 * i + 1], scale2, -L[i]));
+          s[x][2 * i] = pow2(fmaf(s[x][2 * i], scale * kLog2e, -L[i]));
+          s[x][2 * i + 1] = pow2(fmaf(s[x][2 * i + 1], scale * kLog2e, -L[i]));
         }
       }
       if (!whole) {
@@ -386,7 +416,11 @@ mixed_head_attention_mma_kernel(const bf16* __restrict__ q, const bf16* __restri
       }
     }
     __syncthreads();                                           // all heads' weights are written; the keys are read
-    if (n + 1 < n_last) fetch_k(tiles.key(n + 1, kMhKeys));
+    if (n + 1 < n_last) fetch_k(n + 1, row_next);
+    if (EXACT) {
+      row_now = row_next;
+      row_next = look_up(n + 2);
+    }
 
     // the mixture, in place: a warp takes 8 keys of a token at a time, all heads
     uint32_t mix_f[4];                                         // one tile of heads: its matrix is loaded once
@@ -481,7 +515,7 @@ __device__ __forceinline__ float mh_remote(const float* p, int rank) {
   uint32_t r;
   float v;
   asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(a), "r"(rank));
-  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(r) : "memory");
+  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(r));
   return v;
 }
 
@@ -634,14 +668,12 @@ mixed_head_attention_decode_kernel(const bf16* __restrict__ q, const bf16* __res
     }
     if (x == n_here - 1) {
       mh_cluster_sync();
-      for (int h = tid; h < nq; h += blockDim.x) {
-        float m = -CUDART_INF_F, l = 0.f;
-        for (int r = 0; r < cluster; ++r) m = fmaxf(m, mh_remote(stats + 2 * h, r));
-        for (int r = 0; r < cluster; ++r) {
-          const float mr = mh_remote(stats + 2 * h, r);
-          if (mr != -CUDART_INF_F) l += mh_remote(stats + 2 * h + 1, r) * pow2(mr - m);
-        }
-        lse[h] = m + log2f(l);
+      for (int h = warp; h < nq; h += kMdWarps) {              // a lane a block of the cluster
+        const float mr = lane < cluster ? mh_remote(stats + 2 * h, lane) : -CUDART_INF_F;
+        const float lr = lane < cluster ? mh_remote(stats + 2 * h + 1, lane) : 0.f;
+        const float m = warp_max(mr);
+        const float l = warp_sum(mr != -CUDART_INF_F ? lr * pow2(mr - m) : 0.f);
+        if (lane == 0) lse[h] = m + log2f(l);
       }
       __syncthreads();
       for (int h = warp; h < nq; h += kMdWarps)
@@ -709,7 +741,12 @@ mixed_head_attention_decode_kernel(const bf16* __restrict__ q, const bf16* __res
   mh_cluster_sync();
   for (int c = rank * kMdThreads + tid; c < nq * dv; c += cluster * kMdThreads) {
     float a = 0.f;
-    for (int r = 0; r < cluster; ++r) a += mh_remote(o_s + c, r);
+    for (int r = 0; r < cluster; r += 4) {                     // four loads on their way at a time
+      float v[4];
+#pragma unroll
+      for (int x = 0; x < 4; ++x) v[x] = r + x < cluster ? mh_remote(o_s + c, r + x) : 0.f;
+      a += (v[0] + v[1]) + (v[2] + v[3]);
+    }
     out[(size_t)t * nq * dv + c] = __float2bfloat16_rn(a * gate.at(t, c));
   }
   mh_cluster_sync();                                           // nobody leaves while its sums are read
@@ -770,14 +807,13 @@ extern "C" int srlm_mixed_head_attention_mma(const void* q, const void* k_cache,
   const MixMask mask{window, window > 0 ? keep : 0};
   const DistanceBias db{bias, n_dist};
   const ElementGate gate{gate_logits, ld_gate};
-  const float scale2 = scale * kLog2e;
   {
     const size_t smem = mh_lse_smem(G, dk);
     auto kern = dk == 64 ? mixed_head_lse_kernel<4> : dk == 128 ? mixed_head_lse_kernel<8> : mixed_head_lse_kernel<0>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     launch_pdl(kern, dim3((unsigned)(((long long)max_q_len * G + kLseRows - 1) / kLseRows), nkv, n_entries), dim3(128),
                smem, stream, (const bf16*)q, (const bf16*)k_cache, lse, block_table, table_stride, cu_q, kv_lens, nq, nkv, dk,
-               page_size, mh_page_shift(page_size), scale2, mask, db, mh_lse_span(G));
+               page_size, mh_page_shift(page_size), scale, mask, db, mh_lse_span(G));
   }
   const size_t smem = mh_rows_smem(nq, nkv, dk, dv);
   const dim3 grid((unsigned)((max_q_len + R - 1) / R), (unsigned)(slabs * nsplit), (unsigned)n_entries);
@@ -787,7 +823,7 @@ extern "C" int srlm_mixed_head_attention_mma(const void* q, const void* k_cache,
     auto kern = mixed_head_attention_mma_kernel<KS, NT, HT, EX>;                                                            \
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);           \
     launch_pdl(kern, grid, dim3(threads), smem, stream, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, lse, \
-               (bf16*)out, block_table, table_stride, cu_q, kv_lens, nq, nkv, dk, dv, slab, page_size, mh_page_shift(page_size), scale2, mask, db, \
+               (bf16*)out, block_table, table_stride, cu_q, kv_lens, nq, nkv, dk, dv, slab, page_size, mh_page_shift(page_size), scale, mask, db, \
                mix, mix_low, gate, nsplit, part);                                                                       \
   } while (0)
 #define SRLM_MH_SIZES(HT)                               \

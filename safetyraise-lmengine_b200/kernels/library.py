@@ -1254,13 +1254,15 @@ class KernelLibrary:
 
     def mixed_head_decode_plan(self, n_entries, tiles, smem_of):
         """(cluster, tiles a block, buffers) of the decode form, or None: as many blocks an entry as keep the step within
-        one block an SM, more when a block's slice does not fit its shared memory (smem_of(tiles, buffers), 0: no)."""
+        one block an SM, more when a block's slice does not fit its shared memory (smem_of(tiles, buffers), 0: no).  A
+        cluster of 16 needs blocks of which two fit an SM: with one an SM too few such clusters run at a time."""
         sizes = [c for c in (1, 2, 4, 8, 16) if c <= self.mixed_heads_cluster]
         fits = [c for c in sizes if c <= tiles and c * n_entries <= self.SMS] or [1]
-        for c in [fits[-1]] + [c for c in sizes if c > fits[-1]]:
+        for c in fits[::-1] + [c for c in sizes if c > fits[-1]]:
             here = -(-tiles // c)
             for nbuf in (2, 1):
-                if smem_of(here, nbuf):
+                smem = smem_of(here, nbuf)
+                if smem and (c < 16 or smem <= 112 * 1024 or c > fits[-1]):
                     return c, here, nbuf
         return None
 
