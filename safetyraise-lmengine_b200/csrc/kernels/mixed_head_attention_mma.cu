@@ -71,9 +71,10 @@ struct MixCopy {
 // ---- the softmax's sums -------------------------------------------------------------------------------------------
 constexpr int kLseRows = 64, kLseKeys = 64;
 
-// KS > 0: keys of exactly KS * 16 elements; 0: of dk_ elements.
+// KS > 0: keys of exactly KS * 16 elements; 0: of dk_ elements.  Eight warps: warps w and w + 4 hold the same 16 rows, one the
+// first half of every tile's keys, the other the second; their maxima and sums meet at the end.
 template <int KS>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache, float* __restrict__ lse,
                       const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_q,
                       const int* __restrict__ kv_lens, int nq, int nkv, int dk_, int page_size, int page_shift, float scale,
@@ -92,7 +93,8 @@ mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
   float* bias_s = reinterpret_cast<float*>(k_s + 2 * kLseKeys * ks);    // [2][G][span]
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const MixPages pages{block_table + (size_t)e * table_stride, nkv, page_size, page_shift};
-  const MixCopy copy(dk / 8, 128);
+  const MixCopy copy(dk / 8, 256);
+  const int row0 = (warp & 3) * 16, half = (warp >> 2) * (kLseKeys / 2);
   for (int x = copy.r; x < kLseRows; x += copy.step) {
     const int row = r0 + x;
     const bool there = row < rows;
@@ -103,7 +105,7 @@ mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
   int pos[2], head[2];
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
-    const int row = r0 + warp * 16 + (lane >> 2) + 8 * i;
+    const int row = r0 + row0 + (lane >> 2) + 8 * i;
     pos[i] = row < rows ? start + row / G : -1;
     head[i] = row < rows ? row % G : 0;
     m[i] = -CUDART_INF_F;
@@ -118,7 +120,7 @@ mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
     bf16* to = k_s + buf * kLseKeys * ks + copy.c * 8;
     if (jb >= first_seen && jb + kLseKeys - 1 <= max_pos) {
 #pragma unroll
-      for (int x = 0; x < 8; ++x) {              // (a step of 8 rows or more: keys of up to 128 elements)
+      for (int x = 0; x < 4; ++x) {              // (a step of 16 rows or more: keys of up to 128 elements)
         const int jj = copy.r + x * copy.step;
         if (jj < kLseKeys) cp_async_16(to + jj * ks, pool + (size_t)pages.row(jb + jj) * dk, true);
       }
@@ -132,7 +134,7 @@ mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
     if (bias.table) {
       // bias_s[h][x] belongs to distance min_pos - (jb + 63) + x
       const int d0 = min_pos - jb - (kLseKeys - 1);
-      for (int h = warp; h < G; h += 4)
+      for (int h = warp; h < G; h += 8)
         for (int x = lane; x < span; x += 32)
           cp_async_4(bias_s + (size_t)(buf * G + h) * span + x, bias.of(kvh * G + h, max(d0 + x, 0)));
     }
@@ -148,19 +150,19 @@ mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
       cp_async_wait<0>();
     }
     __syncthreads();
-    float s[8][4];
+    float s[4][4];
 #pragma unroll
-    for (int i = 0; i < 8; ++i)
+    for (int i = 0; i < 4; ++i)
 #pragma unroll
       for (int c = 0; c < 4; ++c) s[i][c] = 0.f;
-    const bf16* qa = q_s + (warp * 16 + (lane & 15)) * ks + (lane >> 4) * 8;
-    const bf16* kb = k_s + (buf * kLseKeys + (lane & 7) + (lane >> 4) * 8) * ks + ((lane >> 3) & 1) * 8;
+    const bf16* qa = q_s + (row0 + (lane & 15)) * ks + (lane >> 4) * 8;
+    const bf16* kb = k_s + (buf * kLseKeys + half + (lane & 7) + (lane >> 4) * 8) * ks + ((lane >> 3) & 1) * 8;
 #pragma unroll(KS > 0 ? KS : 1)
     for (int k0 = 0; k0 < dk; k0 += 16) {
       uint32_t a[4];
       ldmatrix_x4(a, qa + k0);
 #pragma unroll
-      for (int n2 = 0; n2 < 4; ++n2) {
+      for (int n2 = 0; n2 < 2; ++n2) {
         uint32_t b[4];
         ldmatrix_x4(b, kb + n2 * 16 * ks + k0);
         mma_bf16(s[2 * n2], a, b[0], b[1]);
@@ -172,29 +174,29 @@ mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       if (bias.table) {
-        const float* bs = bias_s + (size_t)(buf * G + head[i]) * span + max(pos[i] - min_pos, 0) + (kLseKeys - 1) - (lane & 3) * 2;
+        const float* bs = bias_s + (size_t)(buf * G + head[i]) * span + max(pos[i] - min_pos, 0) + (kLseKeys - 1) - half - (lane & 3) * 2;
 #pragma unroll
-        for (int x = 0; x < 8; ++x) {
+        for (int x = 0; x < 4; ++x) {
           s[x][2 * i] = fmaf(s[x][2 * i], scale, bs[-x * 8]);
           s[x][2 * i + 1] = fmaf(s[x][2 * i + 1], scale, bs[-x * 8 - 1]);
         }
       } else {
 #pragma unroll
-        for (int x = 0; x < 8; ++x) {
+        for (int x = 0; x < 4; ++x) {
           s[x][2 * i] *= scale;
           s[x][2 * i + 1] *= scale;
         }
       }
       if (!whole) {
 #pragma unroll
-        for (int x = 0; x < 8; ++x)
+        for (int x = 0; x < 4; ++x)
 #pragma unroll
           for (int c = 0; c < 2; ++c)
-            if (!mask.visible(pos[i], jb + x * 8 + (lane & 3) * 2 + c)) s[x][2 * i + c] = -CUDART_INF_F;
+            if (!mask.visible(pos[i], jb + half + x * 8 + (lane & 3) * 2 + c)) s[x][2 * i + c] = -CUDART_INF_F;
       }
       float mx = -CUDART_INF_F;
 #pragma unroll
-      for (int x = 0; x < 8; ++x) mx = fmaxf(mx, fmaxf(s[x][2 * i], s[x][2 * i + 1]));
+      for (int x = 0; x < 4; ++x) mx = fmaxf(mx, fmaxf(s[x][2 * i], s[x][2 * i + 1]));
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
       const float m_new = fmaxf(m[i], mx);
@@ -202,7 +204,7 @@ mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
         const float m2 = m_new * kLog2e;
         float sum[2] = {0.f, 0.f};
 #pragma unroll
-        for (int x = 0; x < 8; ++x) {
+        for (int x = 0; x < 4; ++x) {
           sum[0] += pow2(fmaf(s[x][2 * i], kLog2e, -m2));
           sum[1] += pow2(fmaf(s[x][2 * i + 1], kLog2e, -m2));
         }
@@ -212,13 +214,25 @@ mixed_head_lse_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cac
     }
     __syncthreads();
   }
+  float* other = reinterpret_cast<float*>(smem_raw);           // [64][2]: what the second half found (the queries are read)
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
-    float sum = l[i];
-    sum += __shfl_xor_sync(0xffffffffu, sum, 1);
-    sum += __shfl_xor_sync(0xffffffffu, sum, 2);
-    const int row = r0 + warp * 16 + (lane >> 2) + 8 * i;
-    if (row < rows && (lane & 3) == 0) lse[(size_t)(t0 + row / G) * nq + kvh * G + row % G] = m[i] * kLog2e + log2f(sum);
+    l[i] += __shfl_xor_sync(0xffffffffu, l[i], 1);
+    l[i] += __shfl_xor_sync(0xffffffffu, l[i], 2);
+    const int x = row0 + (lane >> 2) + 8 * i;
+    if (half && (lane & 3) == 0) {
+      other[2 * x] = m[i];
+      other[2 * x + 1] = l[i];
+    }
+  }
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int x = row0 + (lane >> 2) + 8 * i, row = r0 + x;
+    if (half || row >= rows || (lane & 3) != 0) continue;
+    const float m_new = fmaxf(m[i], other[2 * x]);             // a row sees its own key at least: finite
+    const float sum = l[i] * pow2((m[i] - m_new) * kLog2e) + other[2 * x + 1] * pow2((other[2 * x] - m_new) * kLog2e);
+    lse[(size_t)(t0 + row / G) * nq + kvh * G + row % G] = m_new * kLog2e + log2f(sum);
   }
 }
 
@@ -811,7 +825,7 @@ extern "C" int srlm_mixed_head_attention_mma(const void* q, const void* k_cache,
     const size_t smem = mh_lse_smem(G, dk);
     auto kern = dk == 64 ? mixed_head_lse_kernel<4> : dk == 128 ? mixed_head_lse_kernel<8> : mixed_head_lse_kernel<0>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    launch_pdl(kern, dim3((unsigned)(((long long)max_q_len * G + kLseRows - 1) / kLseRows), nkv, n_entries), dim3(128),
+    launch_pdl(kern, dim3((unsigned)(((long long)max_q_len * G + kLseRows - 1) / kLseRows), nkv, n_entries), dim3(256),
                smem, stream, (const bf16*)q, (const bf16*)k_cache, lse, block_table, table_stride, cu_q, kv_lens, nq, nkv, dk,
                page_size, mh_page_shift(page_size), scale, mask, db, mh_lse_span(G));
   }
