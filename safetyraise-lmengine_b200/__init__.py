@@ -8,6 +8,7 @@ the scheduler), ``SamplingParams``, and the command line
 """
 from .config import dovorax as _dovorax
 from .config import lokizen as _lokizen
+from .config import mapovik as _mapovik
 from .config import nekedra as _nekedra
 from .config import qwen3 as _qwen3
 from .config import pabalorn as _pabalorn
@@ -29,6 +30,7 @@ register_architecture(_pabalorn.ARCHITECTURE, _pabalorn.read_spec, _build_decode
 
 register_architecture(_dovorax.ARCHITECTURE, _dovorax.read_spec, _build_decoder)
 register_architecture(_lokizen.ARCHITECTURE, _lokizen.read_spec, _build_decoder)
+register_architecture(_mapovik.ARCHITECTURE, _mapovik.read_spec, _build_decoder)
 
 __version__ = "0.1.0"
 

@@ -35,6 +35,7 @@ class PositionSpec:
     # l < original / high, divided by factor where l > original / low, and blended between the two with
     # s = (original / l - low) / (high - low): (1 - s) f / factor + s f.  None: the plain frequencies.
     scaling: Optional[Tuple[float, float, float, float]] = None
+    divisor: float = 1.0      # every frequency is divided by this (a longer context turned at a slower pace)
     # a ramp over the pair index (factor, original, fast, slow): with index(n) = rotary_dim ln(original / (2 pi n)) /
     # (2 ln theta), lo = max(floor(index(fast)), 0), hi = min(ceil(index(slow)), rotary_dim - 1) and r_i = clamp((i - lo) /
     # max(hi - lo, 0.001), 0, 1), pair i turns at f_i (1 - r_i) + f_i r_i / factor, and cos and sin are multiplied by
@@ -172,6 +173,73 @@ class DeltaRuleSpec(MixerSpec):
     norm_eps: float = 1e-6                  # of the per-head norm of the read-out
     unit_eps: float = 1e-6                  # inside the root that makes q and k unit vectors
     names: DeltaRuleNames = DeltaRuleNames()
+
+
+@dataclass(frozen=True)
+class ChannelDeltaNames:
+    q: str = "mix.q"
+    k: str = "mix.k"
+    v: str = "mix.v"
+    conv_suffix: str = ".conv"              # the short convolution of a projection: its weight's name + this
+    beta: str = "mix.b"
+    decay_down: str = "mix.a1"              # [rank, hidden]; the rank is the tensor's
+    decay_up: str = "mix.a2"                # [heads * head_dim, rank]
+    decay_log: str = "mix.A_log"            # [heads]
+    decay_bias: str = "mix.dt_bias"         # [heads * head_dim]
+    gate_down: str = "mix.g1"               # [rank, hidden]; likewise
+    gate_up: str = "mix.g2"                 # [heads * v_head_dim, rank]
+    out_norm: str = "mix.norm"              # [v_head_dim]
+    o: str = "mix.o"
+
+
+@dataclass(frozen=True)
+class ChannelDeltaSpec(MixerSpec):
+    """The gated delta rule with a decay per head and key channel, on a matrix of state S [head_dim, v_head_dim] per head:
+
+        S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+        g = exp(-exp(A_h) softplus(W_a2 W_a1 x + dt_bias)),  beta = logistic(W_b x);   q and k unit vectors, q / sqrt(head_dim)
+        out = W_o (N(w, o) * logistic(W_g2 W_g1 x))           N: each head over its root mean square
+
+    q, k and v pass a short causal convolution and silu first.  S starts at zero and is float32."""
+    hidden_size: int = 0
+    heads: int = 0                          # value heads; q / k heads are shared by heads / kv_heads of them
+    kv_heads: int = 0
+    head_dim: int = 0
+    v_head_dim: int = 0
+    conv_taps: int = 1
+    norm_eps: float = 1e-6                  # of the per-head norm of the read-out
+    unit_eps: float = 1e-6                  # inside the root that makes q and k unit vectors
+    names: ChannelDeltaNames = ChannelDeltaNames()
+
+
+@dataclass(frozen=True)
+class StateSpaceNames:
+    inp: str = "mix.in"                     # [2 inner + 2 groups * state + heads, hidden]: z, x, B, C, dt rows
+    conv: str = "mix.conv"                  # [inner + 2 groups * state, taps]; its bias: this name + ".b"
+    dt_bias: str = "mix.dt_bias"            # [heads]
+    a_log: str = "mix.A_log"                # [heads]
+    d: str = "mix.D"                        # [heads]
+    out_norm: str = "mix.norm"              # [inner]
+    o: str = "mix.o"
+
+
+@dataclass(frozen=True)
+class StateSpaceSpec(MixerSpec):
+    """A state space with one decay a head (inner = heads * head_dim; head h uses B and C of group h // (heads / groups)):
+
+        S <- exp(-exp(A_h) dt) S + dt B x^T;   y = S^T C + D_h x,   S [state, head_dim],   dt = softplus(dt_in + dt_bias)
+        out = W_o N(w, y * silu(z))            N: each of norm_parts equal parts over its root mean square
+
+    x, B and C pass a short causal convolution with a bias and silu first.  S starts at zero and is float32."""
+    hidden_size: int = 0
+    heads: int = 0
+    head_dim: int = 0
+    state: int = 0
+    groups: int = 1
+    norm_parts: int = 1
+    conv_taps: int = 1
+    norm_eps: float = 1e-6
+    names: StateSpaceNames = StateSpaceNames()
 
 
 @dataclass(frozen=True)
@@ -461,7 +529,7 @@ class DenseNames:
 
 @dataclass(frozen=True)
 class DenseSpec(FeedForwardSpec):
-    """down(act(up(x))): no gate.  ``activation``: "gelu" (the exact one, with erf)."""
+    """down(act(up(x))): no gate.  ``activation``: "gelu" (the exact one, with erf) or "relu_squared" (max(z, 0)^2)."""
     dense_names: DenseNames = DenseNames()
 
 
@@ -471,6 +539,7 @@ class RoutedExpertsNames:
     router: str = "mlp.router"
     router_bias: str = "mlp.router.b"
     correction: str = "mlp.correction"      # [experts]
+    table: str = "mlp.table"                # [vocab, top], integers: scoring "table"
     expert: str = "mlp.e{}."
     shared: str = "mlp.shared."
     gate: str = "gate"
@@ -496,6 +565,7 @@ class RoutedExpertsSpec(FeedForwardSpec):
     # "softmax_over_all": scores = softmax over every expert's logit; the experts form ``groups`` equal groups of
     # neighbours, a group counts as its largest score, only experts of the best ``groups_kept`` groups can be chosen;
     # weights = the chosen scores over their sum (+ 1e-20).
+    # "table": no router; a table of ``vocab`` rows gives each token id its ``top`` experts, each with the weight 1 / top.
     scoring: str = "softmax_of_chosen"
     weight_on_input: bool = False           # a weight multiplies its expert's input instead of its output
     groups: int = 1
@@ -505,6 +575,7 @@ class RoutedExpertsSpec(FeedForwardSpec):
     correction: bool = False                # scoring "logistic": the experts are chosen by their scores plus a learned number
                                             # each; the weights are the scores without it
     weight_scale: float = 1.0               # a factor on every weight
+    vocab: int = 0                          # scoring "table": rows of the table
     expert_names: RoutedExpertsNames = RoutedExpertsNames()
 
 
@@ -526,6 +597,7 @@ class LayerSpec:
     mixer_gate_name: str = "rg1"             # weight [hidden, hidden]; its bias: this name + ".b"
     feed_forward_gate_name: str = "rg2"
     residual_scale: float = 1.0              # block "post_norm": x <- norm(residual_scale * x + sublayer(x))
+    sublayer_scale: float = 1.0              # block "pre_norm": x <- x + sublayer_scale * sublayer(norm(x))
 
 
 @dataclass(frozen=True)
@@ -536,6 +608,9 @@ class RunStep:
     writes_cache: bool = True  # False: reads what another step wrote under ``cache``
     more_caches: Tuple[int, ...] = ()   # a mixer made of several (side by side): the entries of the second, third, ...
     add_embedding: bool = False         # what the embedding left (the stream ahead of the first run step) joins the stream first
+    # the step begins a pass: x <- W [x; x_0] + v_p first, W the model's entry product, x_0 what the embedding left, v_p
+    # row p of the model's table of pass vectors; None: it does not
+    begins_pass: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -558,10 +633,17 @@ class ModelSpec:
     embed_norm_name: str = "embed.norm"
     embed_scale: float = 1.0                        # a factor on the embedded tokens
     logit_softcap: Optional[float] = None           # logits <- cap * tanh(logits / cap)
+    logit_scale: float = 1.0                        # a factor on the logits (ahead of the cap)
+    pass_product_name: str = "loop.in"              # [hidden, 2 hidden], run steps with begins_pass: columns of x, of x_0
+    pass_vectors_name: str = "loop.step"            # [passes, hidden]
     extra: dict = field(default_factory=dict, compare=False)
 
     def to_json(self) -> dict:
         return asdict(self)
+
+    @property
+    def num_passes(self) -> int:
+        return max((s.begins_pass + 1 for s in self.run_order if s.begins_pass is not None), default=0)
 
     @property
     def num_cache_entries(self) -> int:

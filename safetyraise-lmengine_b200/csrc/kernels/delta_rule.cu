@@ -221,11 +221,11 @@ delta_recurrence_kernel(const float* __restrict__ qkv, const float* __restrict__
   }
 }
 
-// One block per token, a warp per head: o / sqrt(mean(o^2) + eps) * w * silu(gate).
+// One block per token, a warp per head: o / sqrt(mean(o^2) + eps) * w * silu(gate), or logistic(gate) in silu's place.
 template <typename TP, typename TA>
 __global__ void delta_output_kernel(const float* __restrict__ o, const float* __restrict__ norm_w, float eps,
                                     const TP* __restrict__ proj, long long ldp, int gate_off, TA* __restrict__ out,
-                                    int H, int dv) {
+                                    int H, int dv, int logistic) {
   pdl_wait();        // launched as a dependent of the kernel ahead: nothing is read before it has finished
   pdl_trigger();
   const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
@@ -236,7 +236,7 @@ __global__ void delta_output_kernel(const float* __restrict__ o, const float* __
     const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)dv + eps);
     for (int d = lane; d < dv; d += 32) {
       const float z = to_float(proj[(size_t)t * ldp + gate_off + (size_t)h * dv + d]);
-      out[((size_t)t * H + h) * dv + d] = from_float<TA>(row[d] * inv * norm_w[d] * (z / (1.f + expf(-z))));
+      out[((size_t)t * H + h) * dv + d] = from_float<TA>(row[d] * inv * norm_w[d] * ((logistic ? 1.f : z) / (1.f + expf(-z))));
     }
   }
 }
@@ -304,13 +304,13 @@ extern "C" int srlm_delta_recurrence(const float* qkv, const float* beta, const 
 
 extern "C" int srlm_delta_output(const float* o, const float* norm_w, float eps, const void* proj, int proj_dtype,
                                  long long ldp, int gate_off, void* out, int out_dtype, int T, int H, int dv,
-                                 cudaStream_t stream) {
+                                 int logistic, cudaStream_t stream) {
   if (T <= 0) return ST_OK;
   if (H <= 0 || dv <= 0 || !(eps > 0.f) || gate_off < 0 || ldp < gate_off + (long long)H * dv)
     return refuse(ST_BAD_SIZE, "delta_output: H=%d dv=%d gate_off=%d ldp=%lld", H, dv, gate_off, ldp);
   const int threads = 32 * (H < 8 ? H : 8);
 #define SRLM_DELTA_OUT(TP, TA)                                                                                    \
-  launch_pdl(delta_output_kernel<TP, TA>, dim3(T), dim3(threads), 0, stream, o, norm_w, eps, (const TP*)proj, ldp, gate_off, (TA*)out, H, dv)
+  launch_pdl(delta_output_kernel<TP, TA>, dim3(T), dim3(threads), 0, stream, o, norm_w, eps, (const TP*)proj, ldp, gate_off, (TA*)out, H, dv, logistic)
   if (proj_dtype == DT_F32 && out_dtype == DT_F32) SRLM_DELTA_OUT(float, float);
   else if (proj_dtype == DT_F32 && out_dtype == DT_BF16) SRLM_DELTA_OUT(float, bf16);
   else if (proj_dtype == DT_BF16 && out_dtype == DT_BF16) SRLM_DELTA_OUT(bf16, bf16);

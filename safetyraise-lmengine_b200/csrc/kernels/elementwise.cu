@@ -1,4 +1,4 @@
-// Embedding gather, residual-add + RMSNorm, SwiGLU and casts.
+// Embedding gather, residual-add + RMSNorm or layer norm, SwiGLU and casts.
 //
 // The residual stream is float32 in every mode; norms reduce in float32 in an
 // order fixed by the row width alone, so a row's result does not depend on
@@ -41,12 +41,13 @@ __global__ void embed_gather_kernel(const int* __restrict__ ids, const TW* __res
   }
 }
 
-// x = residual[src] (+ delta[src]); residual[src] = x when rows == nullptr;
-// out[r] = x * rsqrt(mean(x^2) + eps) * (w (+1)).
-template <typename TA>
-__global__ void add_rmsnorm_kernel(float* __restrict__ residual, const TA* __restrict__ delta,
-                                   const float* __restrict__ weight, float eps, TA* __restrict__ out,
-                                   const int* __restrict__ rows, int H, int unit_offset) {
+// x = residual[src] (+ delta_scale * delta[src]); residual[src] = x when rows == nullptr;
+// out[r] = x * rsqrt(mean(x^2) + eps) * (w (+1)).  CENTER: the mean of the row is taken off x first (layer norm: the
+// residual keeps it), so that the second moment is the variance.
+template <typename TA, bool CENTER>
+__global__ void add_norm_kernel(float* __restrict__ residual, const TA* __restrict__ delta, float delta_scale,
+                                const float* __restrict__ weight, float eps, TA* __restrict__ out,
+                                const int* __restrict__ rows, int H, int unit_offset) {
   __shared__ float scratch[32];
   pdl_wait();
   pdl_trigger();
@@ -54,23 +55,33 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ residual, const TA* __res
   const size_t src = rows ? (size_t)rows[r] : (size_t)r;
   float* res = residual + src * H;
   const TA* del = delta ? delta + src * H : nullptr;
-  float ss = 0.f;
+  float ss = 0.f, sum = 0.f;
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
     float x = res[i];
     if (del) {
-      x += to_float(del[i]);
+      x = fmaf(delta_scale, to_float(del[i]), x);
       if (!rows) res[i] = x;
     }
-    ss += x * x;
+    if (CENTER) sum += x;
+    else ss += x * x;
+  }
+  float mean = 0.f;
+  if (CENTER) {
+    mean = block_sum(sum, scratch) / (float)H;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+      float x = res[i];
+      if (del && rows) x = fmaf(delta_scale, to_float(del[i]), x);
+      ss += (x - mean) * (x - mean);
+    }
   }
   const float total = block_sum(ss, scratch);
   const float inv = 1.0f / sqrtf(total / (float)H + eps);
   TA* o = out + (size_t)r * H;
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
     float x = res[i];
-    if (del && rows) x += to_float(del[i]);
+    if (del && rows) x = fmaf(delta_scale, to_float(del[i]), x);
     const float w = weight[i] + (unit_offset ? 1.f : 0.f);
-    o[i] = from_float<TA>(x * inv * w);
+    o[i] = from_float<TA>((CENTER ? x - mean : x) * inv * w);
   }
 }
 
@@ -78,10 +89,11 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ residual, const TA* __res
 // pieces; a thread keeps up to CACHE pieces in registers, so a row of up to 4 * CACHE * blockDim elements
 // is read once.  The sum of squares adds a thread's elements in index order, then the threads in the
 // order of block_sum: fixed by the width.
-template <int CACHE>
+template <int CACHE, bool CENTER>
 __global__ void __launch_bounds__(1024)
-add_rmsnorm_vec_kernel(float* __restrict__ residual, const bf16* __restrict__ delta, const float* __restrict__ weight,
-                       float eps, bf16* __restrict__ out, const int* __restrict__ rows, int H, int unit_offset) {
+add_norm_vec_kernel(float* __restrict__ residual, const bf16* __restrict__ delta, float delta_scale,
+                    const float* __restrict__ weight, float eps, bf16* __restrict__ out, const int* __restrict__ rows, int H,
+                    int unit_offset) {
   __shared__ float scratch[32];
   pdl_wait();
   pdl_trigger();
@@ -91,7 +103,7 @@ add_rmsnorm_vec_kernel(float* __restrict__ residual, const bf16* __restrict__ de
   const uint2* del = delta ? reinterpret_cast<const uint2*>(delta + src * H) : nullptr;
   const int pieces = H / 4;
   float4 x[CACHE];
-  float ss = 0.f;
+  float ss = 0.f, sum = 0.f;
 #pragma unroll
   for (int c = 0; c < CACHE; ++c) {
     const int i = threadIdx.x + c * blockDim.x;
@@ -101,11 +113,23 @@ add_rmsnorm_vec_kernel(float* __restrict__ residual, const bf16* __restrict__ de
         const uint2 d = del[i];
         const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&d.x));
         const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&d.y));
-        v.x += lo.x; v.y += lo.y; v.z += hi.x; v.w += hi.y;
+        v.x = fmaf(delta_scale, lo.x, v.x); v.y = fmaf(delta_scale, lo.y, v.y);
+        v.z = fmaf(delta_scale, hi.x, v.z); v.w = fmaf(delta_scale, hi.y, v.w);
         if (!rows) res[i] = v;
       }
-      ss += v.x * v.x; ss += v.y * v.y; ss += v.z * v.z; ss += v.w * v.w;
+      if (CENTER) sum += (v.x + v.y) + (v.z + v.w);
+      else { ss += v.x * v.x; ss += v.y * v.y; ss += v.z * v.z; ss += v.w * v.w; }
       x[c] = v;
+    }
+  }
+  if (CENTER) {
+    const float mean = block_sum(sum, scratch) / (float)H;
+#pragma unroll
+    for (int c = 0; c < CACHE; ++c) {
+      if (threadIdx.x + c * blockDim.x < pieces) {
+        x[c].x -= mean; x[c].y -= mean; x[c].z -= mean; x[c].w -= mean;
+        ss += x[c].x * x[c].x; ss += x[c].y * x[c].y; ss += x[c].z * x[c].z; ss += x[c].w * x[c].w;
+      }
     }
   }
   const float total = block_sum(ss, scratch);
@@ -168,9 +192,42 @@ __global__ void cast_columns_kernel(const float* __restrict__ in, long long ld, 
 
 // out[t] += delta[t]  (float32 residual, any activation type)
 template <typename TA>
-__global__ void residual_add_kernel(float* __restrict__ residual, const TA* __restrict__ delta, size_t n) {
+__global__ void residual_add_kernel(float* __restrict__ residual, const TA* __restrict__ delta, float scale, size_t n) {
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x)
-    residual[i] += to_float(delta[i]);
+    residual[i] = fmaf(scale, to_float(delta[i]), residual[i]);
+}
+
+// The stream beside the embedding, a product's input: x = residual[t] (+ scale * delta[t]), x0 = the token's row of the
+// table times table_scale (or kept[t], when given).  float32: out[t] = [x | x0].  bfloat16: out[t] = [hi | lo | x0] with
+// hi = x rounded and lo = the rounded rest, so that a product whose weights repeat the columns of x sees 16 bits of it.
+template <typename TA, typename TW>
+__global__ void stream_beside_embedding_kernel(const float* __restrict__ residual, const TA* __restrict__ delta, float scale,
+                                               const int* __restrict__ ids, const TW* __restrict__ table, float table_scale,
+                                               int vocab, const float* __restrict__ kept, TA* __restrict__ out, int H) {
+  pdl_wait();
+  pdl_trigger();
+  constexpr bool kSplit = sizeof(TA) == 2;
+  const size_t t = blockIdx.x;
+  const int id = ids[t];
+  const bool known = id >= 0 && id < vocab;           // the gather has raised the step's fault word for any other
+  TA* o = out + t * H * (kSplit ? 3 : 2);
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    float x = residual[t * H + i];
+    if (delta) x = fmaf(scale, to_float(delta[t * H + i]), x);
+    const TA hi = from_float<TA>(x);
+    o[i] = hi;
+    if (kSplit) o[H + i] = from_float<TA>(x - to_float(hi));
+    const float x0 = kept ? kept[t * H + i] : known ? to_float(table[(size_t)id * H + i]) * table_scale : 0.f;
+    o[(size_t)H * (kSplit ? 2 : 1) + i] = from_float<TA>(x0);
+  }
+}
+
+// residual[t] += row, for every t
+__global__ void add_row_kernel(float* __restrict__ residual, const float* __restrict__ row, int H, size_t n) {
+  pdl_wait();
+  pdl_trigger();
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x)
+    residual[i] += row[i % H];
 }
 
 // flag[0] = 1 if any a[i] (+ b[i], when b is given) is NaN or infinite.
@@ -220,11 +277,12 @@ extern "C" int srlm_embed_gather(const int* ids, const void* table, int table_dt
   return launched();
 }
 
-extern "C" int srlm_add_rmsnorm(float* residual, const void* delta, const float* weight, float eps,
-                                void* out, int act_dtype, const int* rows, int R, int H, int unit_offset,
-                                cudaStream_t stream) {
+// center: layer norm (the row's mean is taken off first); delta_scale: a factor on delta
+extern "C" int srlm_add_norm(float* residual, const void* delta, float delta_scale, const float* weight, float eps,
+                             void* out, int act_dtype, const int* rows, int R, int H, int unit_offset, int center,
+                             cudaStream_t stream) {
   if (R <= 0) return ST_OK;
-  if (H <= 0 || !(eps > 0.f)) return refuse(ST_BAD_SIZE, "add_rmsnorm: H=%d eps=%g", H, (double)eps);
+  if (H <= 0 || !(eps > 0.f)) return refuse(ST_BAD_SIZE, "add_norm: H=%d eps=%g", H, (double)eps);
   if (act_dtype == DT_BF16 && H % 4 == 0 && H <= 4 * 4 * 1024 &&
       (((uintptr_t)residual | (uintptr_t)weight) & 15) == 0 && (((uintptr_t)delta | (uintptr_t)out) & 7) == 0) {
     // whole rows in registers: one read of the residual, vector loads and stores
@@ -234,19 +292,25 @@ extern "C" int srlm_add_rmsnorm(float* residual, const void* delta, const float*
     int block = 32;
     while (block < 1024 && block * 4 < pieces) block <<= 1;
     const int per_thread = (pieces + block - 1) / block;
-    if (per_thread <= 1)
-      launch_pdl(add_rmsnorm_vec_kernel<1>, dim3(R), dim3(block), 0, stream, residual, (const bf16*)delta, weight, eps,
-                 (bf16*)out, rows, H, unit_offset);
-    else if (per_thread <= 2)
-      launch_pdl(add_rmsnorm_vec_kernel<2>, dim3(R), dim3(block), 0, stream, residual, (const bf16*)delta, weight, eps,
-                 (bf16*)out, rows, H, unit_offset);
-    else
-      launch_pdl(add_rmsnorm_vec_kernel<4>, dim3(R), dim3(block), 0, stream, residual, (const bf16*)delta, weight, eps,
-                 (bf16*)out, rows, H, unit_offset);
+#define SRLM_NORM_VEC(C)                                                                                                    \
+  do {                                                                                                                      \
+    if (center) launch_pdl(add_norm_vec_kernel<C, true>, dim3(R), dim3(block), 0, stream, residual, (const bf16*)delta,    \
+                           delta_scale, weight, eps, (bf16*)out, rows, H, unit_offset);                                    \
+    else launch_pdl(add_norm_vec_kernel<C, false>, dim3(R), dim3(block), 0, stream, residual, (const bf16*)delta,          \
+                    delta_scale, weight, eps, (bf16*)out, rows, H, unit_offset);                                           \
+  } while (0)
+    if (per_thread <= 1) SRLM_NORM_VEC(1);
+    else if (per_thread <= 2) SRLM_NORM_VEC(2);
+    else SRLM_NORM_VEC(4);
+#undef SRLM_NORM_VEC
     return launched();
   }
-  SRLM_DISPATCH_ACT(act_dtype, TA, launch_pdl(add_rmsnorm_kernel<TA>, dim3(R), dim3(norm_block(H)), 0, stream,
-      residual, (const TA*)delta, weight, eps, (TA*)out, rows, H, unit_offset));
+  SRLM_DISPATCH_ACT(act_dtype, TA, {
+    if (center) launch_pdl(add_norm_kernel<TA, true>, dim3(R), dim3(norm_block(H)), 0, stream, residual, (const TA*)delta,
+                           delta_scale, weight, eps, (TA*)out, rows, H, unit_offset);
+    else launch_pdl(add_norm_kernel<TA, false>, dim3(R), dim3(norm_block(H)), 0, stream, residual, (const TA*)delta,
+                    delta_scale, weight, eps, (TA*)out, rows, H, unit_offset);
+  });
   return launched();
 }
 
@@ -283,11 +347,32 @@ extern "C" int srlm_cast_columns(const float* in, long long ld, void* out, int o
   return launched();
 }
 
-extern "C" int srlm_residual_add(float* residual, const void* delta, int act_dtype, long long n,
+extern "C" int srlm_residual_add(float* residual, const void* delta, int act_dtype, float scale, long long n,
                                  cudaStream_t stream) {
   if (n <= 0) return ST_OK;
   SRLM_DISPATCH_ACT(act_dtype, TA, (residual_add_kernel<TA><<<flat_grid((size_t)n, 256), 256, 0, stream>>>(
-      residual, (const TA*)delta, (size_t)n)));
+      residual, (const TA*)delta, scale, (size_t)n)));
+  return launched();
+}
+
+// delta (act_dtype) or null; table [vocab, H] (float32 or bfloat16), not read when kept (float32 [T, H]) is given; out
+// [T, 2 H] in float32 or [T, 3 H] in bfloat16
+extern "C" int srlm_stream_beside_embedding(const float* residual, const void* delta, float scale, const int* ids,
+                                            const void* table, int table_dtype, float table_scale, int vocab,
+                                            const float* kept, void* out, int act_dtype, int T, int H, cudaStream_t stream) {
+  if (T <= 0) return ST_OK;
+  if (H <= 0 || vocab <= 0) return refuse(ST_BAD_SIZE, "stream_beside_embedding: H=%d vocab=%d", H, vocab);
+  SRLM_DISPATCH_ACT(act_dtype, TA, SRLM_DISPATCH_ACT(table_dtype, TW, launch_pdl(stream_beside_embedding_kernel<TA, TW>,
+      dim3(T), dim3(H >= 1024 ? 256 : 128), 0, stream, residual, (const TA*)delta, scale, ids, (const TW*)table, table_scale,
+      vocab, kept, (TA*)out, H)));
+  return launched();
+}
+
+extern "C" int srlm_add_row(float* residual, const float* row, int T, int H, cudaStream_t stream) {
+  if (T <= 0) return ST_OK;
+  if (H <= 0) return refuse(ST_BAD_SIZE, "add_row: H=%d", H);
+  const size_t n = (size_t)T * H;
+  launch_pdl(add_row_kernel, dim3(flat_grid(n, 256)), dim3(256), 0, stream, residual, row, H, n);
   return launched();
 }
 

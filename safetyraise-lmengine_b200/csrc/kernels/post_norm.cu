@@ -68,7 +68,7 @@ __global__ void activation_kernel(const TI* __restrict__ in, long long ld, const
   for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
     const size_t t = idx / F, f = idx - t * F;
     const float z = to_float(in[t * ld + f]) + (bias ? bias[f] : 0.f);
-    out[idx] = from_float<TO>(kind == 0 ? gelu_erf_f(z) : gelu_tanh_f(z));
+    out[idx] = from_float<TO>(kind == 2 ? (z < 0.f ? 0.f : z * z) : kind == 0 ? gelu_erf_f(z) : gelu_tanh_f(z));
   }
 }
 
@@ -130,7 +130,7 @@ extern "C" int srlm_rmsnorm_columns(const float* in, long long ld, const float* 
 extern "C" int srlm_activation(const void* in, int in_dtype, long long ld, const float* bias, void* out, int out_dtype,
                                int T, int F, int kind, cudaStream_t stream) {
   if (T <= 0) return ST_OK;
-  if (F <= 0 || ld < F || kind < 0 || kind > 1) return refuse(ST_BAD_SIZE, "activation: F=%d ld=%lld kind=%d", F, ld, kind);
+  if (F <= 0 || ld < F || kind < 0 || kind > 2) return refuse(ST_BAD_SIZE, "activation: F=%d ld=%lld kind=%d", F, ld, kind);
   const size_t total = (size_t)T * F;
   const unsigned grid = (unsigned)((total + 255) / 256 < 4096 ? (total + 255) / 256 : 4096);
   SRLM_TWO_TYPES(in_dtype, out_dtype, TI, TO, launch_pdl(activation_kernel<TI, TO>, dim3(grid), dim3(256), 0, stream,

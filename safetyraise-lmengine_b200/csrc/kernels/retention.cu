@@ -17,7 +17,7 @@
 //   retention_read     o_t = decay^(t + 1) S_c^T q_t + sum_(s <= t) decay^(t - s) (q_t . k_s) v_s, norm and gate
 // The decays are known ahead, so nothing but the fold runs along the tokens.  All sums are float32 FMAs: what enters the
 // recurrence is 32-bit by design.  Two FMAs of neighbouring columns are one packed instruction (fma.rn.f32x2).
-#include "common.cuh"
+#include "state_walk.cuh"
 
 namespace srlm {
 
@@ -133,15 +133,6 @@ retention_walk_kernel(const float* __restrict__ proj, long long ldp, const float
 
 // ---- chunks ------------------------------------------------------------------------------------------------------------
 constexpr int kRetChunk = 64;
-
-__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
-  unsigned long long d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;"
-      : "=l"(d)
-      : "l"(*reinterpret_cast<unsigned long long*>(&a)), "l"(*reinterpret_cast<unsigned long long*>(&b)),
-        "l"(*reinterpret_cast<unsigned long long*>(&c)));
-  return *reinterpret_cast<float2*>(&d);
-}
 
 // decay^n, formed in double precision and rounded once.
 __device__ __forceinline__ float decay_power(float decay, int n) {

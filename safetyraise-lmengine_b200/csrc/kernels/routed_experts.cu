@@ -1,7 +1,8 @@
 // A feed-forward of routed experts: every token runs the `top` experts with the largest router logits and
 // adds their outputs, weighted by the softmax over those logits alone (scoring 0), or by the logistic of each
 // chosen logit, not renormalised (scoring 1), or by the softmax over ALL experts' logits, renormalised over the chosen
-// ones (scoring 2; the experts may then form equal groups of neighbours of which only the best few, judged by their
+// ones (scoring 2), or, without a router, the experts that a table lists for its token id, with equal weights
+// (scoring 2: the experts may form equal groups of neighbours of which only the best few, judged by their
 // largest score, can be chosen).  A weight multiplies its expert's output (in `combine`) or, for
 // experts without biases, its input: then the first grouped product scales its gate and up sums by the pair's
 // weight before the activation (W (w h) = w (W h)), and `combine` adds the rows as they are.
@@ -126,6 +127,24 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, lo
   __syncwarp();
 }
 
+// No router: a table [vocab, top] names the experts of every token id, each with the weight `share`.  An id outside the
+// table (the embedding has raised the step's fault word) takes the first row; an entry outside [0, E) becomes expert 0.
+__device__ __forceinline__ void look_up_pair(const int* __restrict__ ids, const int* __restrict__ table, int vocab, int E, int top,
+                                             int pair, float share, int* __restrict__ choice, float* __restrict__ weight) {
+  const int id = ids[pair / top];
+  const int e = table[(size_t)(id >= 0 && id < vocab ? id : 0) * top + pair % top];
+  choice[pair] = e >= 0 && e < E ? e : 0;
+  weight[pair] = share;
+}
+
+__global__ void moe_look_up_kernel(const int* __restrict__ ids, const int* __restrict__ table, int vocab, int E, int top, int n,
+                                   float share, int* __restrict__ choice, float* __restrict__ weight) {
+  pdl_wait();
+  pdl_trigger();
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < n) look_up_pair(ids, table, vocab, E, top, i, share, choice, weight);
+}
+
 __global__ void moe_route_kernel(const float* __restrict__ logits, long long ld, const float* __restrict__ bias,
                                  int T, int E, int top, int* __restrict__ choice, float* __restrict__ weight, int scoring,
                                  int groups, int kept, const float* __restrict__ correction, float wscale) {
@@ -146,13 +165,15 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, long long ld,
 // operands); pair_of_row then has rows_cap entries, -1 where a row holds no pair, and group_of_tile[max_tiles]
 // names the expert of every tile, -1 for a tile without rows.
 // logits != null: the block first routes the n / top tokens itself (small steps: one launch fewer), a warp a
-// token at a time, and writes choice and weight; then it orders what it chose.
+// token at a time, and writes choice and weight; then it orders what it chose.  table != null: likewise, by looking the
+// token ids up (weight: wscale each).
 __global__ void moe_sort_kernel(int* __restrict__ choice, int n, int E, int tile_rows, int align,
                                 int* __restrict__ offsets, int* __restrict__ tiles, int* __restrict__ pair_of_row,
                                 int* __restrict__ row_of_pair, int* __restrict__ group_of_tile, int max_tiles, int rows_cap,
                                 const float* __restrict__ logits, long long ld, const float* __restrict__ bias, int top,
                                 float* __restrict__ weight, int scoring, int groups, int kept,
-                                const float* __restrict__ correction, float wscale) {
+                                const float* __restrict__ correction, float wscale, const int* __restrict__ ids,
+                                const int* __restrict__ table, int vocab) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ int sort_smem[];
@@ -163,6 +184,9 @@ __global__ void moe_sort_kernel(int* __restrict__ choice, int n, int E, int tile
     for (int t = threadIdx.x >> 5; t < n / top; t += blockDim.x >> 5)
       route_token(logits, ld, bias, t, E, top, z, choice, weight, scoring, groups, kept, correction, wscale);
     __syncthreads();                 // the choices of all tokens are written (and visible to the block)
+  } else if (table) {
+    for (int i = threadIdx.x; i < n; i += blockDim.x) look_up_pair(ids, table, vocab, E, top, i, wscale, choice, weight);
+    __syncthreads();
   }
   for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = 0;
   if (align) {
@@ -519,19 +543,33 @@ extern "C" int srlm_moe_route(const float* logits, long long ld, const float* bi
   return launched();
 }
 
+// ids int32 [T]; table int32 [vocab, top]; choice int32 [T, top], weight float32 [T, top] (share each)
+extern "C" int srlm_moe_look_up(const int* ids, const int* table, int vocab, int T, int E, int top, float share, int* choice,
+                                float* weight, cudaStream_t stream) {
+  if (T <= 0) return ST_OK;
+  if (vocab <= 0 || E <= 0 || top <= 0 || top > E) return refuse(ST_BAD_SIZE, "moe_look_up: vocab=%d experts=%d top=%d", vocab, E, top);
+  const int n = T * top;
+  launch_pdl(moe_look_up_kernel, dim3((n + 255) / 256), dim3(256), 0, stream, ids, table, vocab, E, top, n, share, choice, weight);
+  return launched();
+}
+
 // choice int32 [n] (n = tokens x top); offsets, tiles int32 [E + 1]; pair_of_row, row_of_pair int32 [n]
 // tile_rows 0: the tiles of the grouped kernels of this file, rows packed.  tile_rows > 0: every expert's rows
 // start at a multiple of it; group_of_tile [max_tiles >= (n + E * (tile_rows - 1)) / tile_rows] names each tile's
 // expert (-1: none) and pair_of_row has rows_cap >= max_tiles * tile_rows entries (-1: no pair).
 // logits (float32 [n / top, ld >= E], with bias [E] or null) given: the kernel routes the tokens first and
 // writes choice and weight [n / top, top] itself; offered for E <= 256 (srlm_moe_sort_routes).
+// table (int32 [vocab, top]) with ids (int32 [n / top]) given: likewise, by looking the ids up; every weight weight_scale.
 extern "C" int srlm_moe_sort_routes(int tokens, int E) { return tokens <= 512 && E <= 256; }
 
 extern "C" int srlm_moe_sort(int* choice, int n, int E, int* offsets, int* tiles, int* pair_of_row,
                              int* row_of_pair, int tile_rows, int* group_of_tile, int max_tiles, int rows_cap,
                              const float* logits, long long ld, const float* bias, int top, float* weight, int scoring,
-                             int groups, int kept, const float* correction, float weight_scale, cudaStream_t stream) {
+                             int groups, int kept, const float* correction, float weight_scale, const int* ids,
+                             const int* table, int vocab, cudaStream_t stream) {
   if (n <= 0) return ST_OK;
+  if (table && (logits || !ids || !weight || vocab <= 0 || top <= 0 || n % top))
+    return refuse(ST_BAD_SIZE, "moe_sort: a table of %d token ids, top=%d, %d pairs", vocab, top, n);
   if (E <= 0 || E > 4096) return refuse(ST_BAD_SIZE, "moe_sort: experts=%d (at most 4096)", E);
   if (logits)
     if (int r = routing_ok("moe_sort", E, top, scoring, groups, kept)) return r;
@@ -546,7 +584,7 @@ extern "C" int srlm_moe_sort(int* choice, int n, int E, int* offsets, int* tiles
   const size_t smem = (size_t)(2 * E + 1) * sizeof(int) + (logits ? (size_t)32 * E * sizeof(float) : 0);
   launch_pdl(moe_sort_kernel, dim3(1), dim3(1024), smem, stream, choice, n, E,
              align ? tile_rows : kTile, align, offsets, tiles, pair_of_row, row_of_pair, group_of_tile, max_tiles, rows_cap,
-             logits, ld, bias, top, weight, scoring, groups, kept, correction, weight_scale);
+             logits, ld, bias, top, weight, scoring, groups, kept, correction, weight_scale, ids, table, vocab);
   return launched();
 }
 

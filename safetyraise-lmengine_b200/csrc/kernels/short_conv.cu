@@ -7,51 +7,28 @@
 // leaves the last taps - 1 inputs of every channel after each step ([taps - 1][C] floats at state_off of the slot's row,
 // oldest first; zeros for a new request).  So a request may be cut anywhere, down to single tokens.
 //
-//   short_conv             y as float32 (and, optionally, a copy in the activation dtype)
+//   short_conv             y, or silu(y), as float32 (and, optionally, a copy in the activation dtype)
 //   conv_carry             renews the slots' carried inputs; runs behind every kernel that reads them
 //   conv_norm_rope_append  for an attention whose q, k and v each pass such a convolution: convolution, RMS norm per head
 //                          of q and k, rotation of their leading pairs, q to its buffer and k, v to the pages, in one kernel
-#include "common.cuh"
+#include "state_walk.cuh"
 
 namespace srlm {
 
 constexpr int kMaxTaps = 16;
 
-struct ConvInput {
-  const float* proj;        // [T, ld], the channels' columns start at proj
-  long long ld;
-  const float* in_bias;     // [C] or null: added to every input of the step (the carried ones hold it already)
-  const float* state;       // [slots, state_stride]
-  long long state_stride;
-  int state_off;
-  int taps, C;
-};
-
-// The convolution of channel c at token t, which is token `idx` of its entry's portion.
-__device__ __forceinline__ float conv_at(const ConvInput& in, const float* __restrict__ w, int t, int idx, int slot, int c) {
-  float acc = 0.f;
-  const float bias = in.in_bias ? in.in_bias[c] : 0.f;
-  for (int j = 0; j < in.taps; ++j) {
-    const int back = in.taps - 1 - j;
-    float u;
-    if (back <= idx) u = in.proj[(size_t)(t - back) * in.ld + c] + bias;
-    else u = in.state[(size_t)slot * in.state_stride + in.state_off + (size_t)(in.taps - 1 - (back - idx)) * in.C + c];
-    acc = fmaf(w[(size_t)c * in.taps + j], u, acc);
-  }
-  return acc;
-}
-
 template <typename TO>
 __global__ void short_conv_kernel(ConvInput in, const float* __restrict__ w, const float* __restrict__ out_bias,
                                   const int* __restrict__ entry_of_token, const int* __restrict__ cu_q,
-                                  const int* __restrict__ slots, float* __restrict__ out, TO* __restrict__ out_low, int T) {
+                                  const int* __restrict__ slots, float* __restrict__ out, TO* __restrict__ out_low, int T, int silu) {
   pdl_wait();
   pdl_trigger();
   const int t = blockIdx.y;
   const int e = entry_of_token[t];
   const int idx = t - cu_q[e], slot = slots[e];
   for (int c = blockIdx.x * blockDim.x + threadIdx.x; c < in.C; c += gridDim.x * blockDim.x) {
-    const float y = conv_at(in, w, t, idx, slot, c) + (out_bias ? out_bias[c] : 0.f);
+    float y = conv_at(in, w, t, idx, slot, c) + (out_bias ? out_bias[c] : 0.f);
+    if (silu) y = silu_of(y);
     out[(size_t)t * in.C + c] = y;
     if (out_low) out_low[(size_t)t * in.C + c] = from_float<TO>(y);
   }
@@ -154,11 +131,12 @@ static int conv_input_ok(const char* what, int taps, int C, long long ld, long l
   return ST_OK;
 }
 
-// proj float32 [T, ld] (the channels' first column at proj); w float32 [C, taps]; out float32 [T, C]; out_low [T, C] or null
+// proj float32 [T, ld] (the channels' first column at proj); w float32 [C, taps]; out float32 [T, C]; out_low [T, C] or null;
+// silu: y * logistic(y) instead of y
 extern "C" int srlm_short_conv(const float* proj, long long ld, const float* in_bias, const float* w, const float* out_bias,
                                const float* state, long long state_stride, int state_off, const int* entry_of_token,
                                const int* cu_q, const int* slots, float* out, void* out_low, int low_dtype, int T, int C,
-                               int taps, cudaStream_t stream) {
+                               int taps, int silu, cudaStream_t stream) {
   if (T <= 0) return ST_OK;
   if (int r = conv_input_ok("short_conv", taps, C, ld, state_stride, state_off)) return r;
   ConvInput in{proj, ld, in_bias, state, state_stride, state_off, taps, C};
@@ -166,7 +144,7 @@ extern "C" int srlm_short_conv(const float* proj, long long ld, const float* in_
   if (T > 65535) return refuse(ST_BAD_SIZE, "short_conv: %d tokens", T);
   SRLM_DISPATCH_ACT(out_low ? low_dtype : DT_F32, TO,
                     launch_pdl(short_conv_kernel<TO>, grid, dim3(256), 0, stream, in, w, out_bias, entry_of_token, cu_q,
-                               slots, out, (TO*)out_low, T));
+                               slots, out, (TO*)out_low, T, silu));
   return launched();
 }
 

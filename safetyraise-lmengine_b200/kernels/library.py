@@ -80,6 +80,7 @@ class KernelLibrary:
         self.mixed_heads_cluster = 16                   # ... most blocks of a decode step's cluster
         self.split_mixed_heads = True                   # ... short prompts: the keys in slices
         self.retention_in_chunks = True                 # retention: portions in chunks of 64 tokens
+        self.states_by_groups = True                    # channel-wise delta rule, state space: portions in groups of 8 tokens
         self.grouped_pairs = True                       # ... whose largest steps run pairs of SMs on tiles of 256 tokens
 
     @property
@@ -148,12 +149,17 @@ class KernelLibrary:
                                                C.c_int(T), C.c_int(H), C.c_int(table.shape[0]),
                                                _ptr(bad_flag), C.c_float(scale), C.c_int(int(add)), _stream()), "embed_gather")
 
-    def add_rmsnorm(self, residual, delta, weight, eps, out, rows=None, unit_offset=False):
+    def add_norm(self, residual, delta, weight, eps, out, rows=None, unit_offset=False, center=False, delta_scale=1.0):
+        """residual (float32) += delta_scale * delta (kept when rows is None); out = the RMS norm of the sum, or its layer
+        norm (``center``: the row's mean is taken off first), times weight (or 1 + weight)."""
         R, H = out.shape
-        self._check(self.lib.srlm_add_rmsnorm(_ptr(residual), _ptr(delta), _ptr(weight), C.c_float(eps),
-                                              _ptr(out), dtype_code(out.dtype), _ptr(rows), C.c_int(R),
-                                              C.c_int(H), C.c_int(int(unit_offset)), _stream()),
-                    "add_rmsnorm")
+        self._check(self.lib.srlm_add_norm(_ptr(residual), _ptr(delta), C.c_float(delta_scale), _ptr(weight), C.c_float(eps),
+                                           _ptr(out), dtype_code(out.dtype), _ptr(rows), C.c_int(R),
+                                           C.c_int(H), C.c_int(int(unit_offset)), C.c_int(int(center)), _stream()),
+                    "add_layernorm" if center else "add_rmsnorm")
+
+    def add_rmsnorm(self, residual, delta, weight, eps, out, rows=None, unit_offset=False, delta_scale=1.0):
+        self.add_norm(residual, delta, weight, eps, out, rows, unit_offset, delta_scale=delta_scale)
 
     def swiglu(self, gate_up, out):
         T, I = out.shape
@@ -189,9 +195,27 @@ class KernelLibrary:
         self._check(self.lib.srlm_check_finite(_ptr(a), _ptr(b), dtype_code(b.dtype) if b is not None else DT_F32,
                                                C.c_longlong(a.numel()), _ptr(flag), _stream()), "check_finite")
 
-    def residual_add(self, residual, delta):
-        self._check(self.lib.srlm_residual_add(_ptr(residual), _ptr(delta), dtype_code(delta.dtype),
+    def residual_add(self, residual, delta, scale=1.0):
+        self._check(self.lib.srlm_residual_add(_ptr(residual), _ptr(delta), dtype_code(delta.dtype), C.c_float(scale),
                                                C.c_longlong(delta.numel()), _stream()), "residual_add")
+
+    def add_row(self, residual, row):
+        """residual [T, H] += row [H] (float32), in every row."""
+        T, H = residual.shape
+        self._check(self.lib.srlm_add_row(_ptr(residual), _ptr(row), C.c_int(T), C.c_int(H), _stream()), "add_row")
+
+    def stream_beside_embedding(self, residual, delta, delta_scale, ids, table, table_scale, kept, out):
+        """out [T, 2 H] float32 = [x | x0], or [T, 3 H] bfloat16 = [x's upper | lower half | x0], with x = residual +
+        delta_scale * delta (None: nothing) and x0 = the table's rows of the token ids times table_scale, or ``kept``
+        (float32 [T, H]) where it is given."""
+        T, H = residual.shape
+        if tuple(out.shape) != (T, (3 if out.dtype == torch.bfloat16 else 2) * H) or (
+                delta is not None and (delta.dtype != out.dtype or tuple(delta.shape) != (T, H))):
+            raise ShapeError(f"stream_beside_embedding: residual {tuple(residual.shape)}, out {tuple(out.shape)} {out.dtype}")
+        self._check(self.lib.srlm_stream_beside_embedding(
+            _ptr(residual), _ptr(delta), C.c_float(delta_scale), _ptr(ids), _ptr(table), dtype_code(table.dtype),
+            C.c_float(table_scale), C.c_int(table.shape[0]), _ptr(kept), _ptr(out), dtype_code(out.dtype), C.c_int(T),
+            C.c_int(H), _stream()), "stream_beside_embedding")
 
     # ---- position encoding and cache append ------------------------------
     def rope_table(self, positions, cos, sin, theta, rotary_dim):
@@ -971,24 +995,38 @@ class KernelLibrary:
         return bool(self.lib.srlm_moe_sort_routes(C.c_int(tokens), C.c_int(experts)))
 
     def moe_sort(self, choice, experts, offsets, tiles, pair_of_row, row_of_pair, tile_rows=0, group_of_tile=None,
-                 route=None, scoring="softmax_of_chosen", groups=(1, 1), correction=None, weight_scale=1.0):
+                 route=None, scoring="softmax_of_chosen", groups=(1, 1), correction=None, weight_scale=1.0, look_up=None):
         """The (token, choice) pairs ordered by expert: offsets / tiles int32 [experts + 1] (first row and first
         tile of each expert), pair_of_row / row_of_pair int32 [pairs].  tile_rows > 0: every expert's rows start at
         a multiple of tile_rows; pair_of_row then covers all rows of group_of_tile's tiles (-1: a row without a
         pair) and group_of_tile int32 [tiles] names each tile's expert (-1: none).  route (logits, column, bias,
-        weight): the kernel first routes the tokens itself, as moe_route does, and writes choice and weight."""
+        weight): the kernel first routes the tokens itself, as moe_route does, and writes choice and weight.  look_up
+        (ids, table, weight): likewise, as moe_look_up does, every weight weight_scale."""
+        ids = table = None
         if route is not None:
             logits, column, bias, weight = route
             ptr, ld = self._columns(logits, column, experts)
             routing = (ptr, ld, _ptr(bias), C.c_int(choice.shape[1]), _ptr(weight))
         else:
             routing = (C.c_void_p(0), C.c_longlong(0), C.c_void_p(0), C.c_int(0), C.c_void_p(0))
+        if look_up is not None:
+            ids, table, weight = look_up
+            routing = (*routing[:3], C.c_int(choice.shape[1]), _ptr(weight))
         self._check(self.lib.srlm_moe_sort(
             _ptr(choice), C.c_int(choice.numel()), C.c_int(experts), _ptr(offsets), _ptr(tiles), _ptr(pair_of_row),
             _ptr(row_of_pair), C.c_int(tile_rows), _ptr(group_of_tile),
             C.c_int(group_of_tile.numel() if group_of_tile is not None else 0),
             C.c_int(pair_of_row.numel()), *routing, C.c_int(self.ROUTER_SCORING[scoring]), C.c_int(groups[0]),
-            C.c_int(groups[1]), _ptr(correction), C.c_float(weight_scale), _stream()), "moe_sort")
+            C.c_int(groups[1]), _ptr(correction), C.c_float(weight_scale), _ptr(ids), _ptr(table),
+            C.c_int(table.shape[0] if table is not None else 0), _stream()), "moe_sort")
+
+    def moe_look_up(self, ids, table, experts, share, choice, weight):
+        """choice int32 [T, top] = the rows of table (int32 [vocab, top]) of the token ids; weight float32 [T, top] = share."""
+        T, top = choice.shape
+        if table.dtype != torch.int32 or table.shape[1] != top or choice.dtype != torch.int32 or weight.dtype != torch.float32:
+            raise ShapeError(f"moe_look_up: table {tuple(table.shape)} {table.dtype}, choice {tuple(choice.shape)}")
+        self._check(self.lib.srlm_moe_look_up(_ptr(ids), _ptr(table), C.c_int(table.shape[0]), C.c_int(T), C.c_int(experts),
+                                              C.c_int(top), C.c_float(share), _ptr(choice), _ptr(weight), _stream()), "moe_look_up")
 
     GROUPED_TILE = 128       # token rows of a tile of the grouped tensor-memory product (one SM a tile)
     GROUPED_PAIR_TILE = 256  # ... of its pair form (two SMs on 256 weight rows x 256 tokens)
@@ -1132,10 +1170,11 @@ class KernelLibrary:
                                                   dtype_code(out.dtype), C.c_int(x.shape[0]), C.c_int(width), _stream()),
                     "rmsnorm_columns")
 
-    ACTIVATIONS = {"gelu": 0, "gelu_tanh": 1}
+    ACTIVATIONS = {"gelu": 0, "gelu_tanh": 1, "relu_squared": 2}
 
     def activation(self, x, out, kind, bias=None, column=0):
-        """out [T, F] = act(x[:, column : column + F] + bias); kind "gelu" (exact) or "gelu_tanh"."""
+        """out [T, F] = act(x[:, column : column + F] + bias); kind "gelu" (exact), "gelu_tanh" or "relu_squared"
+        (max(z, 0)^2)."""
         T, F = out.shape
         if not x.is_cuda or x.stride(1) != 1 or x.shape[1] < column + F:
             raise ShapeError("activation: columns of a row-major CUDA tensor are wanted")
@@ -1152,17 +1191,19 @@ class KernelLibrary:
                     "weighted_sum")
 
     # ---- short convolutions over time ---------------------------------------------------------------
-    def short_conv(self, ctx, x, column, channels, weight, state, state_off, out, in_bias=None, out_bias=None, out_low=None):
+    def short_conv(self, ctx, x, column, channels, weight, state, state_off, out, in_bias=None, out_bias=None, out_low=None,
+                   silu=False):
         """out float32 [T, channels] = the causal convolution over time of the columns [column, + channels) of x (float32),
         per channel with weight float32 [channels, taps]; in_bias is added to every input, out_bias to every result.  A
         portion's first tokens read the slot's carried inputs ([taps - 1][channels] floats at state_off of its row of
-        ``state``, float32 [slots, row]); ``conv_carry`` renews them afterwards.  out_low: a copy in its own dtype."""
+        ``state``, float32 [slots, row]); ``conv_carry`` renews them afterwards.  out_low: a copy in its own dtype.
+        silu: every result z becomes z * logistic(z)."""
         ptr, ld = self._columns(x, column, channels)
         self._check(self.lib.srlm_short_conv(
             ptr, ld, _ptr(in_bias), _ptr(weight), _ptr(out_bias), _ptr(state), C.c_longlong(state.stride(0)),
             C.c_int(state_off), _ptr(ctx.entry_of_token), _ptr(ctx.cu_q), _ptr(ctx.slots), _ptr(out), _ptr(out_low),
             dtype_code(out_low.dtype) if out_low is not None else 0, C.c_int(x.shape[0]), C.c_int(channels),
-            C.c_int(weight.shape[1]), _stream()), "short_conv")
+            C.c_int(weight.shape[1]), C.c_int(int(silu)), _stream()), "short_conv")
 
     def conv_carry(self, ctx, x, column, channels, taps, state, state_off, in_bias=None):
         """The slots' carried inputs of a short convolution <- the last taps - 1 inputs of every entry (what was carried
@@ -1449,11 +1490,87 @@ class KernelLibrary:
             _ptr(ctx.slots), C.c_int(ctx.n_entries), _ptr(o_out), C.c_int(H), C.c_int(G), C.c_int(dk), C.c_int(dv),
             _stream()), "delta_recurrence")
 
-    def delta_output(self, o, norm_w, eps, proj, gate_off, out, H, dv):
+    def delta_output(self, o, norm_w, eps, proj, gate_off, out, H, dv, logistic=False):
+        """out = per head o / sqrt(mean(o^2) + eps) * norm_w * silu(gate) (``logistic``: logistic(gate) in silu's place),
+        the gate in the columns of proj from gate_off."""
         self._check(self.lib.srlm_delta_output(
             _ptr(o), _ptr(norm_w), C.c_float(eps), _ptr(proj), dtype_code(proj.dtype), C.c_longlong(proj.stride(0)),
             C.c_int(gate_off), _ptr(out), dtype_code(out.dtype), C.c_int(o.shape[0]), C.c_int(H), C.c_int(dv),
-            _stream()), "delta_output")
+            C.c_int(int(logistic)), _stream()), "delta_output")
+
+    # ---- walks over a matrix of state: token by token, or by groups of 8 tokens --------------------------
+    STATE_WALK = 2           # steps whose portions all have at most this many tokens go token by token
+
+    def _by_groups(self, ctx, record):
+        """How many groups of 8 tokens the step's entries make, 0 where the step goes token by token (short portions, or
+        heads that the grouped kernels do not take: ``record`` 0)."""
+        if not self.states_by_groups or not record or ctx.max_q_len <= self.STATE_WALK:
+            return 0
+        return sum(-(-n // 8) for n in ctx.host["q_lens"])
+
+    def channel_delta(self, ctx, proj, conv_w, low, a_log, dt_bias, state, norm_w, eps, out, H, G, dk, dv, taps, unit_eps):
+        """out [T, H dv] = the gated delta rule with a decay per head and key channel, from the projections
+        proj (float32: q | k | v | beta ...) and low (float32: decay | gate), as csrc/kernels/channel_delta.cu says: short
+        convolutions, unit vectors, recurrence, per-head norm, weight and logistic gate.  state float32 [slots, row]: S and
+        the convolutions' carried inputs, both renewed."""
+        T, channels, carry = proj.shape[0], 2 * G * dk + H * dv, H * dk * dv
+        ws, sizes = ctx.workspace, (C.c_int(H), C.c_int(G), C.c_int(dk), C.c_int(dv))
+        record = int(self.lib.srlm_channel_delta_record(C.c_int(dk)))
+        groups = self._by_groups(ctx, record)
+        o = None
+        if groups or not self.lib.srlm_channel_delta_walk_finishes(C.c_int(dk), C.c_int(dv)):
+            o = ws.get("channel_delta.o", T, H * dv, torch.float32)
+        where = (_ptr(state), C.c_longlong(state.stride(0)), _ptr(ctx.cu_q), _ptr(ctx.slots), C.c_int(ctx.n_entries))
+        if groups:
+            conv = ws.get("channel_delta.conv", T, channels, torch.float32)
+            self.short_conv(ctx, proj, 0, channels, conv_w, state, carry, conv, silu=True)
+            records = ws.get("channel_delta.records", groups * H, record, torch.float32, reserve=0)
+            self._check(self.lib.srlm_channel_delta_groups(
+                _ptr(conv), _ptr(proj), C.c_longlong(proj.stride(0)), _ptr(low), C.c_longlong(low.stride(0)), _ptr(a_log),
+                _ptr(dt_bias), *where, _ptr(records), _ptr(o), C.c_int(groups), *sizes, C.c_float(unit_eps), _stream()),
+                "channel_delta_groups")
+            self.launches += 1           # the walk along the groups
+        else:
+            self._check(self.lib.srlm_channel_delta_walk(
+                _ptr(proj), C.c_longlong(proj.stride(0)), _ptr(conv_w), _ptr(low), C.c_longlong(low.stride(0)), _ptr(a_log),
+                _ptr(dt_bias), *where, _ptr(norm_w), C.c_float(eps), _ptr(o), _ptr(out), dtype_code(out.dtype), *sizes,
+                C.c_int(taps), C.c_float(unit_eps), _stream()), "channel_delta_walk")
+        self.conv_carry(ctx, proj, 0, channels, taps, state, carry)
+        if o is not None:
+            self.delta_output(o, norm_w, eps, low, H * dk, out, H, dv, logistic=True)
+
+    def state_space(self, ctx, proj, conv_w, conv_b, dt_bias, a_log, D, state, y, H, G, N, P, taps):
+        """y float32 [T, H P] = the read-out of a state with one decay a head (+ D x), from the projection proj (float32:
+        z | x | B | C | dt), as csrc/kernels/state_space.cu says; state float32 [slots, row]: S and the convolution's carried
+        inputs, both renewed.  ``state_space_output`` gates and norms it."""
+        T, inner = proj.shape[0], H * P
+        channels, carry = inner + 2 * G * N, H * N * P
+        sizes = (C.c_int(H), C.c_int(G), C.c_int(N), C.c_int(P))
+        params = (_ptr(dt_bias), _ptr(a_log), _ptr(D), _ptr(state), C.c_longlong(state.stride(0)), _ptr(ctx.cu_q),
+                  _ptr(ctx.slots), C.c_int(ctx.n_entries))
+        record = int(self.lib.srlm_state_space_record(C.c_int(N)))
+        groups = self._by_groups(ctx, record)
+        if groups:
+            conv = ctx.workspace.get("state_space.conv", T, channels, torch.float32)
+            self.short_conv(ctx, proj, inner, channels, conv_w, state, carry, conv, out_bias=conv_b, silu=True)
+            records = ctx.workspace.get("state_space.records", groups * H, record, torch.float32, reserve=0)
+            self._check(self.lib.srlm_state_space_groups(
+                _ptr(conv), _ptr(proj), C.c_longlong(proj.stride(0)), *params, _ptr(records), _ptr(y), C.c_int(groups), *sizes,
+                _stream()), "state_space_groups")
+            self.launches += 1           # the walk along the groups
+        else:
+            self._check(self.lib.srlm_state_space_walk(
+                _ptr(proj), C.c_longlong(proj.stride(0)), _ptr(conv_w), _ptr(conv_b), *params, _ptr(y), *sizes, C.c_int(taps),
+                _stream()), "state_space_walk")
+        self.conv_carry(ctx, proj, inner, channels, taps, state, carry)
+
+    def state_space_output(self, y, proj, weight, eps, out, parts):
+        """out [T, inner] = weight * u / sqrt(mean(u^2) + eps) over each of ``parts`` equal parts of the row, u = y * silu(z)
+        with z the first inner columns of proj."""
+        T, inner = y.shape
+        self._check(self.lib.srlm_state_space_output(
+            _ptr(y), _ptr(proj), C.c_longlong(proj.stride(0)), _ptr(weight), C.c_float(eps), _ptr(out), dtype_code(out.dtype),
+            C.c_int(T), C.c_int(inner), C.c_int(parts), _stream()), "state_space_output")
 
     # ---- sampling -------------------------------------------------------------
     def argmax(self, logits, out_tokens, bad_flag):

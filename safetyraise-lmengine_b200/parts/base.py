@@ -180,6 +180,18 @@ class NormedInput:
     eps: float
 
 
+@dataclass
+class ScaledDelta:
+    """A tensor still to be added to the residual stream, times a factor."""
+    x: torch.Tensor
+    scale: float
+
+
+def split_delta(pending):
+    """(tensor or None, factor) of what is still to be added to the residual stream."""
+    return (pending.x, pending.scale) if isinstance(pending, ScaledDelta) else (pending, 1.0)
+
+
 class Part:
     """Common behaviour: a part declares its tensors before it is built.
 
@@ -215,12 +227,13 @@ class Block(Part):
 
     ``forward(ctx, residual, pending, run_step, next_block) -> pending``.  ``residual`` [T, hidden] float32
     is updated in place.  ``pending`` is what the block before left behind: None, a tensor still to be
-    added to the residual (the next norm kernel adds it while it norms), or a ``NormedInput`` -- the input
+    added to the residual (the next norm kernel adds it while it norms; a ``ScaledDelta``: times its scale), or a
+    ``NormedInput`` -- the input
     of this block's first part, already prepared by the product that wrote the residual.  A block may
     hand its successor such a prepared input only if the successor says it takes one for this step:
     ``next_block.prepared_input_norm(ctx)`` returns the norm whose weight the input must carry, or None
     (the default: the successor wants a plain pending tensor).  ``next_block`` is None behind the last
-    block; what the last block returns goes to the final norm, so it must be a tensor or None."""
+    block; what the last block returns goes to the final norm, so it must be a tensor, a ScaledDelta or None."""
 
     def prepared_input_norm(self, ctx):
         return None

@@ -1,6 +1,7 @@
 """The arrangements of norms, mixer and feed-forward around the residual stream.
 
-``pre_norm``: r = x + mixer(norm(x)); x' = r + ff(norm(r))  (src/model/native.rs:526-562).
+``pre_norm``: r = x + a mixer(norm(x)); x' = r + a ff(norm(r)), a = 1 unless a layer says otherwise
+(src/model/native.rs:526-562).
 ``sandwich_gated``: a norm before and after each sublayer and a learned gate on its result (see the class).
 ``parallel``: h = norm(x); x' = x + mixer(h) + ff(h): one norm, both sublayers read it.
 ``post_norm``: x' = norm(a x + mixer(x)), then x'' = norm(a x' + ff(x')): the norm comes after the sum.
@@ -18,7 +19,7 @@ import torch
 from ..config.spec import LayerSpec, RunStep
 from ..kernels import ops
 from ..weights.loader import MATRIX, VECTOR, TensorDecl
-from .base import FEED_FORWARDS, MIXERS, NORMS, Block, NormedInput, lookup, register_block
+from .base import FEED_FORWARDS, MIXERS, NORMS, Block, NormedInput, ScaledDelta, lookup, register_block, split_delta
 from .linear import Linear
 
 
@@ -37,6 +38,7 @@ class PreNormBlock(Block):
             self.feed_forward = lookup(FEED_FORWARDS, spec.feed_forward.kind, "feed-forward")(
                 spec.feed_forward, p, tensors, mctx)
         self.hidden = spec.mixer_norm.size
+        self.scale = float(spec.sublayer_scale)
         self.replayable = all(getattr(part, "replayable", True)
                               for part in (self.mixer_norm, self.ff_norm, self.mixer, self.feed_forward))
 
@@ -55,7 +57,7 @@ class PreNormBlock(Block):
     def fuses(self, ctx) -> bool:
         """Whether this block runs its norms inside the products around them for this step: both parts
         offer forward_fused and the step is small enough for the kernels that carry the fusions."""
-        return (self.feed_forward is not None
+        return (self.feed_forward is not None and self.scale == 1.0
                 and getattr(self.mixer_norm, "fusable", False) and getattr(self.ff_norm, "fusable", False)
                 and hasattr(self.mixer, "forward_fused") and hasattr(self.feed_forward, "forward_fused")
                 and self.mixer.can_fuse(ctx) and self.feed_forward.can_fuse(ctx)
@@ -83,11 +85,14 @@ class PreNormBlock(Block):
         assert not isinstance(pending, NormedInput), "a prepared input was handed to a block that did not ask for one"
         n = ctx.workspace.get("block.normed", T, self.hidden, ctx.dtype)
         self.mixer_norm.apply(residual, pending, n)
-        mixed = self.mixer.forward(ctx, n, run_step)
+        mixed = self._scaled(self.mixer.forward(ctx, n, run_step))
         if self.feed_forward is None:
             return mixed                      # the next norm adds it
         self.ff_norm.apply(residual, mixed, n)
-        return self.feed_forward.forward(ctx, n)
+        return self._scaled(self.feed_forward.forward(ctx, n))
+
+    def _scaled(self, sub):
+        return sub if self.scale == 1.0 else ScaledDelta(sub, self.scale)
 
 
 @register_block("parallel")
@@ -256,7 +261,7 @@ class PostNormBlock(Block):
                 "only a block of this kind hands this block a prepared input"
         else:
             if pending is not None:
-                ops.residual_add(residual, pending)
+                ops.residual_add(residual, *split_delta(pending))
             if low:
                 ops.cast(residual, x)
         if getattr(self.mixer, "offers_terms", False):      # a weighted pair: its sum rides in the kernel below

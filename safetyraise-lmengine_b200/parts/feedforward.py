@@ -65,11 +65,11 @@ class GatedDense(Part):
 
 @register_feed_forward("dense")
 class Dense(Part):
-    """down(act(up(x))) without a gate; ``activation`` "gelu": the exact one.  The first product writes float32 and the
+    """down(act(up(x))) without a gate; ``activation`` "gelu": the exact one, "relu_squared": max(z, 0)^2.  The first product writes float32 and the
     activation rounds once, into the second product's input."""
 
     def __init__(self, spec, prefix: str, tensors: dict, mctx):
-        if spec.activation != "gelu":
+        if spec.activation not in ("gelu", "relu_squared"):
             raise Unsupported(f"a dense feed-forward with activation {spec.activation!r} is not implemented")
         self.spec = spec
         nm = spec.dense_names

@@ -14,9 +14,9 @@ from ..cache.manager import FIXED_STATE, CacheGroupSpec
 from ..config.spec import ModelSpec
 from ..errors import ConfigError
 from ..kernels import ops
-from ..weights.loader import MATRIX, TABLE, TensorDecl, load_tensors
+from ..weights.loader import MATRIX, TABLE, VECTOR, TensorDecl, load_tensors
 from .base import (BLOCKS, EMBEDDING, FAULT_ACTIVATION, FAULT_TOKEN, NORMS, POSITION_ENCODINGS, STATUS_WORDS,
-                   ModelContext, lookup)
+                   ModelContext, lookup, split_delta)
 from .linear import Linear
 
 
@@ -30,6 +30,10 @@ def tensor_decls(spec: ModelSpec) -> List[TensorDecl]:
     for layer in spec.layers:
         decls += lookup(BLOCKS, layer.block, "block").tensor_decls(layer)
     decls += lookup(NORMS, spec.final_norm.kind, "norm").tensor_decls(spec.final_norm, spec.final_norm_name)
+    if spec.num_passes:
+        H = spec.hidden_size
+        decls += [TensorDecl(spec.pass_product_name, (H, 2 * H), MATRIX),
+                  TensorDecl(spec.pass_vectors_name, (spec.num_passes, H), VECTOR)]
     if not spec.tie_word_embeddings:
         decls.append(TensorDecl(spec.head_name, (spec.vocab_size, spec.hidden_size), MATRIX))
     return decls
@@ -95,7 +99,18 @@ class DecoderModel:
                                                                       tensors, mctx)
         # tied: the head IS the embedding table (same storage), src/model/native.rs:171-179
         self.head = Linear(self.embed if spec.tie_word_embeddings else tensors[spec.head_name], "lm_head")
-        self.keeps_embedding = any(s.add_embedding for s in spec.run_order) and \
+        if spec.logit_scale != 1.0:      # on the final norm's weight: head (c n) = c (head n), and the weight is float32
+            if spec.final_norm.unit_offset:
+                raise ConfigError("a factor on the logits needs a final norm whose weight is applied as it is")
+            self.final_norm.weight = self.final_norm.weight * spec.logit_scale
+        self.pass_product = self.pass_vectors = None
+        if spec.num_passes:
+            w, H = tensors[spec.pass_product_name], spec.hidden_size
+            if mctx.dtype == torch.bfloat16:       # the stream's two halves meet the same columns
+                w = torch.cat([w[:, :H], w], dim=1)
+            self.pass_product = Linear(w.contiguous(), spec.pass_product_name)
+            self.pass_vectors = tensors[spec.pass_vectors_name]
+        self.keeps_embedding = any(s.add_embedding or s.begins_pass is not None for s in spec.run_order) and \
             (self.embed_norm is not None or self.embed_position is not None)
         for step in spec.run_order:
             if not 0 <= step.layer < len(self.blocks):
@@ -129,6 +144,8 @@ class DecoderModel:
         pending = None
         order = self.spec.run_order
         for i, step in enumerate(order):
+            if step.begins_pass is not None:
+                pending = self._begin_pass(ctx, residual, pending, kept, step.begins_pass)
             if step.add_embedding:
                 if kept is not None:
                     ops.residual_add(residual, kept)
@@ -136,12 +153,14 @@ class DecoderModel:
                     ops.embed_gather(ctx.token_ids, self.embed, residual, status[FAULT_TOKEN:FAULT_TOKEN + 1],
                                      scale=self.spec.embed_scale, add=True)
             # a block ahead of an addition to the stream prepares no input: what it leaves is pending or in the stream
-            nxt = self.blocks[order[i + 1].layer] if i + 1 < len(order) and not order[i + 1].add_embedding else None
+            nxt = order[i + 1] if i + 1 < len(order) else None
+            nxt = self.blocks[nxt.layer] if nxt is not None and not nxt.add_embedding and nxt.begins_pass is None else None
             pending = self.blocks[step.layer].forward(ctx, residual, pending, step, nxt)
         # NaN and infinity stay in a residual stream that is only ever added to, and every key or value
         # a step writes is read by its own token: one look at the end covers every block
         # (src/model/native.rs:276-278, src/engine/state.rs:56-58)
-        ops.check_finite(residual, pending if isinstance(pending, torch.Tensor) else None,
+        left, _ = split_delta(pending)
+        ops.check_finite(residual, left if isinstance(left, torch.Tensor) else None,
                          status[FAULT_ACTIVATION:FAULT_ACTIVATION + 1])
         R = ctx.logit_rows.shape[0]
         logits = ctx.workspace.get("logits", R, self.spec.vocab_size, torch.float32, reserve=64)
@@ -153,6 +172,17 @@ class DecoderModel:
         if self.spec.logit_softcap is not None:
             ops.softcap(logits, self.spec.logit_softcap)
         return logits
+
+    def _begin_pass(self, ctx, residual, pending, kept, index: int):
+        """x <- W [x; x_0] + v_index, in place; what was pending is part of x.  -> None: nothing is pending behind it."""
+        T, H = residual.shape
+        delta, scale = split_delta(pending)
+        low = ctx.dtype == torch.bfloat16
+        both = ctx.workspace.get("pass.both", T, (3 if low else 2) * H, ctx.dtype)
+        ops.stream_beside_embedding(residual, delta, scale, ctx.token_ids, self.embed, self.spec.embed_scale, kept, both)
+        self.pass_product.into(ctx, both, residual)
+        ops.add_row(residual, self.pass_vectors[index])
+        return None
 
     def weight_bytes(self) -> int:
         seen, total = set(), 0

@@ -3,7 +3,8 @@
 angle = pos / theta^(2i/rotary_dim); src/model/math.rs:52-99.  ``prepare``
 fills one cos/sin table per step; every mixer that shares the same
 specification reuses it.  A specification with ``scaling`` rescales the
-frequencies by their wavelength (see ``rescaled_frequencies``).
+frequencies by their wavelength, one with a ``divisor`` divides all of them
+(see ``rescaled_frequencies``).
 """
 from __future__ import annotations
 
@@ -17,13 +18,13 @@ from ..kernels import ops
 from .base import ROTATION, Part, Rotation, register_position_encoding
 
 
-def rescaled_frequencies(theta: float, rotary_dim: int, scaling) -> list:
-    """f_i = theta^(-2i/rotary_dim) for i < rotary_dim / 2, in double precision; with scaling = (factor, low, high,
+def rescaled_frequencies(theta: float, rotary_dim: int, scaling, divisor: float = 1.0) -> list:
+    """f_i = theta^(-2i/rotary_dim) / divisor for i < rotary_dim / 2, in double precision; with scaling = (factor, low, high,
     original) and wavelength l = 2 pi / f: f where l < original / high, f / factor where l > original / low, and
     between the two (1 - s) f / factor + s f with s = (original / l - low) / (high - low)."""
     out = []
     for i in range(rotary_dim // 2):
-        f = theta ** (-2.0 * i / rotary_dim)
+        f = theta ** (-2.0 * i / rotary_dim) / divisor
         if scaling is not None:
             factor, low, high, original = scaling
             wave = 2.0 * math.pi / f
@@ -61,12 +62,14 @@ class RotaryHalf(Part):
     def __init__(self, spec: PositionSpec, mctx):
         self.spec = spec
         self.half = spec.rotary_dim // 2
-        self.key = ("rotary_half", spec.theta, spec.rotary_dim, spec.scaling, spec.ramp)
+        self.key = ("rotary_half", spec.theta, spec.rotary_dim, spec.scaling, spec.ramp, spec.divisor)
         self.freq, self.length = None, 1.0
         if spec.scaling is not None and spec.ramp is not None:
             raise Unsupported("a rotary encoding rescales its frequencies by wavelength or along a ramp, not both")
-        if spec.scaling is not None:
-            self.freq = torch.tensor(rescaled_frequencies(spec.theta, spec.rotary_dim, spec.scaling),
+        if spec.ramp is not None and spec.divisor != 1.0:
+            raise Unsupported("a rotary encoding divides its frequencies by one number or rescales them along a ramp, not both")
+        if spec.scaling is not None or spec.divisor != 1.0:
+            self.freq = torch.tensor(rescaled_frequencies(spec.theta, spec.rotary_dim, spec.scaling, spec.divisor),
                                      dtype=torch.float64, device=mctx.device)
         if spec.ramp is not None:
             freq, self.length = ramped_frequencies(spec.theta, spec.rotary_dim, spec.ramp)
@@ -76,7 +79,7 @@ class RotaryHalf(Part):
         """The rotation of this step's tokens: cos / sin float32 [T, rotary_dim/2], half-split pairs."""
         got = ctx.tables.get(self.key)
         if got is None:
-            tag = f"{self.spec.theta}" if self.freq is None else f"{self.spec.theta}.{self.spec.scaling}.{self.spec.ramp}"
+            tag = f"{self.spec.theta}" if self.freq is None else f"{self.spec.theta}.{self.spec.scaling}.{self.spec.ramp}.{self.spec.divisor}"
             cos = ctx.workspace.get(f"rope.cos.{tag}", ctx.T, self.half, torch.float32)
             sin = ctx.workspace.get(f"rope.sin.{tag}", ctx.T, self.half, torch.float32)
             if self.freq is None:
@@ -93,7 +96,7 @@ class RotaryInterleaved(RotaryHalf):
 
     def __init__(self, spec: PositionSpec, mctx):
         super().__init__(spec, mctx)
-        self.key = ("rotary_interleaved", spec.theta, spec.rotary_dim, spec.scaling, spec.ramp)
+        self.key = ("rotary_interleaved", spec.theta, spec.rotary_dim, spec.scaling, spec.ramp, spec.divisor)
 
     def rotation(self, ctx) -> Rotation:
         got = ctx.tables.get(self.key)

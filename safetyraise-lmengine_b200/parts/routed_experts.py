@@ -17,6 +17,7 @@ s + correction are chosen and weighted by s; ``weight_scale`` is a factor on eve
 ``scoring`` "softmax_over_all": the scores are the softmax over all experts' logits, the choice may be limited to the
 best ``groups_kept`` of ``groups`` equal groups of neighbouring experts (a group counts as its largest score), and the
 weights are the chosen scores over their sum.
+``scoring`` "table": no router; a table gives each token id its experts, each with the weight 1 / top.
 
 The pairs (token, chosen expert) are ordered by expert on the device and every expert's rows run through
 one grouped product per projection; a token's result does not depend on what else is in the step, and
@@ -31,7 +32,7 @@ import torch
 from ..config.spec import RoutedExpertsSpec
 from ..errors import Unsupported
 from ..kernels import ops
-from ..weights.loader import MATRIX, VECTOR, TensorDecl
+from ..weights.loader import INT_TABLE, MATRIX, VECTOR, TensorDecl
 from .base import Part, register_feed_forward
 from .linear import Linear
 
@@ -43,7 +44,7 @@ class RoutedExperts(Part):
             raise Unsupported(f"routed experts with activation {spec.activation!r} are not implemented")
         if not spec.gated and spec.weight_on_input:
             raise Unsupported("a weight on an expert's input comes with gated experts only")
-        if spec.scoring not in ops.ROUTER_SCORING:
+        if spec.scoring != "table" and spec.scoring not in ops.ROUTER_SCORING:
             raise Unsupported(f"routed experts with router scoring {spec.scoring!r} are not implemented")
         if spec.correction and spec.scoring != "logistic":
             raise Unsupported("a correction of the experts' choice comes with logistic scores only")
@@ -52,6 +53,11 @@ class RoutedExperts(Part):
         if spec.activation == "silu" and spec.shared_size:
             raise Unsupported("an expert that every token runs comes with the clamped activation only")
         self.spec = spec
+        self.table = None
+        if spec.scoring == "table":
+            if spec.shared_size or not spec.gated or spec.weight_on_input:
+                raise Unsupported("experts named by a table are gated, weigh their outputs and come without a shared one")
+            self.table = tensors[prefix + spec.expert_names.table]
         self.routing = dict(scoring=spec.scoring, groups=(spec.groups, spec.groups_kept), weight_scale=spec.weight_scale,
                             correction=tensors[prefix + spec.expert_names.correction] if spec.correction else None)
         if not spec.gated:
@@ -74,6 +80,9 @@ class RoutedExperts(Part):
         self.in_tiles = self.interleaved         # steps of many tokens may run the experts' products in whole tiles
         self.gate_up = torch.stack([pair(g, u) for g, u in zip(each(nm.gate), each(nm.up))]).contiguous()
         self.down = torch.stack(each(nm.down)).contiguous()
+        if self.table is not None:               # no router and no shared expert: nothing reads the layer's input whole
+            self.first, self.shared_down = None, None
+            return
         # one product for everything that reads the layer's input whole: the shared expert's gate rows, its up
         # rows, then the router's rows; its result is float32 (the router's logits are)
         first, self.shared_down = [tensors[p + nm.router]], None
@@ -116,7 +125,10 @@ class RoutedExperts(Part):
                 decls.append(TensorDecl(ep + nm.gate, (s.intermediate_size, H), MATRIX))
             decls += [TensorDecl(ep + nm.up, (s.intermediate_size, H), MATRIX),
                       TensorDecl(ep + nm.down, (H, s.intermediate_size), MATRIX)]
-        decls.append(TensorDecl(p + nm.router, (s.experts, H), MATRIX))
+        if s.scoring == "table":
+            decls.append(TensorDecl(p + nm.table, (s.vocab, s.top), INT_TABLE, below=s.experts, distinct=True))
+        else:
+            decls.append(TensorDecl(p + nm.router, (s.experts, H), MATRIX))
         if s.router_bias:
             decls.append(TensorDecl(p + nm.router_bias, (s.experts,), VECTOR))
         if s.correction:
@@ -138,26 +150,27 @@ class RoutedExperts(Part):
         if add is not None and self.shared_down is not None:
             raise Unsupported("routed experts add either their shared expert's output or a given tensor")
         # the router in float32: its input may be the activation dtype's rounding of the normed stream
-        first = self.first(ctx, x, "moe.first", out_dtype=torch.float32)
+        first = self.first(ctx, x, "moe.first", out_dtype=torch.float32) if self.table is None else None
         choice = ws.get("moe.choice", T, s.top, torch.int32)
         weight = ws.get("moe.weight", T, s.top, torch.float32)
         # steps of many tokens (64 rows an expert on average): the experts' products on the persistent tensor-memory
         # kernel, every expert's rows in whole tiles of 128 of a gathered copy of the input
         if (self.in_tiles and ops.grouped_products_in_tensor_memory and pairs >= 64 * s.experts
                 and s.intermediate_size % 8 == 0):
-            ops.moe_route(first, self.router_bias, s.top, choice, weight, column=self.router_column, experts=s.experts,
-                          **self.routing)
+            self._route(ctx, first, choice, weight)
             return self._forward_tiles(ctx, x, first, choice, weight, add)
         heads = ws.get("moe.heads", 2, s.experts + 1, torch.int32, reserve=2)
         order = ws.get("moe.order", 2 * T, s.top, torch.int32, reserve=2 * ws.max_tokens)
         offsets, tiles = heads[0], heads[1]
         pair_of_row, row_of_pair = order[:T].view(-1), order[T:].view(-1)
-        if ops.moe_sort_routes(T, s.experts):          # a small step: the block that orders the pairs routes them too
+        if self.table is not None and pairs <= 4096:   # a small step: the block that orders the pairs looks them up too
+            ops.moe_sort(choice, s.experts, offsets, tiles, pair_of_row, row_of_pair,
+                         look_up=(ctx.token_ids, self.table, weight), weight_scale=s.weight_scale / s.top)
+        elif self.table is None and ops.moe_sort_routes(T, s.experts):   # likewise, and routes them
             ops.moe_sort(choice, s.experts, offsets, tiles, pair_of_row, row_of_pair,
                          route=(first, self.router_column, self.router_bias, weight), **self.routing)
         else:
-            ops.moe_route(first, self.router_bias, s.top, choice, weight, column=self.router_column, experts=s.experts,
-                          **self.routing)
+            self._route(ctx, first, choice, weight)
             ops.moe_sort(choice, s.experts, offsets, tiles, pair_of_row, row_of_pair)
         y = ws.get("moe.y", pairs, s.intermediate_size, ctx.dtype, reserve=ws.max_tokens * s.top)
         if s.gated:
@@ -171,6 +184,14 @@ class RoutedExperts(Part):
         ops.moe_combine(rows, row_of_pair.view(T, s.top), None if s.weight_on_input else weight,
                         add if add is not None else self._shared(ctx, first), out)
         return out
+
+    def _route(self, ctx, first, choice, weight):
+        s = self.spec
+        if self.table is not None:
+            ops.moe_look_up(ctx.token_ids, self.table, s.experts, s.weight_scale / s.top, choice, weight)
+        else:
+            ops.moe_route(first, self.router_bias, s.top, choice, weight, column=self.router_column, experts=s.experts,
+                          **self.routing)
 
     def _shared(self, ctx, first):
         """The output of the expert that every token runs (its gate and up columns lead the first product), or None."""

@@ -28,6 +28,8 @@ class TensorDecl:
     shape: Tuple[Optional[int], ...]      # None: a free dimension, whose size is the stored tensor's
     role: str = MATRIX        # MATRIX | VECTOR (norm scale) | TABLE (embedding rows) | INT_TABLE
     free_size: int = 32       # what a free dimension is made as where weights are generated and not read
+    below: int = 2 ** 31 - 1  # INT_TABLE: entries lie in [0, below) ...
+    distinct: bool = False    # ... and the entries of a row differ
 
     @property
     def made_shape(self) -> Tuple[int, ...]:
@@ -78,7 +80,11 @@ def load_tensors(source, decls: Sequence[TensorDecl], compute_dtype: torch.dtype
         if d.role == INT_TABLE:
             if t.dtype != torch.int32:
                 raise WeightError(f"tensor {d.name} must be stored as I32, found {t.dtype}")
-            out[d.name] = t.to(device)
+            if t.numel() and (int(t.min()) < 0 or int(t.max()) >= d.below):
+                raise WeightError(f"tensor {d.name} must hold integers from 0 to {d.below - 1}, found {int(t.min())} to {int(t.max())}")
+            if d.distinct and bool((t.sort(dim=-1).values.diff(dim=-1) == 0).any()):
+                raise WeightError(f"tensor {d.name} repeats an entry within a row")
+            out[d.name] = t.to(device).contiguous()
             continue
         if not t.dtype.is_floating_point:
             raise WeightError(f"tensor {d.name} must be a float tensor, found {t.dtype}")

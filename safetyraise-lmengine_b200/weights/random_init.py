@@ -35,7 +35,10 @@ def random_tensor(decl: TensorDecl, seed: int, device="cpu", matrix_dtype=torch.
     if decl.role == VECTOR:
         return 1.0 + 0.1 * torch.randn(decl.made_shape, generator=gen, device=device, dtype=torch.float32)
     if decl.role == INT_TABLE:
-        return torch.randint(0, 2 ** 31 - 1, decl.made_shape, generator=gen, device=device, dtype=torch.int32)
+        if decl.distinct:            # every row a random choice without repetition
+            keys = torch.rand((*decl.made_shape[:-1], decl.below), generator=gen, device=device)
+            return keys.topk(decl.made_shape[-1], dim=-1).indices.to(torch.int32)
+        return torch.randint(0, decl.below, decl.made_shape, generator=gen, device=device, dtype=torch.int32)
     t = torch.empty(decl.made_shape, device=device, dtype=matrix_dtype)
     # generated in slabs so that a large table needs no float32 copy of itself
     flat = t.view(-1)
