@@ -2,7 +2,7 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
                     [--shape 8b|14b|32b] [--workload decode|mixed]
-    python bench.py --design nekedra|tonanex|pabalorn|dovorax [--design-size 2048|4096]
+    python bench.py --design nekedra|tonanex|pabalorn|dovorax|lokizen|mapovik [--design-size 2048|4096]
 
 A "step" is one decode step: every request of the batch gets its next token.
 The default run has the sizes of the 8B configuration (36 layers, hidden 4096,
@@ -42,7 +42,11 @@ layers, of layers with an attention and a selective scan side by side, and of
 both in turn, beside Qwen3 and the Tonanex stack with routed experts,
 ``--design dovorax`` for Dovorax stacks of each of its three layer kinds and of
 all of them, beside Qwen3, Nekedra's latent attention and delta rule, and the
-Tonanex stack with routed experts.
+Tonanex stack with routed experts, ``--design lokizen`` for Lokizen stacks of
+attention, of retention and of both in a loop, ``--design mapovik`` for Mapovik
+stacks of delta-rule layers, of layers with an attention and a state space side
+by side, and of both in a loop, beside Nekedra's delta rule, Tonanex's routed
+experts and Pabalorn's side-by-side layers.
 """
 from __future__ import annotations
 
@@ -661,6 +665,31 @@ def lokizen_config(size: dict, kinds) -> dict:
     return cfg
 
 
+def mapovik_config(size: dict, kinds) -> dict:
+    """A Mapovik configuration whose layers have the sizes of a Qwen3 layer of the same width: a delta rule of as many heads
+    of 128 x 128 with half as many q / k heads, 4 taps and low-rank projections of the generated rank, 32; a 'parallel' layer of attention with
+    heads of 128, half of each rotated, beside a state space of two widths of channels in heads of 64 with 128 states, 4
+    taps; 16 gated experts of three quarters of a width of which a token's row of a table names 4, or ('... dense') a dense
+    feed-forward of four and a half widths without a gate.  'loop' in the list: the layer behind it runs twice."""
+    W, H, G = size["width"], size["heads"], size["kv_heads"]
+    mixers = {
+        "channel_delta": {"heads": H, "kv_heads": H // 2, "dim": 128, "vdim": 128, "conv": 4},
+        "parallel": {"left": {"heads": H, "kv_heads": G, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                              "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 4.0}}},
+                     "right": {"heads": 2 * W // 64, "vdim": 64, "state": 128, "groups": 4, "norm_groups": 4, "conv": 4}},
+    }
+    moe = {"kind": "moe", "expert": {"ff": 3 * W // 4}, "router": {"experts": 16, "top": 4}}
+    cfg = {"architecture": "Mapovik", "width": W, "vocab": DESIGN_VOCAB, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+           "logit_scale": 0.25,
+           "layers": [{"type": k.removesuffix(" dense"), "mixer": mixers[k.removesuffix(" dense")],
+                       "mlp": {"kind": "dense", "ff": 9 * W // 2} if k.endswith(" dense") else moe}
+                      for k in kinds if k != "loop"]}
+    if "loop" in kinds:
+        at = kinds.index("loop")
+        cfg["loop"] = {"start": at, "stop": at + 1, "times": 2}
+    return cfg
+
+
 def qwen3_config(size: dict) -> dict:
     return dict(BASE, num_hidden_layers=DESIGN_LAYERS, hidden_size=size["width"], num_attention_heads=size["heads"],
                 num_key_value_heads=size["kv_heads"], intermediate_size=3 * size["width"], vocab_size=DESIGN_VOCAB)
@@ -697,6 +726,12 @@ def run_design(args) -> dict:
                   "lokizen attention": ["attention"] * DESIGN_LAYERS, "lokizen retention": ["retention"] * DESIGN_LAYERS,
                   "lokizen looped": ["retention", "loop", "attention", "retention"]}
         make = tonanex_config
+    if args.design == "mapovik":
+        stacks = {"qwen3": None, "nekedra delta": ["delta"] * DESIGN_LAYERS, "tonanex experts": ["moe"] * DESIGN_LAYERS,
+                  "pabalorn parallel": ["parallel"] * DESIGN_LAYERS,
+                  "mapovik delta": ["channel_delta"] * DESIGN_LAYERS, "mapovik parallel": ["parallel"] * DESIGN_LAYERS,
+                  "mapovik looped": ["channel_delta dense", "loop", "parallel", "channel_delta"]}
+        make = lambda size, kinds: (tonanex_config if kinds[0] == "moe" else pabalorn_config)(size, kinds)
     out = {"metric": args.design + "_beside_qwen3", "layers": DESIGN_LAYERS, "prefill_tokens": PREFILL_TOKENS,
            "decode_batch": batch, "decode_context": context, "dtype": "bf16", "data": "synthetic", "sizes": {}}
     sizes = [args.design_size] if args.design_size else sorted(DESIGN_SIZES)
@@ -709,6 +744,8 @@ def run_design(args) -> dict:
                 cfg = dovorax_config(size, kinds)
             elif label.startswith("lokizen"):
                 cfg = lokizen_config(size, kinds)
+            elif label.startswith("mapovik"):
+                cfg = mapovik_config(size, kinds)
             elif label.startswith("nekedra"):
                 cfg = nekedra_config(size, kinds)
             else:
@@ -717,10 +754,10 @@ def run_design(args) -> dict:
                                PREFILL_TOKENS)
             randomize_cache(eng)
             prefill_ms = time_prefill(eng, PREFILL_TOKENS, 3)
-            ptable = prefill_kernel_table(eng, PREFILL_TOKENS, top=6)
+            ptable = prefill_kernel_table(eng, PREFILL_TOKENS, top=args.design_kernels)
             slots = fill_contexts(eng, batch, context)
             d = time_decode(eng, slots, context, args.steps, args.warmup, 0.5)
-            dtable = kernel_table(eng, slots, context, top=6)
+            dtable = kernel_table(eng, slots, context, top=args.design_kernels)
             rows[label] = {"prefill_ms": round(prefill_ms, 3),
                            "prefill_tok_s": round(PREFILL_TOKENS / prefill_ms * 1000.0, 1),
                            "decode_ms_per_step": round(d["ms_per_step"], 4),
@@ -751,10 +788,11 @@ def main() -> int:
     ap.add_argument("--only-prefill", action="store_true", help="run just the 2,048-token prefill (for profilers)")
     ap.add_argument("--streaming-kernel", action="store_true",
                     help="steps of up to 8 tokens on the weight-streaming mma.sync kernel instead of the tensor-core one")
-    ap.add_argument("--design", default=None, choices=["nekedra", "tonanex", "pabalorn", "dovorax", "lokizen"],
+    ap.add_argument("--design", default=None, choices=["nekedra", "tonanex", "pabalorn", "dovorax", "lokizen", "mapovik"],
                     help="instead of the default workload: prefill and decode of that design's stacks beside the Qwen3 decoder "
                          "at equal layer sizes")
     ap.add_argument("--design-stack", default=None, help="only the stacks of --design whose name begins so")
+    ap.add_argument("--design-kernels", type=int, default=6, help="how many kernels of every step --design lists")
     ap.add_argument("--design-size", default=None, choices=sorted(DESIGN_SIZES), help="one width of --design")
     ap.add_argument("--min-seconds", type=float, default=MIN_TIMED_SECONDS,
                     help="repeat the block of --steps steps until this much is timed (0: one block, for profilers)")

@@ -12,13 +12,14 @@
 //
 // Steps of short portions (decoding) take channel_delta_walk: one launch does convolution, decays, recurrence and, where a
 // block holds a whole head, norm, gate and rounding; any sizes.  Steps with longer portions go by groups of 8 tokens:
-//   channel_delta_groups   what 8 tokens do to a column of S that all columns share.  With P_i = g_1 .. g_i (products within
-//                          the group, elementwise) and R_j = g_(j+1) .. g_8:
-//                             kd_i = P_i k_i,  qd_i = P_i q_i,  ke_j = R_j k_j,  whole = P_8,
+//   channel_delta_groups   what 8 tokens do to a column of S and of v, which all columns share.  With P_i = g_1 .. g_i
+//                          (products within the group, elementwise) and R_j = g_(j+1) .. g_8:
 //                             N_ij = sum_r k_i k_j g_(j+1) .. g_i (j < i),  M_ij = likewise with q_i (j <= i),
-//                             X = (I + diag(beta) N)^-1 diag(beta)
-//   channel_delta_read     walks the groups with S in registers: for a column of S and of v,
-//                             u = X (v - [kd_i . S]),   o_i = qd_i . S + sum_j M_ij u_j,   S <- whole S + sum_j ke_j u_j
+//                             X = (I + diag(beta) N)^-1 diag(beta):  u = X (v - [P_i k_i . S]),  o_i = P_i q_i . S + (M u)_i
+//                          and, with the products by X and M taken ahead of S,
+//                             kx = X [P_i k_i],  qm = [P_i q_i] - M kx,  ke_j = R_j k_j,  whole = P_8,  MX = M X
+//   channel_delta_read     walks the groups with S in registers, two products with S and one update a group:
+//                             u = X v - kx . S,   o = MX v + qm . S,   S <- whole S + sum_j ke_j u_j
 // The products of the decays never exceed 1, so nothing grows; a decay that underflows is a zero that stays one.
 #include "state_walk.cuh"
 
@@ -133,10 +134,11 @@ channel_delta_walk_kernel(ConvInput in, const float* __restrict__ conv_w, const 
 }
 
 // ---- groups of 8 tokens ------------------------------------------------------------------------------------------------
-// A group's record for one head, floats: kd [8][dkp] | qd [8][dkp] | ke [8][dkp] | whole [dkp] | X [8][8] | M [8][8].
+// A group's record for one head, floats: kx [8][dkp] | qm [8][dkp] | ke [8][dkp] | whole [dkp] | X [8][8] | MX [8][8].
 __host__ __device__ inline int delta_record(int dkp) { return 25 * dkp + 2 * kStateGroup * kStateGroup; }
 
-// A block per (group, head).  conv: the convolved and activated q | k | v channels, float32 [T, C].
+// A block per (group, head), R key channels a thread.  conv: the convolved and activated q | k | v channels, float32 [T, C].
+template <int R>
 __global__ void __launch_bounds__(128)
 channel_delta_groups_kernel(const float* __restrict__ conv, int C, const float* __restrict__ proj, long long ldp,
                             const float* __restrict__ low, long long ldl, const float* __restrict__ a_log,
@@ -146,184 +148,236 @@ channel_delta_groups_kernel(const float* __restrict__ conv, int C, const float* 
   pdl_trigger();
   constexpr int M = kStateGroup;
   __shared__ float unit_s[2 * M];            // 1 / |k_i|, then dk^-1/2 / |q_i|
+  __shared__ float beta_s[M];
   __shared__ float part[4][64];
   __shared__ float coef[64];
+  __shared__ __align__(16) float x_s[M][M], m_s[M][M];
   const GroupHome home = group_home(cu_q, n_entries, blockIdx.x);
   if (home.entry < 0) return;
   const int h = blockIdx.y, kh = h / (z.H / z.G), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const float* first = conv + (size_t)home.t0 * C;
-  for (int x = warp; x < 2 * M; x += 4) {
-    const int i = x % M;
-    float ss = 0.f;
-    if (i < home.n) {
-      const float* v = first + (size_t)i * C + (size_t)((x < M ? z.G : 0) + kh) * z.dk;
-      for (int r = lane; r < z.dk; r += 32) ss += v[r] * v[r];
+  float k[R][M], q[R][M], g[R][M], sums[2 * M];
+#pragma unroll
+  for (int s = 0; s < 2 * M; ++s) sums[s] = 0.f;
+#pragma unroll
+  for (int x = 0; x < R; ++x) {
+    const int r = tid + 128 * x;
+    const float* row = conv + (size_t)home.t0 * C + (size_t)kh * z.dk + r;
+    const float* a = low + (size_t)home.t0 * ldl + (size_t)h * z.dk + r;
+#pragma unroll
+    for (int i = 0; i < M; ++i) {
+      const bool there = i < home.n && r < z.dk;
+      q[x][i] = there ? row[(size_t)i * C] : 0.f;
+      k[x][i] = there ? row[(size_t)i * C + (size_t)z.G * z.dk] : 0.f;
+      g[x][i] = there ? a[(size_t)i * ldl] : 0.f;
     }
-    ss = warp_sum(ss);
-    if (lane == 0) unit_s[x] = i < home.n ? (x < M ? 1.f : 1.f / sqrtf((float)z.dk)) / sqrtf(ss + unit_eps) : 0.f;
   }
-  __syncthreads();
+  if (tid < M) beta_s[tid] = tid < home.n ? logistic_f(proj[(size_t)(home.t0 + tid) * ldp + C + h]) : 0.f;
   const float rate = expf(a_log[h]);
+#pragma unroll
+  for (int x = 0; x < R; ++x) {
+    const int r = tid + 128 * x;
+    const float bias = r < z.dk ? dt_bias[(size_t)h * z.dk + r] : 0.f;
+#pragma unroll
+    for (int i = 0; i < M; ++i) {
+      sums[i] = fmaf(k[x][i], k[x][i], sums[i]);
+      sums[M + i] = fmaf(q[x][i], q[x][i], sums[M + i]);
+      g[x][i] = i < home.n && r < z.dk ? expf(-rate * softplus_f(g[x][i] + bias)) : 1.f;
+    }
+  }
+  scatter_sums<2 * M, 2 * M>(sums, lane & 15);
+  sums[0] += __shfl_xor_sync(0xffffffffu, sums[0], 16);
+  if (lane < 2 * M) part[warp][lane] = sums[0];
+  __syncthreads();
+  if (tid < 2 * M)
+    unit_s[tid] = (tid < M ? 1.f : 1.f / sqrtf((float)z.dk)) /
+                  sqrtf((part[0][tid] + part[1][tid]) + (part[2][tid] + part[3][tid]) + unit_eps);
+  __syncthreads();
   float* rec = records + ((size_t)blockIdx.x * z.H + h) * delta_record(dkp);
   float acc[64];                             // M_ij at i (i + 1) / 2 + j, N_ij at 36 + i (i - 1) / 2 + j
 #pragma unroll
   for (int s = 0; s < 64; ++s) acc[s] = 0.f;
-  for (int r = tid; r < dkp; r += blockDim.x) {
-    float k[M], q[M], g[M];
-    const float bias = r < z.dk ? dt_bias[(size_t)h * z.dk + r] : 0.f;
+#pragma unroll
+  for (int x = 0; x < R; ++x) {
+    const int r = tid + 128 * x;
 #pragma unroll
     for (int i = 0; i < M; ++i) {
-      const bool there = i < home.n && r < z.dk;
-      const float* row = first + (size_t)i * C + (size_t)kh * z.dk + r;
-      q[i] = there ? row[0] * unit_s[M + i] : 0.f;
-      k[i] = there ? row[(size_t)z.G * z.dk] * unit_s[i] : 0.f;
-      g[i] = there ? expf(-rate * softplus_f(low[(size_t)(home.t0 + i) * ldl + (size_t)h * z.dk + r] + bias)) : 1.f;
-    }
-    float pre = 1.f, suf = 1.f;
-#pragma unroll
-    for (int i = 0; i < M; ++i) {
-      pre *= g[i];
-      rec[i * dkp + r] = k[i] * pre;
-      rec[(M + i) * dkp + r] = q[i] * pre;
-    }
-    rec[3 * M * dkp + r] = pre;
-#pragma unroll
-    for (int i = M - 1; i >= 0; --i) {
-      rec[(2 * M + i) * dkp + r] = k[i] * suf;
-      suf *= g[i];
+      k[x][i] *= unit_s[i];
+      q[x][i] *= unit_s[M + i];
     }
 #pragma unroll
     for (int j = 0; j < M; ++j) {
-      float f = k[j];
-      acc[j * (j + 1) / 2 + j] += q[j] * f;
+      float f = k[x][j];
+      acc[j * (j + 1) / 2 + j] += q[x][j] * f;
 #pragma unroll
       for (int i = j + 1; i < M; ++i) {
-        f *= g[i];
-        acc[i * (i + 1) / 2 + j] += q[i] * f;
-        acc[36 + i * (i - 1) / 2 + j] += k[i] * f;
+        f *= g[x][i];
+        acc[i * (i + 1) / 2 + j] += q[x][i] * f;
+        acc[36 + i * (i - 1) / 2 + j] += k[x][i] * f;
       }
     }
   }
-  const int at = scatter_sums_warp<64>(acc, lane);
-  part[warp][at] = acc[0];
-  part[warp][at + 1] = acc[1];
+  scatter_sums<64, 32>(acc, lane);
+  __syncthreads();                           // part is read
+  part[warp][2 * lane] = acc[0];
+  part[warp][2 * lane + 1] = acc[1];
   __syncthreads();
   if (tid < 64) coef[tid] = (part[0][tid] + part[1][tid]) + (part[2][tid] + part[3][tid]);
   __syncthreads();
-  float* X = rec + 25 * dkp;
   if (tid < M) {                             // column tid of X, forward along the rows
     float x[M];
 #pragma unroll
     for (int i = 0; i < M; ++i) {
-      const float beta = i < home.n ? logistic_f(proj[(size_t)(home.t0 + i) * ldp + C + h]) : 0.f;
       float s = i == tid ? 1.f : 0.f;
 #pragma unroll
       for (int j = 0; j < i; ++j) s -= coef[36 + i * (i - 1) / 2 + j] * x[j];
-      x[i] = beta * s;
-      X[i * M + tid] = x[i];
+      x[i] = beta_s[i] * s;
+      x_s[i][tid] = x[i];
     }
   } else if (tid >= 64) {
     const int i = (tid - 64) / M, j = (tid - 64) % M;
-    X[M * M + i * M + j] = j <= i ? coef[i * (i + 1) / 2 + j] : 0.f;
+    m_s[i][j] = j <= i ? coef[i * (i + 1) / 2 + j] : 0.f;
+  }
+  __syncthreads();
+  if (tid < M * M) {
+    const int i = tid / M, j = tid % M;
+    float s = 0.f;
+    for (int y = 0; y <= i; ++y) s = fmaf(m_s[i][y], x_s[y][j], s);
+    rec[25 * dkp + tid] = x_s[i][j];
+    rec[25 * dkp + M * M + tid] = s;
+  }
+#pragma unroll
+  for (int x = 0; x < R; ++x) {
+    const int r = tid + 128 * x;
+    if (r >= dkp) break;
+    float pre = 1.f, suf = 1.f;
+#pragma unroll
+    for (int i = M - 1; i >= 0; --i) {
+      rec[(2 * M + i) * dkp + r] = k[x][i] * suf;
+      suf *= g[x][i];
+    }
+#pragma unroll
+    for (int i = 0; i < M; ++i) {
+      pre *= g[x][i];
+      k[x][i] *= pre;
+      q[x][i] *= pre;
+    }
+    rec[3 * M * dkp + r] = pre;
+    float kx[M];
+#pragma unroll
+    for (int i = 0; i < M; ++i) {
+      float s = 0.f, qm = q[x][i];
+#pragma unroll
+      for (int j = 0; j <= i; ++j) s = fmaf(x_s[i][j], k[x][j], s);
+      kx[i] = s;
+#pragma unroll
+      for (int j = 0; j <= i; ++j) qm = fmaf(-m_s[i][j], kx[j], qm);
+      rec[i * dkp + r] = s;
+      rec[(M + i) * dkp + r] = qm;
+    }
   }
 }
 
-// Block: 16 columns of one head's S for one entry, 8 lanes a column; a group's record comes into one of three stages
-// while the two ahead of it are worked on.
-constexpr int kReadCols = 16, kReadStages = 3;
+// Block: 16 columns of one head's S for one entry, four a warp; a group's record comes into one of three stages while the
+// two ahead of it are worked on.
+constexpr int kReadCols = 16, kReadStages = 3, kReadThreads = 128;      // 128 = 8 tokens x 16 columns: a value a thread
 
-template <int RPL>
-__global__ void __launch_bounds__(kReadCols* kStateLanes)
+template <int DKP, int L>
+__global__ void __launch_bounds__(kReadThreads, 2)      // two blocks an SM: registers for many loads in flight
 channel_delta_read_kernel(const float* __restrict__ records, const float* __restrict__ conv, int C, float* __restrict__ state,
                           long long state_stride, const int* __restrict__ cu_q, const int* __restrict__ slots,
                           float* __restrict__ o_out, DeltaSizes z, int vec) {
   pdl_wait();
   pdl_trigger();
-  constexpr int M = kStateGroup, DKP = RPL * kStateLanes, REC = 25 * DKP + 2 * M * M;
-  extern __shared__ __align__(16) float read_smem[];        // [kReadStages][REC]
-  const int e = blockIdx.z, h = blockIdx.y, tid = threadIdx.x;
-  const int cg = tid / kStateLanes, l = tid % kStateLanes, col = blockIdx.x * kReadCols + cg;
+  typedef StateTile<DKP, L> Tile;
+  constexpr int M = kStateGroup, REC = 25 * DKP + 2 * M * M, NC = Tile::kColumns;
+  constexpr int STAGE = REC + M * kReadCols;
+  extern __shared__ __align__(16) float read_smem[];        // [kReadStages]: the record | v [8][16]
+  __shared__ __align__(16) float u_s[kReadThreads / 32][32 * NC];
+  const int e = blockIdx.z, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int hl = lane % L, set = lane / L, l = lane & 7;
+  const int col_set = blockIdx.x * kReadCols + 4 * warp + set * NC;        // the first column that the lane holds rows of
+  const int col = blockIdx.x * kReadCols + 4 * warp + (lane >> 3);         // the column whose token l the lane finishes
   const bool live = col < z.dv;
   const int t0 = cu_q[e], n = cu_q[e + 1] - t0, groups = (n + M - 1) / M;
   const float* rec0 = records + ((size_t)first_group(cu_q, e) * z.H + h) * REC;
+  const int v_col = blockIdx.x * kReadCols + tid % kReadCols;
+  const float* v_in = conv + 2 * (size_t)z.G * z.dk + (size_t)h * z.dv + v_col;
   auto fetch = [&](int g) {
     if (g < groups) {
       const float* src = rec0 + (size_t)g * z.H * REC;
-      float* dst = read_smem + (g % kReadStages) * REC;
-      for (int i = tid * 4; i < REC; i += kReadCols * kStateLanes * 4) state_copy_16(dst + i, src + i);
+      float* dst = read_smem + (g % kReadStages) * STAGE;
+#pragma unroll
+      for (int i = tid * 4; i < REC; i += kReadThreads * 4) state_copy_16(dst + i, src + i);
+      const int tok = g * M + tid / kReadCols;              // a thread's value of the group
+      if (tok < n && v_col < z.dv) state_copy_4(dst + REC + tid, v_in + (size_t)(t0 + tok) * C);
+      else dst[REC + tid] = 0.f;
     }
     state_copy_commit();
   };
-  const float* v_in = conv + 2 * (size_t)z.G * z.dk + (size_t)h * z.dv + (live ? col : 0);
-  auto value = [&](int g) {
-    const int i = g * M + l;
-    return live && i < n ? __ldg(v_in + (size_t)(t0 + i) * C) : 0.f;
-  };
   fetch(0);
   fetch(1);
-  float* S_col = state + (size_t)slots[e] * state_stride + ((size_t)h * z.dv + (live ? col : 0)) * z.dk;
-  float S[RPL];
-  load_column<RPL>(S, S_col, l, z.dk, live, vec);
-  float v_next = value(0);
+  float* S_head = state + (size_t)slots[e] * state_stride + (size_t)h * z.dv * z.dk;
+  Tile S;
+  S.load(S_head, col_set, z.dv, hl, z.dk, vec);
+  int row_of[M];                             // where the lane's piece of the vector of token slot i lies
+#pragma unroll
+  for (int i = 0; i < M; ++i) row_of[i] = (i ^ l) * DKP + 4 * hl;
   for (int g = 0; g < groups; ++g) {
     state_copy_wait<1>();
     __syncthreads();                         // group g is here for all; group g - 1 is read by all
     fetch(g + 2);
-    const float v = v_next;
-    v_next = value(g + 1);
-    const float* st = read_smem + (g % kReadStages) * REC;
-    float2 a2[M], b2[M];
+    const float* st = read_smem + (g % kReadStages) * STAGE;
+    float p[8 * NC], w[8 * NC];              // slots of column c and token i, at 8 c + i: kx_i . S, then qm_i . S
 #pragma unroll
-    for (int i = 0; i < M; ++i) a2[i] = b2[i] = make_float2(0.f, 0.f);
+    for (int i = 0; i < M; ++i) {
+      float a[NC];
+      S.dot(st + row_of[i], a);
 #pragma unroll
-    for (int j = 0; j < RPL / 4; ++j) {
-      const float2 s0 = make_float2(S[4 * j], S[4 * j + 1]), s1 = make_float2(S[4 * j + 2], S[4 * j + 3]);
-      const float* at = st + 32 * j + 4 * l;
-#pragma unroll
-      for (int i = 0; i < M; ++i) {
-        const float4 kv = *reinterpret_cast<const float4*>(at + i * DKP);
-        a2[i] = fma2(make_float2(kv.x, kv.y), s0, a2[i]);
-        a2[i] = fma2(make_float2(kv.z, kv.w), s1, a2[i]);
-        const float4 qv = *reinterpret_cast<const float4*>(at + (M + i) * DKP);
-        b2[i] = fma2(make_float2(qv.x, qv.y), s0, b2[i]);
-        b2[i] = fma2(make_float2(qv.z, qv.w), s1, b2[i]);
-      }
+      for (int c = 0; c < NC; ++c) p[8 * c + i] = a[c];
     }
-    float p[M], w[M];
-#pragma unroll
-    for (int i = 0; i < M; ++i) { p[i] = a2[i].x + a2[i].y; w[i] = b2[i].x + b2[i].y; }
-    const float rest = v - scatter_sums_8(p, l);           // of token l
-    float o = scatter_sums_8(w, l);
     const float4* X = reinterpret_cast<const float4*>(st + 25 * DKP + l * M);
     const float4 x0 = X[0], x1 = X[1], m0 = X[M * M / 4], m1 = X[M * M / 4 + 1];
     const float xr[M] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
     const float mr[M] = {m0.x, m0.y, m0.z, m0.w, m1.x, m1.y, m1.z, m1.w};
-    float u = 0.f;
-#pragma unroll
-    for (int j = 0; j < M; ++j) u = fmaf(xr[j], __shfl_sync(0xffffffffu, rest, j, kStateLanes), u);
-    float us[M];
+    float u = 0.f, o = 0.f;
 #pragma unroll
     for (int j = 0; j < M; ++j) {
-      us[j] = __shfl_sync(0xffffffffu, u, j, kStateLanes);
-      o = fmaf(mr[j], us[j], o);
+      const float v = st[REC + j * kReadCols + 4 * warp + (lane >> 3)];
+      u = fmaf(xr[j], v, u);
+      o = fmaf(mr[j], v, o);
+    }
+    permuted_sums<8 * NC, L>(p);
+    u -= p[0];
+    Tile::share(u_s[warp], set, hl, u);
+#pragma unroll
+    for (int i = 0; i < M; ++i) {            // does not wait for u: fills the exchanges' latency
+      float a[NC];
+      S.dot(st + M * DKP + row_of[i], a);
+#pragma unroll
+      for (int c = 0; c < NC; ++c) w[8 * c + i] = a[c];
     }
 #pragma unroll
-    for (int j = 0; j < RPL / 4; ++j) {
-      const float* at = st + 2 * M * DKP + 32 * j + 4 * l;
-      const float4 wh = *reinterpret_cast<const float4*>(at + M * DKP);
-      float2 s0 = make_float2(S[4 * j] * wh.x, S[4 * j + 1] * wh.y), s1 = make_float2(S[4 * j + 2] * wh.z, S[4 * j + 3] * wh.w);
+    for (int j = 0; j < Tile::kPieces; ++j) {
+      const float4 wh = *reinterpret_cast<const float4*>(st + 3 * M * DKP + 4 * hl + 4 * L * j);
 #pragma unroll
-      for (int i = 0; i < M; ++i) {
-        const float4 kv = *reinterpret_cast<const float4*>(at + i * DKP);
-        s0 = fma2(make_float2(kv.x, kv.y), make_float2(us[i], us[i]), s0);
-        s1 = fma2(make_float2(kv.z, kv.w), make_float2(us[i], us[i]), s1);
+      for (int c = 0; c < NC; ++c) {
+        S.s[c][2 * j].x *= wh.x; S.s[c][2 * j].y *= wh.y;
+        S.s[c][2 * j + 1].x *= wh.z; S.s[c][2 * j + 1].y *= wh.w;
       }
-      S[4 * j] = s0.x; S[4 * j + 1] = s0.y; S[4 * j + 2] = s1.x; S[4 * j + 3] = s1.y;
     }
+    __syncwarp();
+#pragma unroll
+    for (int j = 0; j < M; ++j) {
+      alignas(16) float uj[NC];
+      Tile::shared(u_s[warp], set, hl, j, uj);
+      S.add(st + (2 * M + j) * DKP + 4 * hl, uj);
+    }
+    permuted_sums<8 * NC, L>(w);
+    o += w[0];
     if (live && g * M + l < n) o_out[((size_t)(t0 + g * M + l) * z.H + h) * z.dv + col] = o;
   }
   state_copy_wait<0>();
-  store_column<RPL>(S, S_col, l, z.dk, live, vec);
+  S.store(S_head, col_set, z.dv, hl, z.dk, vec);
 }
 
 }  // namespace srlm
@@ -383,35 +437,48 @@ extern "C" int srlm_channel_delta_walk(const float* proj, long long ldp, const f
 extern "C" int srlm_channel_delta_record(int dk) { return dk > 0 && dk <= 256 ? delta_record(rows_per_lane(dk) * kStateLanes) : 0; }
 
 // groups: how many groups of 8 tokens the step's entries have together; records float32 [groups, H, record]; conv float32
-// [T, C]; o_out float32 [T, H dv].
+// [T, C].
 extern "C" int srlm_channel_delta_groups(const float* conv, const float* proj, long long ldp, const float* low, long long ldl,
-                                         const float* a_log, const float* dt_bias, float* state, long long state_stride,
-                                         const int* cu_q, const int* slots, int n_entries, float* records, float* o_out, int groups,
-                                         int H, int G, int dk, int dv, float unit_eps, cudaStream_t stream) {
+                                         const float* a_log, const float* dt_bias, const int* cu_q, int n_entries,
+                                         float* records, int groups, int H, int G, int dk, int dv, float unit_eps,
+                                         cudaStream_t stream) {
   if (n_entries <= 0 || groups <= 0) return ST_OK;
   if (int r = channel_delta_ok("channel_delta_groups", H, G, dk, dv, n_entries)) return r;
   const int C = 2 * G * dk + H * dv;
-  if (!srlm_channel_delta_record(dk) || ldp < C + H || ldl < (long long)H * dk || state_stride < (long long)H * dk * dv)
-    return refuse(ST_BAD_SIZE, "channel_delta_groups: dk=%d (at most 256) ldp=%lld ldl=%lld state=%lld", dk, ldp, ldl, state_stride);
-  if (((uintptr_t)records & 15) != 0) return refuse(ST_BAD_ALIGN, "channel_delta_groups: records must be 16-byte aligned");
-  const int rpl = rows_per_lane(dk), dkp = rpl * kStateLanes;
+  if (!srlm_channel_delta_record(dk) || ldp < C + H || ldl < (long long)H * dk)
+    return refuse(ST_BAD_SIZE, "channel_delta_groups: dk=%d (at most 256) ldp=%lld ldl=%lld", dk, ldp, ldl);
+  const int dkp = rows_per_lane(dk) * kStateLanes;
+  auto kern = dkp <= 128 ? channel_delta_groups_kernel<1> : channel_delta_groups_kernel<2>;
+  launch_pdl(kern, dim3(groups, H), dim3(128), 0, stream, conv, C, proj, ldp, low, ldl, a_log, dt_bias, cu_q, n_entries, records,
+             DeltaSizes{H, G, dk, dv}, dkp, unit_eps);
+  return launched();
+}
+
+// The walk along the records that srlm_channel_delta_groups made; o_out float32 [T, H dv].
+extern "C" int srlm_channel_delta_read(const float* records, const float* conv, float* state, long long state_stride,
+                                       const int* cu_q, const int* slots, int n_entries, float* o_out, int H, int G, int dk,
+                                       int dv, cudaStream_t stream) {
+  if (n_entries <= 0) return ST_OK;
+  if (int r = channel_delta_ok("channel_delta_read", H, G, dk, dv, n_entries)) return r;
+  if (!srlm_channel_delta_record(dk) || state_stride < (long long)H * dk * dv)
+    return refuse(ST_BAD_SIZE, "channel_delta_read: dk=%d (at most 256) state=%lld", dk, state_stride);
+  if (((uintptr_t)records & 15) != 0) return refuse(ST_BAD_ALIGN, "channel_delta_read: records must be 16-byte aligned");
+  const int C = 2 * G * dk + H * dv, rpl = rows_per_lane(dk);
   const DeltaSizes z{H, G, dk, dv};
-  launch_pdl(channel_delta_groups_kernel, dim3(groups, H), dim3(128), 0, stream, conv, C, proj, ldp, low, ldl, a_log, dt_bias,
-             cu_q, n_entries, records, z, dkp, unit_eps);
   const int vec = dk % 4 == 0 && state_stride % 4 == 0 && ((uintptr_t)state & 15) == 0;
-  const size_t smem = (size_t)kReadStages * delta_record(dkp) * sizeof(float);
+  const size_t smem = (size_t)kReadStages * (delta_record(rpl * kStateLanes) + kStateGroup * kReadCols) * sizeof(float);
   dim3 grid((dv + kReadCols - 1) / kReadCols, H, n_entries);
-#define SRLM_CDR(R)                                                                                                     \
+#define SRLM_CDR(ROWS, L)                                                                                               \
   do {                                                                                                                  \
-    auto kern = channel_delta_read_kernel<R>;                                                                           \
-    if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);           \
-    launch_pdl_if(false, kern, grid, dim3(kReadCols * kStateLanes), smem, stream, records, conv, C, state, state_stride, cu_q, \
-                  slots, o_out, z, vec);                                                                                \
+    auto kern = channel_delta_read_kernel<ROWS, L>;                                                                     \
+    if (smem > 40 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);           \
+    launch_pdl_if(false, kern, grid, dim3(kReadThreads), smem, stream, records, conv, C, state, state_stride, cu_q, slots, \
+                  o_out, z, vec);                                                                                       \
   } while (0)
-  if (rpl == 4) SRLM_CDR(4);
-  else if (rpl == 8) SRLM_CDR(8);
-  else if (rpl == 16) SRLM_CDR(16);
-  else SRLM_CDR(32);
+  if (rpl == 4) SRLM_CDR(32, 8);
+  else if (rpl == 8) SRLM_CDR(64, 16);
+  else if (rpl == 16) SRLM_CDR(128, 32);
+  else SRLM_CDR(256, 32);
 #undef SRLM_CDR
   return launched();
 }

@@ -34,6 +34,63 @@ __global__ void short_conv_kernel(ConvInput in, const float* __restrict__ w, con
   }
 }
 
+// The same for steps of many tokens: a thread takes one channel of TOK neighbouring tokens, fetches their inputs at once and
+// keeps the weights and the TAPS - 1 inputs behind the token in registers.
+template <int TAPS, int TOK, typename TO>
+__global__ void __launch_bounds__(256)
+short_conv_run_kernel(ConvInput in, const float* __restrict__ w, const float* __restrict__ out_bias,
+                      const int* __restrict__ entry_of_token, const int* __restrict__ cu_q, const int* __restrict__ slots,
+                      float* __restrict__ out, TO* __restrict__ out_low, int T, int silu) {
+  pdl_wait();
+  pdl_trigger();
+  const int c = blockIdx.x * blockDim.x + threadIdx.x, t0 = blockIdx.y * TOK;
+  if (c >= in.C) return;
+  const float bias = in.in_bias ? in.in_bias[c] : 0.f, rest = out_bias ? out_bias[c] : 0.f;
+  float u[TOK], wt[TAPS], back[TAPS - 1];
+#pragma unroll
+  for (int i = 0; i < TOK; ++i) u[i] = t0 + i < T ? in.proj[(size_t)(t0 + i) * in.ld + c] + bias : 0.f;
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) wt[j] = w[(size_t)c * TAPS + j];
+  auto behind = [&](int t, int e) {            // back[j]: the input TAPS - 1 - j tokens ahead of token t of entry e
+    const int idx = t - cu_q[e];
+    const float* carry = in.state + (size_t)slots[e] * in.state_stride + in.state_off + c;
+#pragma unroll
+    for (int j = 0; j < TAPS - 1; ++j) {
+      const int ago = TAPS - 1 - j;
+      back[j] = ago <= idx ? in.proj[(size_t)(t - ago) * in.ld + c] + bias : carry[(size_t)(j + idx) * in.C];
+    }
+  };
+  auto finish = [&](int t, float now) {
+    float acc = 0.f;
+#pragma unroll
+    for (int j = 0; j < TAPS - 1; ++j) acc = fmaf(wt[j], back[j], acc);
+    acc = fmaf(wt[TAPS - 1], now, acc);
+#pragma unroll
+    for (int j = 0; j < TAPS - 2; ++j) back[j] = back[j + 1];
+    back[TAPS - 2] = now;
+    float y = acc + rest;
+    if (silu) y = silu_of(y);
+    out[(size_t)t * in.C + c] = y;
+    if (out_low) out_low[(size_t)t * in.C + c] = from_float<TO>(y);
+  };
+  const int e0 = entry_of_token[t0];
+  behind(t0, e0);
+  if (t0 + TOK <= T && entry_of_token[t0 + TOK - 1] == e0) {     // whole and of one entry: nothing to look up on the way
+#pragma unroll
+    for (int i = 0; i < TOK; ++i) finish(t0 + i, u[i]);
+    return;
+  }
+  int entry = e0;
+#pragma unroll
+  for (int i = 0; i < TOK; ++i) {
+    const int t = t0 + i;
+    if (t >= T) break;
+    const int e = entry_of_token[t];
+    if (e != entry) behind(t, entry = e);      // the same for the whole block
+    finish(t, u[i]);
+  }
+}
+
 // New carry of entry e: the last taps - 1 of (old carry, the portion's inputs).
 __global__ void conv_carry_kernel(ConvInput in, float* __restrict__ state, const int* __restrict__ cu_q,
                                   const int* __restrict__ slots) {
@@ -140,6 +197,19 @@ extern "C" int srlm_short_conv(const float* proj, long long ld, const float* in_
   if (T <= 0) return ST_OK;
   if (int r = conv_input_ok("short_conv", taps, C, ld, state_stride, state_off)) return r;
   ConvInput in{proj, ld, in_bias, state, state_stride, state_off, taps, C};
+  constexpr int kRun = 16;
+  if (T >= 8 * kRun && taps >= 2 && taps <= 4) {
+    dim3 runs((unsigned)((C + 255) / 256), (unsigned)((T + kRun - 1) / kRun));
+#define SRLM_CONV_RUN(TAPS)                                                                                             \
+  SRLM_DISPATCH_ACT(out_low ? low_dtype : DT_F32, TO,                                                                   \
+                    launch_pdl(short_conv_run_kernel<TAPS, kRun, TO>, runs, dim3(256), 0, stream, in, w, out_bias,      \
+                               entry_of_token, cu_q, slots, out, (TO*)out_low, T, silu))
+    if (taps == 2) SRLM_CONV_RUN(2);
+    else if (taps == 3) SRLM_CONV_RUN(3);
+    else SRLM_CONV_RUN(4);
+#undef SRLM_CONV_RUN
+    return launched();
+  }
   dim3 grid((unsigned)((C + 255) / 256), (unsigned)T);
   if (T > 65535) return refuse(ST_BAD_SIZE, "short_conv: %d tokens", T);
   SRLM_DISPATCH_ACT(out_low ? low_dtype : DT_F32, TO,

@@ -125,7 +125,8 @@ state_space_groups_kernel(const float* __restrict__ conv, int C, const float* __
 #pragma unroll
       for (int j = 0; j <= i; ++j) acc[8 * i + j] = fmaf(c[i], b[j], acc[8 * i + j]);
   }
-  const int at = scatter_sums_warp<64>(acc, lane);
+  scatter_sums<64, 32>(acc, lane);
+  const int at = 2 * lane;
   sums[warp][at] = acc[0];
   sums[warp][at + 1] = acc[1];
   __syncwarp();
@@ -146,114 +147,113 @@ state_space_groups_kernel(const float* __restrict__ conv, int C, const float* __
   }
 }
 
-constexpr int kSpaceCols = 16, kSpaceStages = 3;
+constexpr int kSpaceCols = 16, kSpaceStages = 3, kSpaceThreads = 128;  // 128 = 8 tokens x 16 columns: a value a thread
 
-// Block: 16 columns of one head's S for one entry, 8 lanes a column.
-template <int RPL>
-__global__ void __launch_bounds__(kSpaceCols* kStateLanes)
+// Block: 16 columns of one head's S for one entry, four a warp.
+template <int NP, int L>
+__global__ void __launch_bounds__(kSpaceThreads, 4)     // four blocks an SM: up to 128 registers, loads in flight
 state_space_read_kernel(const float* __restrict__ records, const float* __restrict__ conv, int C, const float* __restrict__ D,
                         float* __restrict__ state, long long state_stride, const int* __restrict__ cu_q,
                         const int* __restrict__ slots, float* __restrict__ y_out, SpaceSizes z, int vec, int vec_rows) {
   pdl_wait();
   pdl_trigger();
-  constexpr int M = kStateGroup, NP = RPL * kStateLanes, STAGE = 2 * M * NP + kSpaceRecord;
-  constexpr int kThreads = kSpaceCols * kStateLanes;
-  extern __shared__ __align__(16) float read_smem[];        // [kSpaceStages]: C rows [8][NP] | B rows [8][NP] | the record
-  const int e = blockIdx.z, h = blockIdx.y, tid = threadIdx.x;
+  typedef StateTile<NP, L> Tile;
+  constexpr int M = kStateGroup, STAGE = 2 * M * NP + kSpaceRecord + M * kSpaceCols, NC = Tile::kColumns;
+  extern __shared__ __align__(16) float read_smem[];        // [kSpaceStages]: C rows [8][NP] | B rows [8][NP] | the record | x [8][16]
+  __shared__ __align__(16) float w_s[kSpaceThreads / 32][32 * NC];
+  const int e = blockIdx.z, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int grp = h / (z.H / z.G);
-  const int cg = tid / kStateLanes, l = tid % kStateLanes, col = blockIdx.x * kSpaceCols + cg;
+  const int hl = lane % L, set = lane / L, l = lane & 7;
+  const int col_set = blockIdx.x * kSpaceCols + 4 * warp + set * NC;       // the first column that the lane holds rows of
+  const int col = blockIdx.x * kSpaceCols + 4 * warp + (lane >> 3);        // the column whose token l the lane finishes
   const bool live = col < z.P;
   const int t0 = cu_q[e], n = cu_q[e + 1] - t0, groups = (n + M - 1) / M;
   const float* rec0 = records + ((size_t)first_group(cu_q, e) * z.H + h) * kSpaceRecord;
   const float* rows0 = conv + (size_t)t0 * C + (size_t)z.H * z.P + (size_t)grp * z.N;
-  for (int i = tid; i < kSpaceStages * STAGE; i += kThreads) read_smem[i] = 0.f;
+  for (int i = tid; i < kSpaceStages * STAGE; i += kSpaceThreads) read_smem[i] = 0.f;
   __syncthreads();                           // rows behind N and tokens behind the portion stay zero (or finite)
+  constexpr int kCopies = 2 * M * NP / 4 / kSpaceThreads;   // a thread's 16-byte pieces of a group's rows
+  int copy_to[kCopies], copy_tok[kCopies];
+  unsigned copy_from[kCopies];
+#pragma unroll
+  for (int i = 0; i < kCopies; ++i) {
+    const int x = tid + i * kSpaceThreads, pieces = z.N / 4, row = pieces ? x / pieces : 2 * M, at = (x - row * pieces) * 4;
+    copy_tok[i] = row < 2 * M ? row % M : M;                // M: no piece
+    copy_to[i] = row * NP + at;
+    copy_from[i] = (unsigned)(row % M) * (unsigned)C + (row < M ? (unsigned)(z.G * z.N) : 0u) + (unsigned)at;
+  }
+  const int x_col = blockIdx.x * kSpaceCols + tid % kSpaceCols;
+  const float* x_in = conv + (size_t)h * z.P + x_col;
   auto fetch = [&](int g) {
     if (g < groups) {
       float* dst = read_smem + (g % kSpaceStages) * STAGE;
       const int m = min(M, n - g * M);
       const float* src = rows0 + (size_t)g * M * C;
       if (vec_rows) {
-        const int pieces = z.N / 4;
-        for (int i = tid; i < 2 * M * pieces; i += kThreads) {
-          const int row = i / pieces, x = (i - row * pieces) * 4, tok = row % M;
-          if (tok < m)
-            state_copy_16(dst + row * NP + x, src + (size_t)tok * C + (row < M ? (size_t)z.G * z.N : 0) + x);
-        }
+#pragma unroll
+        for (int i = 0; i < kCopies; ++i)
+          if (copy_tok[i] < m) state_copy_16(dst + copy_to[i], src + copy_from[i]);
       } else {
-        for (int i = tid; i < 2 * M * z.N; i += kThreads) {
+        for (int i = tid; i < 2 * M * z.N; i += kSpaceThreads) {
           const int row = i / z.N, x = i - row * z.N, tok = row % M;
           if (tok < m)
             state_copy_4(dst + row * NP + x, src + (size_t)tok * C + (row < M ? (size_t)z.G * z.N : 0) + x);
         }
       }
       if (tid < kSpaceRecord / 4) state_copy_16(dst + 2 * M * NP + 4 * tid, rec0 + (size_t)g * z.H * kSpaceRecord + 4 * tid);
+      const int tok = tid / kSpaceCols;                     // a thread's value of the group
+      float* x_at = dst + 2 * M * NP + kSpaceRecord + tid;
+      if (tok < m && x_col < z.P) state_copy_4(x_at, x_in + (size_t)(t0 + g * M + tok) * C);
+      else *x_at = 0.f;
     }
     state_copy_commit();
-  };
-  const float* x_in = conv + (size_t)h * z.P + (live ? col : 0);
-  auto value = [&](int g) {
-    const int i = g * M + l;
-    return live && i < n ? __ldg(x_in + (size_t)(t0 + i) * C) : 0.f;
   };
   fetch(0);
   fetch(1);
   const float d_h = D[h];
-  float* S_col = state + (size_t)slots[e] * state_stride + ((size_t)h * z.P + (live ? col : 0)) * z.N;
-  float S[RPL];
-  load_column<RPL>(S, S_col, l, z.N, live, vec);
-  float x_next = value(0);
+  float* S_head = state + (size_t)slots[e] * state_stride + (size_t)h * z.P * z.N;
+  Tile S;
+  S.load(S_head, col_set, z.P, hl, z.N, vec);
+  int row_of[M];                             // where the lane's piece of the vector of token slot i lies
+#pragma unroll
+  for (int i = 0; i < M; ++i) row_of[i] = (i ^ l) * NP + 4 * hl;
   for (int g = 0; g < groups; ++g) {
     state_copy_wait<1>();
     __syncthreads();                         // group g is here for all; group g - 1 is read by all
     fetch(g + 2);
-    const float x = x_next;
-    x_next = value(g + 1);
     const float* st = read_smem + (g % kSpaceStages) * STAGE;
     const float* rec = st + 2 * M * NP;
-    float2 b2[M];
+    const float x = rec[kSpaceRecord + l * kSpaceCols + 4 * warp + (lane >> 3)];
+    float p[8 * NC];                         // slots of column c and token i: C_i . S at 8 c + i
 #pragma unroll
-    for (int i = 0; i < M; ++i) b2[i] = make_float2(0.f, 0.f);
+    for (int i = 0; i < M; ++i) {
+      float b[NC];
+      S.dot(st + row_of[i], b);
 #pragma unroll
-    for (int j = 0; j < RPL / 4; ++j) {
-      const float2 s0 = make_float2(S[4 * j], S[4 * j + 1]), s1 = make_float2(S[4 * j + 2], S[4 * j + 3]);
-#pragma unroll
-      for (int i = 0; i < M; ++i) {
-        const float4 cv = *reinterpret_cast<const float4*>(st + i * NP + 32 * j + 4 * l);
-        b2[i] = fma2(make_float2(cv.x, cv.y), s0, b2[i]);
-        b2[i] = fma2(make_float2(cv.z, cv.w), s1, b2[i]);
-      }
+      for (int c = 0; c < NC; ++c) p[8 * c + i] = b[c];
     }
-    float p[M], w[M];
-#pragma unroll
-    for (int i = 0; i < M; ++i) p[i] = b2[i].x + b2[i].y;
-    float y = scatter_sums_8(p, l) * rec[M * M + l] + d_h * x;
+    Tile::share(w_s[warp], set, hl, rec[M * M + M + l] * x);
+    permuted_sums<8 * NC, L>(p);
+    float y = p[0] * rec[M * M + l] + d_h * x;
     const float4 m0 = *reinterpret_cast<const float4*>(rec + l * M), m1 = *reinterpret_cast<const float4*>(rec + l * M + 4);
-    const float4 r0 = *reinterpret_cast<const float4*>(rec + M * M + M), r1 = *reinterpret_cast<const float4*>(rec + M * M + M + 4);
     const float mr[M] = {m0.x, m0.y, m0.z, m0.w, m1.x, m1.y, m1.z, m1.w};
-    const float rd[M] = {r0.x, r0.y, r0.z, r0.w, r1.x, r1.y, r1.z, r1.w};
-#pragma unroll
-    for (int j = 0; j < M; ++j) {
-      const float xj = __shfl_sync(0xffffffffu, x, j, kStateLanes);
-      y = fmaf(mr[j], xj, y);
-      w[j] = rd[j] * xj;
-    }
+    __syncwarp();
     const float keep = rec[M * M + M - 1];
 #pragma unroll
-    for (int j = 0; j < RPL / 4; ++j) {
-      float2 s0 = make_float2(S[4 * j] * keep, S[4 * j + 1] * keep), s1 = make_float2(S[4 * j + 2] * keep, S[4 * j + 3] * keep);
+    for (int c = 0; c < NC; ++c)
 #pragma unroll
-      for (int i = 0; i < M; ++i) {
-        const float4 bv = *reinterpret_cast<const float4*>(st + (M + i) * NP + 32 * j + 4 * l);
-        s0 = fma2(make_float2(bv.x, bv.y), make_float2(w[i], w[i]), s0);
-        s1 = fma2(make_float2(bv.z, bv.w), make_float2(w[i], w[i]), s1);
-      }
-      S[4 * j] = s0.x; S[4 * j + 1] = s0.y; S[4 * j + 2] = s1.x; S[4 * j + 3] = s1.y;
+      for (int j = 0; j < 2 * Tile::kPieces; ++j) { S.s[c][j].x *= keep; S.s[c][j].y *= keep; }
+#pragma unroll
+    for (int j = 0; j < M; ++j) {
+      alignas(16) float wj[NC];
+      Tile::shared(w_s[warp], set, hl, j, wj);
+      S.add(st + (M + j) * NP + 4 * hl, wj);
+      y = fmaf(mr[j], __shfl_sync(0xffffffffu, x, j, M), y);
     }
     if (live && g * M + l < n) y_out[((size_t)(t0 + g * M + l) * z.H + h) * z.P + col] = y;
   }
   state_copy_wait<0>();
-  store_column<RPL>(S, S_col, l, z.N, live, vec);
+  S.store(S_head, col_set, z.P, hl, z.N, vec);
 }
 
 // A block per (part, token): out = w * u / sqrt(mean(u^2) + eps) over the part, u = y * silu(z).
@@ -327,32 +327,42 @@ extern "C" int srlm_state_space_record(int N) { return N > 0 && N <= 256 ? kSpac
 // groups: how many groups of 8 tokens the step's entries have together; records float32 [groups, H, record]; conv float32
 // [T, H P + 2 G N].
 extern "C" int srlm_state_space_groups(const float* conv, const float* proj, long long ldp, const float* dt_bias,
-                                       const float* a_log, const float* D, float* state, long long state_stride,
-                                       const int* cu_q, const int* slots, int n_entries, float* records, float* y_out, int groups,
-                                       int H, int G, int N, int P, cudaStream_t stream) {
+                                       const float* a_log, const int* cu_q, int n_entries, float* records, int groups, int H,
+                                       int G, int N, int P, cudaStream_t stream) {
   if (n_entries <= 0 || groups <= 0) return ST_OK;
-  if (int r = space_ok("state_space_groups", H, G, N, P, ldp, state_stride, n_entries)) return r;
-  if (N > 256) return refuse(ST_BAD_SIZE, "state_space_groups: state=%d (at most 256)", N);
-  if (((uintptr_t)records & 15) != 0) return refuse(ST_BAD_ALIGN, "state_space_groups: records must be 16-byte aligned");
+  if (int r = space_ok("state_space_groups", H, G, N, P, ldp, 0x7fffffffffffLL, n_entries)) return r;
+  const int inner = H * P, C = inner + 2 * G * N;
+  launch_pdl(state_space_groups_kernel, dim3(groups, (H + 3) / 4), dim3(128), 0, stream, conv, C, proj + inner + C, ldp, dt_bias,
+             a_log, cu_q, n_entries, records, SpaceSizes{H, G, N, P});
+  return launched();
+}
+
+// The walk along the records that srlm_state_space_groups made; y_out float32 [T, H P].
+extern "C" int srlm_state_space_read(const float* records, const float* conv, const float* D, float* state,
+                                     long long state_stride, const int* cu_q, const int* slots, int n_entries, float* y_out,
+                                     int H, int G, int N, int P, cudaStream_t stream) {
+  if (n_entries <= 0) return ST_OK;
+  if (int r = space_ok("state_space_read", H, G, N, P, 0x7fffffffffffLL, state_stride, n_entries)) return r;
+  if (N > 256) return refuse(ST_BAD_SIZE, "state_space_read: state=%d (at most 256)", N);
+  if (((uintptr_t)records & 15) != 0) return refuse(ST_BAD_ALIGN, "state_space_read: records must be 16-byte aligned");
   const int inner = H * P, C = inner + 2 * G * N, rpl = rows_per_lane(N);
   const SpaceSizes z{H, G, N, P};
-  launch_pdl(state_space_groups_kernel, dim3(groups, (H + 3) / 4), dim3(128), 0, stream, conv, C, proj + inner + C, ldp, dt_bias,
-             a_log, cu_q, n_entries, records, z);
   const int vec = N % 4 == 0 && state_stride % 4 == 0 && ((uintptr_t)state & 15) == 0;
   const int vec_rows = N % 4 == 0 && inner % 4 == 0 && ((uintptr_t)conv & 15) == 0;
-  const size_t smem = (size_t)kSpaceStages * (2 * kStateGroup * rpl * kStateLanes + kSpaceRecord) * sizeof(float);
+  const size_t smem = (size_t)kSpaceStages * (2 * kStateGroup * rpl * kStateLanes + kSpaceRecord + kStateGroup * kSpaceCols) *
+                      sizeof(float);
   dim3 grid((P + kSpaceCols - 1) / kSpaceCols, H, n_entries);
-#define SRLM_SSR(R)                                                                                                     \
+#define SRLM_SSR(ROWS, L)                                                                                               \
   do {                                                                                                                  \
-    auto kern = state_space_read_kernel<R>;                                                                             \
-    if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);           \
-    launch_pdl_if(false, kern, grid, dim3(kSpaceCols * kStateLanes), smem, stream, records, conv, C, D, state, state_stride, \
-                  cu_q, slots, y_out, z, vec, vec_rows);                                                                \
+    auto kern = state_space_read_kernel<ROWS, L>;                                                                       \
+    if (smem > 40 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);           \
+    launch_pdl_if(false, kern, grid, dim3(kSpaceThreads), smem, stream, records, conv, C, D, state, state_stride, cu_q, slots, \
+                  y_out, z, vec, vec_rows);                                                                             \
   } while (0)
-  if (rpl == 4) SRLM_SSR(4);
-  else if (rpl == 8) SRLM_SSR(8);
-  else if (rpl == 16) SRLM_SSR(16);
-  else SRLM_SSR(32);
+  if (rpl == 4) SRLM_SSR(32, 8);
+  else if (rpl == 8) SRLM_SSR(64, 16);
+  else if (rpl == 16) SRLM_SSR(128, 32);
+  else SRLM_SSR(256, 32);
 #undef SRLM_SSR
   return launched();
 }

@@ -67,41 +67,139 @@ __device__ __forceinline__ void store_column(const float (&S)[RPL], float* colum
   }
 }
 
-// p[0..7]: a lane's share of eight sums over the 8 lanes of a column; returns sum number l to lane l.
-__device__ __forceinline__ float scatter_sums_8(const float (&p)[kStateGroup], int l) {
-  float a[4], b[2];
+// A warp of a grouped walk holds four columns of S: L lanes a set of L / 8 columns, lane hl of the set the rows
+// 4 hl + 4 L j + {0..3}.  More lanes a column mean fewer bytes of shared memory a product (a lane's row pieces serve L / 8
+// columns), fewer lanes mean fewer exchanges a sum.
+//
+// Lane hl finishes token hl & 7 of the set's column hl >> 3.  It keeps its columns in slots, slot c for column
+// c ^ (hl >> 3), and forms a group's sums in slots of tokens, slot i for token i ^ (hl & 7): then the half of the sums
+// that a lane gives away in an exchange always lies in the upper slots (permuted_sums), and no value is selected by lane.
+template <int ROWS, int L>
+struct StateTile {
+  static constexpr int kColumns = L / kStateLanes;          // a lane's columns
+  static constexpr int kPieces = ROWS / (4 * L);            // a lane's pieces of four rows
+  static_assert(L >= 8 && L <= 32 && kPieces * 4 * L == ROWS, "whole pieces");
+  float2 s[kColumns][2 * kPieces];
+
+  __device__ __forceinline__ void load(const float* head, int first, int columns, int hl, int rows, bool vec) {
 #pragma unroll
-  for (int s = 0; s < 4; ++s) {
-    const float keep = l & 4 ? p[s + 4] : p[s], give = l & 4 ? p[s] : p[s + 4];
-    a[s] = keep + __shfl_xor_sync(0xffffffffu, give, 4);
-  }
+    for (int c = 0; c < kColumns; ++c)
 #pragma unroll
-  for (int s = 0; s < 2; ++s) {
-    const float keep = l & 2 ? a[s + 2] : a[s], give = l & 2 ? a[s] : a[s + 2];
-    b[s] = keep + __shfl_xor_sync(0xffffffffu, give, 2);
+      for (int j = 0; j < kPieces; ++j) {
+        const int r = 4 * hl + 4 * L * j, col = first + (c ^ (hl >> 3));
+        const float* at = head + (size_t)col * rows + r;
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (col < columns) {
+          if (vec) {
+            if (r < rows) v = *reinterpret_cast<const float4*>(at);
+          } else {
+            if (r < rows) v.x = at[0];
+            if (r + 1 < rows) v.y = at[1];
+            if (r + 2 < rows) v.z = at[2];
+            if (r + 3 < rows) v.w = at[3];
+          }
+        }
+        s[c][2 * j] = make_float2(v.x, v.y);
+        s[c][2 * j + 1] = make_float2(v.z, v.w);
+      }
   }
-  const float keep = l & 1 ? b[1] : b[0], give = l & 1 ? b[0] : b[1];
-  return keep + __shfl_xor_sync(0xffffffffu, give, 1);
+  __device__ __forceinline__ void store(float* head, int first, int columns, int hl, int rows, bool vec) const {
+#pragma unroll
+    for (int c = 0; c < kColumns; ++c)
+#pragma unroll
+      for (int j = 0; j < kPieces; ++j) {
+        const int r = 4 * hl + 4 * L * j, col = first + (c ^ (hl >> 3));
+        float* at = head + (size_t)col * rows + r;
+        if (col >= columns) continue;
+        const float2 a = s[c][2 * j], b = s[c][2 * j + 1];
+        if (vec) {
+          if (r < rows) *reinterpret_cast<float4*>(at) = make_float4(a.x, a.y, b.x, b.y);
+        } else {
+          if (r < rows) at[0] = a.x;
+          if (r + 1 < rows) at[1] = a.y;
+          if (r + 2 < rows) at[2] = b.x;
+          if (r + 3 < rows) at[3] = b.y;
+        }
+      }
+  }
+  // The lane's share of x . S[:, c] for its columns; x: where its first piece of a vector over the rows lies in shared memory.
+  __device__ __forceinline__ void dot(const float* x, float (&out)[kColumns]) const {
+    float2 acc[kColumns];
+#pragma unroll
+    for (int j = 0; j < kPieces; ++j) {
+      const float4 v = *reinterpret_cast<const float4*>(x + 4 * L * j);
+      const float2 lo = make_float2(v.x, v.y), hi = make_float2(v.z, v.w);
+#pragma unroll
+      for (int c = 0; c < kColumns; ++c) {
+        acc[c] = fma2(lo, s[c][2 * j], j == 0 ? make_float2(0.f, 0.f) : acc[c]);
+        acc[c] = fma2(hi, s[c][2 * j + 1], acc[c]);
+      }
+    }
+#pragma unroll
+    for (int c = 0; c < kColumns; ++c) out[c] = acc[c].x + acc[c].y;
+  }
+  // S[:, c] += x u[c]
+  __device__ __forceinline__ void add(const float* x, const float (&u)[kColumns]) {
+#pragma unroll
+    for (int j = 0; j < kPieces; ++j) {
+      const float4 v = *reinterpret_cast<const float4*>(x + 4 * L * j);
+      const float2 lo = make_float2(v.x, v.y), hi = make_float2(v.z, v.w);
+#pragma unroll
+      for (int c = 0; c < kColumns; ++c) {
+        const float2 uu = make_float2(u[c], u[c]);
+        s[c][2 * j] = fma2(lo, uu, s[c][2 * j]);
+        s[c][2 * j + 1] = fma2(hi, uu, s[c][2 * j + 1]);
+      }
+    }
+  }
+
+  // A number a (token, column) to all lanes of the column's set, by way of shared memory (32 kColumns floats a warp; a
+  // __syncwarp between share and shared): every lane reads its columns in the order of its slots.
+  static __device__ __forceinline__ void share(float* buf, int set, int hl, float u) {
+#pragma unroll
+    for (int x = 0; x < kColumns; ++x)
+      buf[((set * kColumns + x) * kStateGroup + (hl & 7)) * kColumns + ((hl >> 3) ^ x)] = u;
+  }
+  static __device__ __forceinline__ void shared(const float* buf, int set, int hl, int token, float (&u)[kColumns]) {
+    const float* at = buf + ((set * kColumns + (hl >> 3)) * kStateGroup + token) * kColumns;
+    if (kColumns == 4) *reinterpret_cast<float4*>(u) = *reinterpret_cast<const float4*>(at);
+    else if (kColumns == 2) *reinterpret_cast<float2*>(u) = *reinterpret_cast<const float2*>(at);
+    else u[0] = at[0];
+  }
+};
+
+// N values a lane in permuted slots (see StateTile), summed over the L lanes of its set: the first N / L values of lane hl
+// are the sums of its own column and token.
+template <int N, int L>
+__device__ __forceinline__ void permuted_sums(float (&p)[N]) {
+  static_assert(N >= L, "at least one sum a lane");
+  int half = N / 2;
+#pragma unroll
+  for (int o = L / 2; o > 0; o >>= 1, half >>= 1) {
+#pragma unroll
+    for (int s = 0; s < N / 2; ++s) {
+      if (s >= half) break;
+      p[s] += __shfl_xor_sync(0xffffffffu, p[s + half], o);
+    }
+  }
 }
 
-// Sums 2^k values over the 32 lanes of a warp; afterwards lane's first N / 32 values are the sums numbered
-// [first, first + N / 32), first = the return value.
-template <int N>
-__device__ __forceinline__ int scatter_sums_warp(float (&p)[N], int lane) {
-  static_assert(N >= 32, "at least one sum a lane");
-  int first = 0;
+// N values a lane, summed over the L lanes of its set (N >= L); afterwards lane hl's first N / L values are the sums
+// numbered hl * (N / L) onwards.
+template <int N, int L>
+__device__ __forceinline__ void scatter_sums(float (&p)[N], int hl) {
+  static_assert(N >= L, "at least one sum a lane");
+  int half = N / 2;
 #pragma unroll
-  for (int o = 16, half = N / 2; o > 0; o >>= 1, half >>= 1) {
-    const bool up = lane & o;
+  for (int o = L / 2; o > 0; o >>= 1, half >>= 1) {
+    const bool up = hl & o;
 #pragma unroll
     for (int s = 0; s < N / 2; ++s) {
       if (s >= half) break;
       const float keep = up ? p[s + half] : p[s], give = up ? p[s] : p[s + half];
       p[s] = keep + __shfl_xor_sync(0xffffffffu, give, o);
     }
-    if (up) first += half;
   }
-  return first;
 }
 
 // The groups of a step: every entry's tokens in groups of kStateGroup, numbered along the entries.

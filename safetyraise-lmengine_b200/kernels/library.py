@@ -1527,9 +1527,10 @@ class KernelLibrary:
             records = ws.get("channel_delta.records", groups * H, record, torch.float32, reserve=0)
             self._check(self.lib.srlm_channel_delta_groups(
                 _ptr(conv), _ptr(proj), C.c_longlong(proj.stride(0)), _ptr(low), C.c_longlong(low.stride(0)), _ptr(a_log),
-                _ptr(dt_bias), *where, _ptr(records), _ptr(o), C.c_int(groups), *sizes, C.c_float(unit_eps), _stream()),
-                "channel_delta_groups")
-            self.launches += 1           # the walk along the groups
+                _ptr(dt_bias), _ptr(ctx.cu_q), C.c_int(ctx.n_entries), _ptr(records), C.c_int(groups), *sizes,
+                C.c_float(unit_eps), _stream()), "channel_delta_groups")
+            self._check(self.lib.srlm_channel_delta_read(_ptr(records), _ptr(conv), *where, _ptr(o), *sizes, _stream()),
+                        "channel_delta_read")
         else:
             self._check(self.lib.srlm_channel_delta_walk(
                 _ptr(proj), C.c_longlong(proj.stride(0)), _ptr(conv_w), _ptr(low), C.c_longlong(low.stride(0)), _ptr(a_log),
@@ -1546,8 +1547,7 @@ class KernelLibrary:
         T, inner = proj.shape[0], H * P
         channels, carry = inner + 2 * G * N, H * N * P
         sizes = (C.c_int(H), C.c_int(G), C.c_int(N), C.c_int(P))
-        params = (_ptr(dt_bias), _ptr(a_log), _ptr(D), _ptr(state), C.c_longlong(state.stride(0)), _ptr(ctx.cu_q),
-                  _ptr(ctx.slots), C.c_int(ctx.n_entries))
+        where = (_ptr(state), C.c_longlong(state.stride(0)), _ptr(ctx.cu_q), _ptr(ctx.slots), C.c_int(ctx.n_entries))
         record = int(self.lib.srlm_state_space_record(C.c_int(N)))
         groups = self._by_groups(ctx, record)
         if groups:
@@ -1555,13 +1555,14 @@ class KernelLibrary:
             self.short_conv(ctx, proj, inner, channels, conv_w, state, carry, conv, out_bias=conv_b, silu=True)
             records = ctx.workspace.get("state_space.records", groups * H, record, torch.float32, reserve=0)
             self._check(self.lib.srlm_state_space_groups(
-                _ptr(conv), _ptr(proj), C.c_longlong(proj.stride(0)), *params, _ptr(records), _ptr(y), C.c_int(groups), *sizes,
-                _stream()), "state_space_groups")
-            self.launches += 1           # the walk along the groups
+                _ptr(conv), _ptr(proj), C.c_longlong(proj.stride(0)), _ptr(dt_bias), _ptr(a_log), _ptr(ctx.cu_q),
+                C.c_int(ctx.n_entries), _ptr(records), C.c_int(groups), *sizes, _stream()), "state_space_groups")
+            self._check(self.lib.srlm_state_space_read(_ptr(records), _ptr(conv), _ptr(D), *where, _ptr(y), *sizes, _stream()),
+                        "state_space_read")
         else:
             self._check(self.lib.srlm_state_space_walk(
-                _ptr(proj), C.c_longlong(proj.stride(0)), _ptr(conv_w), _ptr(conv_b), *params, _ptr(y), *sizes, C.c_int(taps),
-                _stream()), "state_space_walk")
+                _ptr(proj), C.c_longlong(proj.stride(0)), _ptr(conv_w), _ptr(conv_b), _ptr(dt_bias), _ptr(a_log),
+                _ptr(D), *where, _ptr(y), *sizes, C.c_int(taps), _stream()), "state_space_walk")
         self.conv_carry(ctx, proj, inner, channels, taps, state, carry)
 
     def state_space_output(self, y, proj, weight, eps, out, parts):

@@ -65,8 +65,12 @@ class GatedDense(Part):
 
 @register_feed_forward("dense")
 class Dense(Part):
-    """down(act(up(x))) without a gate; ``activation`` "gelu": the exact one, "relu_squared": max(z, 0)^2.  The first product writes float32 and the
-    activation rounds once, into the second product's input."""
+    """down(act(up(x))) without a gate; ``activation`` "gelu": the exact one, "relu_squared": max(z, 0)^2.  The first
+    product writes float32 and the activation rounds once, into the second product's input; in steps of many tokens the
+    activation rides in the first product's epilogue (the grouped tensor-memory product with one group), where the sum is
+    float32 too."""
+
+    FUSED_TOKENS = 256       # least tokens of a step whose activation rides in the product
 
     def __init__(self, spec, prefix: str, tensors: dict, mctx):
         if spec.activation not in ("gelu", "relu_squared"):
@@ -74,6 +78,9 @@ class Dense(Part):
         self.spec = spec
         nm = spec.dense_names
         self.up = Linear(tensors[prefix + nm.up], prefix + nm.up)
+        w = self.up.weight
+        self.fused = mctx.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.shape[0] % 8 == 0 and w.shape[1] % 8 == 0
+        self.one_group = torch.zeros(-(-mctx.max_batch_tokens // ops.GROUPED_TILE) + 1, dtype=torch.int32, device=mctx.device)
         self.down = Linear(tensors[prefix + nm.down], prefix + nm.down)
 
     @classmethod
@@ -83,7 +90,14 @@ class Dense(Part):
                 TensorDecl(prefix + nm.down, (spec.hidden_size, spec.intermediate_size), MATRIX)]
 
     def forward(self, ctx, x: torch.Tensor) -> torch.Tensor:
-        z = self.up(ctx, x, "dense.z", out_dtype=torch.float32)
-        h = ctx.workspace.get("dense.h", x.shape[0], self.spec.intermediate_size, ctx.dtype)
-        ops.activation(z, h, self.spec.activation)
+        T, (I, H) = x.shape[0], self.up.weight.shape
+        h = ctx.workspace.get("dense.h", T, I, ctx.dtype)
+        tile = ops.grouped_tile_rows(T, 1, I * H)
+        if (self.fused and ops.grouped_products_in_tensor_memory and T >= self.FUSED_TOKENS
+                and self.one_group.numel() * tile >= T):
+            ops.gemm_tn_tcgen05_grouped(x, self.up.weight.view(1, I, H), h, self.one_group, act=self.spec.activation,
+                                        tile_rows=tile)
+        else:
+            z = self.up(ctx, x, "dense.z", out_dtype=torch.float32)
+            ops.activation(z, h, self.spec.activation)
         return self.down(ctx, h, "dense.down")
