@@ -667,10 +667,11 @@ def lokizen_config(size: dict, kinds) -> dict:
 
 def mapovik_config(size: dict, kinds) -> dict:
     """A Mapovik configuration whose layers have the sizes of a Qwen3 layer of the same width: a delta rule of as many heads
-    of 128 x 128 with half as many q / k heads, 4 taps and low-rank projections of the generated rank, 32; a 'parallel' layer of attention with
-    heads of 128, half of each rotated, beside a state space of two widths of channels in heads of 64 with 128 states, 4
-    taps; 16 gated experts of three quarters of a width of which a token's row of a table names 4, or ('... dense') a dense
-    feed-forward of four and a half widths without a gate.  'loop' in the list: the layer behind it runs twice."""
+    of 128 x 128 with half as many q / k heads, 4 taps and low-rank projections of the rank that generated weights get, 32; a
+    'parallel' layer of attention with heads of 128, half of each rotated, beside a state space of two widths of channels in
+    heads of 64 with 128 states, 4 taps; 16 gated experts of three quarters of a width of which a token's row of a table
+    names 4, or ('... dense') a dense feed-forward of four and a half widths without a gate.  'loop' in the list: the layer
+    behind it runs twice."""
     W, H, G = size["width"], size["heads"], size["kv_heads"]
     mixers = {
         "channel_delta": {"heads": H, "kv_heads": H // 2, "dim": 128, "vdim": 128, "conv": 4},
