@@ -6,7 +6,7 @@ convolution over time and silu, beta = logistic(W_b x), g = exp(-exp(A_h) softpl
 
     S <- diag(g) S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
 
-so the read-out sees the token's own write.  o is RMS-normed per head, scaled by a weight shared by the heads and by
+what a token writes is in its own read-out.  o is RMS-normed per head, scaled by a weight shared by the heads and by
 logistic(W_g2 W_g1 x), then projected.  Value head h reads q / k head h // (heads / kv_heads).
 
 One stacked projection gives q | k | v | beta | decay's and gate's low-rank parts, a second, block-diagonal one, gives

@@ -29,7 +29,7 @@ class TensorDecl:
     role: str = MATRIX        # MATRIX | VECTOR (norm scale) | TABLE (embedding rows) | INT_TABLE
     free_size: int = 32       # what a free dimension is made as where weights are generated and not read
     below: int = 2 ** 31 - 1  # INT_TABLE: entries lie in [0, below) ...
-    distinct: bool = False    # ... and the entries of a row differ
+    distinct: bool = False    # ... and no row holds one of them twice
 
     @property
     def made_shape(self) -> Tuple[int, ...]:
